@@ -8,7 +8,7 @@ differs from the keys'; none for a need with `values=False`: one vector per
 token that serves as both), a free list of pages and one page
 table `[slots, max_pages]`.  A sequence holds a slot, and in every group the
 pages that cover its length; groups with a window give pages back once every
-key in them has left the window.  Slots and pages go back to the free lists
+key in them has left the window (except those of the first `keep_first` tokens).  Slots and pages go back to the free lists
 when a sequence ends and are handed out again.  Next to the pages lies
 fixed-size per-sequence state `[slots, ...]` for sites that declare some; it
 is zeroed when a slot is taken.
@@ -36,6 +36,7 @@ class KVNeed:
     window: int = 0          # 0: every key is kept; n: only the last n keys are read
     values: bool = True      # False: one vector per token only (a latent that serves as key and value)
     v_dim: int = 0           # size of a value head when it differs from the key's (0: the same)
+    keep_first: int = 0      # with a window: the first tokens' keys stay visible to every later token
 
 
 @dataclass(frozen=True)
@@ -64,6 +65,7 @@ class CacheGroup:
         self.n_pages, self.page_size, self.max_pages = n_pages, page_size, max_pages
         self.pages = FreeList(n_pages, "cache page")
         self.table_host = np.zeros((n_slots, max_pages), dtype=np.int32)
+        self.kept_pages = -(-need.keep_first // page_size)  # pages at a sequence's start that never leave the window
         self.seq_pages: dict[int, dict[int, int]] = {}      # slot -> {page index in sequence: page}
         self.dirty: set[int] = set()
         shape = (len(sites), n_pages, page_size, need.n_kv_heads, need.head_dim)
@@ -98,12 +100,13 @@ class CacheGroup:
             self.dirty.add(slot)
 
     def trim(self, slot: int, length: int) -> None:
-        """Give back pages whose keys have all left the window of every later token."""
+        """Give back pages whose keys have all left the window of every later token (the first tokens that the need
+        keeps stay)."""
         if not self.need.window:
             return
         have = self.seq_pages.get(slot, {})
         first_live = max(0, length + 1 - self.need.window) // self.page_size
-        for p in [p for p in have if p < first_live]:
+        for p in [p for p in have if self.kept_pages <= p < first_live]:
             self.pages.release(have.pop(p))
 
     def release(self, slot: int) -> None:

@@ -3,7 +3,7 @@ from __future__ import annotations
 
 import os
 from dataclasses import dataclass
-from typing import Any, Callable
+from typing import Any, Callable, Optional
 
 from ..registry import ARCHITECTURES, RegistryError
 from ..spec import ModelSpec
@@ -16,6 +16,9 @@ class Architecture:
     name: str
     config_from_dict: Callable[[dict], Any]
     describe: Callable[[Any], ModelSpec]     # typed config -> ModelSpec
+    # (config.json's dict, tensor name -> shape) -> the dict with the sizes filled in that config.json leaves to the
+    # tensors' shapes; None: config.json gives every size
+    sizes_from_shapes: Optional[Callable[[dict, dict], dict]] = None
 
 
 def architecture_name(raw: dict) -> str:
@@ -29,10 +32,14 @@ def architecture_name(raw: dict) -> str:
 
 
 def load_config(model_dir_or_dict):
-    """Read config.json (or take its dict) and return (Architecture, typed config)."""
-    raw = (read_config_json(model_dir_or_dict)
-           if isinstance(model_dir_or_dict, (str, os.PathLike)) else dict(model_dir_or_dict))
+    """Read config.json (or take its dict) and return (Architecture, typed config).  An architecture whose config.json
+    leaves sizes to the tensors' shapes gets them from the folder's headers, where there are any."""
+    is_dir = isinstance(model_dir_or_dict, (str, os.PathLike))
+    raw = read_config_json(model_dir_or_dict) if is_dir else dict(model_dir_or_dict)
     arch = ARCHITECTURES.get(architecture_name(raw))
+    if is_dir and arch.sizes_from_shapes is not None:
+        from ..weights import stored_shapes
+        raw = arch.sizes_from_shapes(raw, stored_shapes(os.fspath(model_dir_or_dict)))
     return arch, arch.config_from_dict(raw)
 
 
@@ -41,10 +48,12 @@ from . import gevonex_arch  # noqa: E402,F401  registers the Gevonex architectur
 from . import mogevik_arch  # noqa: E402,F401  registers the Mogevik architecture
 from . import tubusun_arch  # noqa: E402,F401  registers the Tubusun architecture
 from . import fizadra_arch  # noqa: E402,F401  registers the Fizadra architecture
+from . import degavik_arch  # noqa: E402,F401  registers the Degavik architecture
+from .degavik import DegavikConfig  # noqa: E402
 from .fizadra import FizadraConfig  # noqa: E402
 from .gevonex import GevonexConfig  # noqa: E402
 from .mogevik import MogevikConfig  # noqa: E402
 from .tubusun import TubusunConfig  # noqa: E402
 
-__all__ = ["Architecture", "ConfigError", "FizadraConfig", "GevonexConfig", "LlamaConfig", "MogevikConfig", "RopeScaling", "RegistryError", "TubusunConfig",
+__all__ = ["Architecture", "ConfigError", "DegavikConfig", "FizadraConfig", "GevonexConfig", "LlamaConfig", "MogevikConfig", "RopeScaling", "RegistryError", "TubusunConfig",
            "architecture_name", "load_config", "read_config_json"]

@@ -84,11 +84,12 @@ head_gate_kernel(T* __restrict__ out, const T* __restrict__ gate, int gate_strid
     }
 }
 
-// `partial` [splits][rows][width]: y is first completed by the partial sums a K-split product left (in split order).
-template <typename TW>
+// `partial` [splits][rows][width]: y is first completed by the partial sums a K-split product left (in split order), or
+// with `only_partial` it is their sum.  `copy`: the new x in the compute dtype, for sublayers that read the stream itself.
+template <typename TW, typename TC>
 __global__ void __launch_bounds__(256)
 rmsnorm_add_kernel(float* __restrict__ x, float* __restrict__ y, const float* __restrict__ partial, int splits,
-                   size_t split_stride, const TW* __restrict__ w, int width, float eps) {
+                   size_t split_stride, int only_partial, const TW* __restrict__ w, int width, float eps, TC* __restrict__ copy) {
     chain_release();
     chain_wait();
     __shared__ float scratch[32];
@@ -96,14 +97,26 @@ rmsnorm_add_kernel(float* __restrict__ x, float* __restrict__ y, const float* __
     float* yr = y + t * width;
     float sq = 0.f;
     for (int e = threadIdx.x; e < width; e += blockDim.x) {
-        float v = yr[e];
+        float v = only_partial ? 0.f : yr[e];
         for (int s = 0; s < splits; ++s) v += partial[(size_t)s * split_stride + t * width + e];
         if (splits > 0) yr[e] = v;
         sq = fmaf(v, v, sq);
     }
     const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)width + eps);
     float* xr = x + t * width;
-    for (int e = threadIdx.x; e < width; e += blockDim.x) xr[e] += yr[e] * inv * to_float(w[e]);
+    for (int e = threadIdx.x; e < width; e += blockDim.x) {
+        const float v = xr[e] + yr[e] * inv * to_float(w[e]);
+        xr[e] = v;
+        if (copy != nullptr) copy[t * width + e] = from_float<TC>(v);
+    }
+}
+
+// out = x in the compute dtype
+__global__ void __launch_bounds__(256)
+copy_rows_kernel(const float* __restrict__ x, __nv_bfloat16* __restrict__ out, long n) {
+    chain_release();
+    chain_wait();
+    for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long)gridDim.x * blockDim.x) out[i] = __float2bfloat16_rn(x[i]);
 }
 
 // y[t] += a * z[t]
@@ -151,15 +164,25 @@ int mdma_head_gate(void* out, const void* gate, int dtype, int gate_stride, int 
     return 0;
 }
 
-int mdma_rmsnorm_add(float* x, float* y, const float* partial, int splits, long split_stride, const void* w, int w_dtype,
-                     int n_rows, int width, float eps, cudaStream_t stream) {
+int mdma_rmsnorm_add(float* x, float* y, const float* partial, int splits, long split_stride, int only_partial, const void* w,
+                     int w_dtype, int n_rows, int width, float eps, void* copy, int copy_dtype, cudaStream_t stream) {
     MDMA_REQUIRE(n_rows >= 0 && width > 0, "rmsnorm_add: bad sizes");
     MDMA_REQUIRE(splits >= 0 && (splits == 0 || partial), "rmsnorm_add: partial sums need a pointer");
     if (n_rows == 0) return 0;
-    MDMA_DISPATCH_DTYPE(w_dtype, TW,
-        launch_chained(rmsnorm_add_kernel<TW>, dim3(n_rows), dim3(256), 0, stream, x, y, partial, splits, (size_t)split_stride,
-                       (const TW*)w, width, eps));
+    MDMA_DISPATCH_DTYPE(w_dtype, TW, MDMA_DISPATCH_DTYPE(copy_dtype, TC,
+        launch_chained(rmsnorm_add_kernel<TW, TC>, dim3(n_rows), dim3(256), 0, stream, x, y, partial, splits, (size_t)split_stride,
+                       only_partial, (const TW*)w, width, eps, (TC*)copy)));
     MDMA_LAUNCH_OK("rmsnorm_add");
+    return 0;
+}
+
+// out [n] bfloat16 = x [n]
+int mdma_copy_rows(const float* x, void* out, long n, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    long blocks = (n + 255) / 256;
+    if (blocks > 1184) blocks = 1184;
+    launch_chained(copy_rows_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, x, (__nv_bfloat16*)out, n);
+    MDMA_LAUNCH_OK("copy_rows");
     return 0;
 }
 

@@ -1,6 +1,7 @@
 // Linear attention with a fixed decay per head, and the gated norm that follows it.
 //
-// Per head, with q, k [dim] and v [vdim] of a token (each the SiLU of its projection, taken in float):
+// Per head, with q, k [dim] and v [vdim] of a token (each the SiLU of its projection, taken in float, or the projection
+// itself; q and k may be turned by the token's position, in float, and k multiplied by a constant: `LinInput`):
 //     S_t = decay * S_(t-1) + k_t v_t^T          S [dim][vdim], floats, carried from token to token per sequence
 //     o_t = S_t^T q_t
 // The columns of S do not touch one another, so a block owns one (sequence, head, part of the columns).
@@ -24,12 +25,36 @@ namespace mdma {
 
 __device__ __forceinline__ float silu_float(float z) { return z / (1.0f + expf(-z)); }
 
+// What happens to a token's projections before they enter the recurrence: SiLU or nothing; the first 2 * half numbers of
+// every q and k head turned by the token's position (pairs (i, i + half), or (2i, 2i + 1) if interleaved; half 0: none);
+// k times k_scale.
+struct LinInput {
+    int silu, half, interleaved;
+    float k_scale;
+    const float* inv_freq;       // [half]
+    const int* tok_pos;
+};
+__device__ __forceinline__ float lin_act(float z, int silu) { return silu ? silu_float(z) : z; }
+// number d of a q or k head whose projection starts at `head`
+template <typename T>
+__device__ __forceinline__ float lin_qk(const T* __restrict__ head, int d, int pos, const LinInput& in) {
+    const float x = lin_act(to_float(head[d]), in.silu);
+    if (d >= 2 * in.half) return x;
+    const bool second = in.interleaved ? (d & 1) : d >= in.half;
+    const int pair = in.interleaved ? d >> 1 : (second ? d - in.half : d);
+    const int other = in.interleaved ? d ^ 1 : (second ? d - in.half : d + in.half);
+    const float y = lin_act(to_float(head[other]), in.silu);
+    float sn, cs;
+    sincosf((float)pos * in.inv_freq[pair], &sn, &cs);
+    return second ? fmaf(x, cs, y * sn) : fmaf(x, cs, -(y * sn));
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 linear_attention_scan_kernel(const T* __restrict__ proj, int row_stride, int q_col, int k_col, int v_col,
                              const float* __restrict__ decay, const int* __restrict__ seq_start,
                              const int* __restrict__ seq_slot, float* __restrict__ state, size_t state_stride,
-                             float* __restrict__ out, int heads, int dim, int vdim, int cols) {
+                             float* __restrict__ out, int heads, int dim, int vdim, int cols, LinInput in) {
     chain_release();
     chain_wait();
     extern __shared__ float sm[];
@@ -50,11 +75,12 @@ linear_attention_scan_kernel(const T* __restrict__ proj, int row_stride, int q_c
     const float dk = decay[h];
     for (int t = t0; t < t1; ++t) {
         const T* row = proj + (size_t)t * row_stride;
+        const int pos = in.half ? in.tok_pos[t] : 0;
         for (int e = threadIdx.x; e < dim; e += blockDim.x) {
-            sq[e] = silu_float(to_float(row[q_col + h * dim + e]));
-            sk[e] = silu_float(to_float(row[k_col + h * dim + e]));
+            sq[e] = lin_qk(row + q_col + h * dim, e, pos, in);
+            sk[e] = lin_qk(row + k_col + h * dim, e, pos, in) * in.k_scale;
         }
-        for (int e = threadIdx.x; e < cw; e += blockDim.x) sv[e] = silu_float(to_float(row[v_col + h * vdim + c0 + e]));
+        for (int e = threadIdx.x; e < cw; e += blockDim.x) sv[e] = lin_act(to_float(row[v_col + h * vdim + c0 + e]), in.silu);
         __syncthreads();
         if (active) {
             const float vj = sv[j];
@@ -90,7 +116,7 @@ __global__ void __launch_bounds__(256)
 linear_attention_step_kernel(const T* __restrict__ proj, int row_stride, int q_col, int k_col, int v_col,
                              const float* __restrict__ decay, const int* __restrict__ seq_start,
                              const int* __restrict__ seq_slot, float* __restrict__ state, size_t state_stride,
-                             float* __restrict__ out, int heads, int dim, int vdim) {
+                             float* __restrict__ out, int heads, int dim, int vdim, LinInput in) {
     chain_release();
     chain_wait();
     extern __shared__ float sm[];
@@ -108,11 +134,12 @@ linear_attention_step_kernel(const T* __restrict__ proj, int row_stride, int q_c
     const float dk = decay[h];
     for (int t = t0; t < t1; ++t) {
         const T* row = proj + (size_t)t * row_stride;
+        const int pos = in.half ? in.tok_pos[t] : 0;
         for (int e = threadIdx.x; e < dim; e += blockDim.x) {
-            sq[e] = silu_float(to_float(row[q_col + h * dim + e]));
-            sk[e] = silu_float(to_float(row[k_col + h * dim + e]));
+            sq[e] = lin_qk(row + q_col + h * dim, e, pos, in);
+            sk[e] = lin_qk(row + k_col + h * dim, e, pos, in) * in.k_scale;
         }
-        if (threadIdx.x < kStepCols) sv[threadIdx.x] = c0 + threadIdx.x < vdim ? silu_float(to_float(row[v_col + h * vdim + c0 + threadIdx.x])) : 0.f;
+        if (threadIdx.x < kStepCols) sv[threadIdx.x] = c0 + threadIdx.x < vdim ? lin_act(to_float(row[v_col + h * vdim + c0 + threadIdx.x]), in.silu) : 0.f;
         __syncthreads();
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
         if (active) {
@@ -172,12 +199,17 @@ __device__ __forceinline__ void copy16_async(void* dst_shared, const void* src_g
 }
 __device__ __forceinline__ void copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
-// eight bfloat16 -> the SiLU of each, times `f`, as two float4
-__device__ __forceinline__ void silu8(const uint4& raw, float f, float4& lo, float4& hi) {
+// eight bfloat16 -> the SiLU of each (or itself), times `f`, as two float4
+__device__ __forceinline__ void act8(const uint4& raw, float f, int silu, float4& lo, float4& hi) {
     const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
     const float2 a = __bfloat1622float2(p[0]), b = __bfloat1622float2(p[1]), c = __bfloat1622float2(p[2]), d = __bfloat1622float2(p[3]);
-    lo = make_float4(silu_float(a.x) * f, silu_float(a.y) * f, silu_float(b.x) * f, silu_float(b.y) * f);
-    hi = make_float4(silu_float(c.x) * f, silu_float(c.y) * f, silu_float(d.x) * f, silu_float(d.y) * f);
+    if (silu) {
+        lo = make_float4(silu_float(a.x) * f, silu_float(a.y) * f, silu_float(b.x) * f, silu_float(b.y) * f);
+        hi = make_float4(silu_float(c.x) * f, silu_float(c.y) * f, silu_float(d.x) * f, silu_float(d.y) * f);
+    } else {
+        lo = make_float4(a.x * f, a.y * f, b.x * f, b.y * f);
+        hi = make_float4(c.x * f, c.y * f, d.x * f, d.y * f);
+    }
 }
 
 template <typename T, int PASS>
@@ -186,7 +218,7 @@ linear_attention_chunk_kernel(const T* __restrict__ proj, int row_stride, int q_
                               const float* __restrict__ decay, const int* __restrict__ seq_start,
                               const int* __restrict__ seq_slot, float* __restrict__ state, size_t state_stride,
                               float* __restrict__ out, int heads, int dim, int vdim, int cols, int run_rows, int max_runs,
-                              float* __restrict__ run_state, int staged) {
+                              float* __restrict__ run_state, int staged, LinInput in) {
     chain_release();
     chain_wait();
     extern __shared__ __align__(16) float sm[];
@@ -300,17 +332,17 @@ linear_attention_chunk_kernel(const T* __restrict__ proj, int row_stride, int q_
                 const int i = e / d8, p = (e % d8) << 3;
                 float4 lo = make_float4(0.f, 0.f, 0.f, 0.f), hi = lo;
                 if (PASS != kLinLocal) {
-                    if (i < n) silu8(*reinterpret_cast<const uint4*>(rq + i * dim + p), 1.0f, lo, hi);
+                    if (i < n) act8(*reinterpret_cast<const uint4*>(rq + i * dim + p), 1.0f, in.silu, lo, hi);
                     st4(sq + i * kd + p, lo); st4(sq + i * kd + p + 4, hi);
                     lo = make_float4(0.f, 0.f, 0.f, 0.f); hi = lo;
                 }
-                if (i < n) silu8(*reinterpret_cast<const uint4*>(rk + i * dim + p), 1.0f, lo, hi);
+                if (i < n) act8(*reinterpret_cast<const uint4*>(rk + i * dim + p), in.k_scale, in.silu, lo, hi);
                 st4(sk + i * kd + p, lo); st4(sk + i * kd + p + 4, hi);
             }
             for (int e = threadIdx.x; e < kChunk * (colsP >> 3); e += blockDim.x) {
                 const int i = e / (colsP >> 3), p = (e % (colsP >> 3)) << 3;
                 float4 lo = make_float4(0.f, 0.f, 0.f, 0.f), hi = lo;
-                if (i < n && p < cw) silu8(*reinterpret_cast<const uint4*>(rv + i * cols + p), PASS == kLinLocal ? rowf[i] : 1.0f, lo, hi);
+                if (i < n && p < cw) act8(*reinterpret_cast<const uint4*>(rv + i * cols + p), PASS == kLinLocal ? rowf[i] : 1.0f, in.silu, lo, hi);
                 st4(sv + i * colsP + p, lo); st4(sv + i * colsP + p + 4, hi);
             }
             __syncthreads();
@@ -320,13 +352,32 @@ linear_attention_chunk_kernel(const T* __restrict__ proj, int row_stride, int q_
                 const int i = e / dimP, d = e % dimP;
                 const bool have = i < n && d < dim;
                 const size_t at = (size_t)(r0 + i) * row_stride + d;
-                if (PASS != kLinLocal) sq[i * kd + d] = have ? silu_float(to_float(qbase[at])) : 0.f;
-                sk[i * kd + d] = have ? silu_float(to_float(kbase[at])) : 0.f;
+                if (PASS != kLinLocal) sq[i * kd + d] = have ? lin_act(to_float(qbase[at]), in.silu) : 0.f;
+                sk[i * kd + d] = have ? lin_act(to_float(kbase[at]), in.silu) * in.k_scale : 0.f;
             }
             for (int e = threadIdx.x; e < kChunk * colsP; e += blockDim.x) {
                 const int i = e / colsP, c = e % colsP;
                 const float f = PASS == kLinLocal ? rowf[i] : 1.0f;
-                sv[e] = (i < n && c < cw) ? silu_float(to_float(vbase[(size_t)(r0 + i) * row_stride + c])) * f : 0.f;
+                sv[e] = (i < n && c < cw) ? lin_act(to_float(vbase[(size_t)(r0 + i) * row_stride + c]), in.silu) * f : 0.f;
+            }
+            __syncthreads();
+        }
+        if (in.half > 0) {     // turn q and k where they lie: a thread a pair, one angle for both
+            for (int e = threadIdx.x; e < n * in.half; e += blockDim.x) {
+                const int i = e / in.half, p = e - i * in.half;
+                const int d0 = in.interleaved ? 2 * p : p, d1 = in.interleaved ? 2 * p + 1 : p + in.half;
+                float sn, cs;
+                sincosf((float)in.tok_pos[r0 + i] * in.inv_freq[p], &sn, &cs);
+                float* kr = sk + i * kd;
+                const float a = kr[d0], b = kr[d1];
+                kr[d0] = fmaf(a, cs, -(b * sn));
+                kr[d1] = fmaf(b, cs, a * sn);
+                if (PASS != kLinLocal) {
+                    float* qr = sq + i * kd;
+                    const float u = qr[d0], v = qr[d1];
+                    qr[d0] = fmaf(u, cs, -(v * sn));
+                    qr[d1] = fmaf(v, cs, u * sn);
+                }
             }
             __syncthreads();
         }
@@ -467,7 +518,7 @@ int mdma_linear_attention_fits(int dim, int vdim, int chunked) {
     return (chunked ? chunk_smem(dim, cols) : scan_smem(dim, cols)) <= kLinSmemMost ? 1 : 0;
 }
 
-// proj rows hold q at q_col + head * dim, k at k_col + head * dim, v at v_col + head * vdim (before their SiLU);
+// proj rows hold q at q_col + head * dim, k at k_col + head * dim, v at v_col + head * vdim (before what `LinInput` names);
 // state [slots][heads * dim * vdim] floats; out [n_tokens][heads * vdim] floats.  chunked == 0: row by row.
 // chunked == 2 (kLinSingleRows): the kernel for steps of one row a sequence (row by row where the state's layout does
 // not allow its 16-byte accesses).  chunked == 1: a chunk of rows at a time, and with run_rows > 0 in runs of that many rows side by side
@@ -475,7 +526,11 @@ int mdma_linear_attention_fits(int dim, int vdim, int chunked) {
 int mdma_linear_attention(const void* proj, int dtype, int row_stride, int q_col, int k_col, int v_col, const float* decay,
                           const int* seq_start, const int* seq_slot, float* state, long state_stride, float* out,
                           int n_seqs, int heads, int dim, int vdim, int chunked, int run_rows, int max_runs,
-                          float* scratch, long scratch_floats, cudaStream_t stream) {
+                          float* scratch, long scratch_floats, int silu, int rotary_dim, int interleaved,
+                          const float* inv_freq, const int* tok_pos, float k_scale, cudaStream_t stream) {
+    MDMA_REQUIRE(rotary_dim >= 0 && rotary_dim % 2 == 0 && rotary_dim <= dim && (rotary_dim == 0 || (inv_freq && tok_pos)),
+                 "linear_attention: %d turned numbers of a head of %d", rotary_dim, dim);
+    const LinInput in = {silu, rotary_dim / 2, interleaved, k_scale, inv_freq, tok_pos};
     MDMA_REQUIRE(n_seqs >= 0 && heads > 0 && dim > 0 && vdim > 0, "linear_attention: bad sizes");
     MDMA_REQUIRE(n_seqs <= 65535 * 32 && heads <= 65535, "linear_attention: too many sequences or heads");
     if (n_seqs == 0) return 0;
@@ -487,7 +542,7 @@ int mdma_linear_attention(const void* proj, int dtype, int row_stride, int q_col
             dim3 step_grid(n_seqs, heads, (vdim + kStepCols - 1) / kStepCols);
             MDMA_DISPATCH_DTYPE(dtype, T, {
                 launch_chained(linear_attention_step_kernel<T>, step_grid, dim3(256), step_smem, stream, (const T*)proj, row_stride,
-                               q_col, k_col, v_col, decay, seq_start, seq_slot, state, (size_t)state_stride, out, heads, dim, vdim);
+                               q_col, k_col, v_col, decay, seq_start, seq_slot, state, (size_t)state_stride, out, heads, dim, vdim, in);
             });
             MDMA_LAUNCH_OK("linear_attention (single rows)");
             return 0;
@@ -503,7 +558,7 @@ int mdma_linear_attention(const void* proj, int dtype, int row_stride, int q_col
             static bool raised = false;
             if (!raised) { cudaFuncSetAttribute(linear_attention_scan_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLinSmemMost); raised = true; }
             launch_chained(linear_attention_scan_kernel<T>, grid, dim3(256), smem, stream, (const T*)proj, row_stride, q_col,
-                           k_col, v_col, decay, seq_start, seq_slot, state, (size_t)state_stride, out, heads, dim, vdim, cols);
+                           k_col, v_col, decay, seq_start, seq_slot, state, (size_t)state_stride, out, heads, dim, vdim, cols, in);
         });
         MDMA_LAUNCH_OK("linear_attention (row by row)");
         return 0;
@@ -525,7 +580,7 @@ int mdma_linear_attention(const void* proj, int dtype, int row_stride, int q_col
         if (!raised) { cudaFuncSetAttribute(linear_attention_chunk_kernel<T, PASS_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLinSmemMost); raised = true; } \
         launch_chained(linear_attention_chunk_kernel<T, PASS_>, grid, dim3(256), smem, stream, (const T*)proj, row_stride, \
                        q_col, k_col, v_col, decay, seq_start, seq_slot, state, (size_t)state_stride, out, heads, dim, vdim, \
-                       cols, run_rows, max_runs, scratch, staged);                                                        \
+                       cols, run_rows, max_runs, scratch, staged, in);                                                        \
     });                                                                                                                   \
     MDMA_LAUNCH_OK(what)
     if (run_rows > 0) {

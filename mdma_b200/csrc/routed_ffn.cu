@@ -1,7 +1,7 @@
 // A feed-forward made of many small gated feed-forwards ("experts") of which each token uses a few.
 //
 // Router (one block per token, float arithmetic):
-//     z = R h                              logits over all routed outputs (experts, then identity experts)
+//     z = R h (+ bias)                     logits over all routed outputs (experts, then identity experts)
 //     s = softmax(z), or sigmoid(z) element by element (`scoring` 1)
 //     c = s + correction                   choice scores
 //     experts form `n_groups` equal groups of neighbours; a group's score is the sum of its `group_top`
@@ -66,7 +66,7 @@ template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(256)
 route_kernel(const TA* __restrict__ h, int h_stride, const TW* __restrict__ router, const TC* __restrict__ correction,
              const TW* __restrict__ shared_gate, int width, int n_routed, int top, int n_groups, int keep_groups,
-             int scoring, int group_top, int renormalize,
+             int scoring, int group_top, int renormalize, int logit_bias,
              int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ shared_scale) {
     chain_release();
     chain_wait();
@@ -77,7 +77,7 @@ route_kernel(const TA* __restrict__ h, int h_stride, const TW* __restrict__ rout
     const TA* row = h + (size_t)t * h_stride;
     for (int e = warp; e < n_routed; e += n_warps) {
         const float v = warp_dot(row, router + (size_t)e * width, width, lane);
-        if (lane == 0) z[e] = v;
+        if (lane == 0) z[e] = v + (logit_bias ? to_float(correction[e]) : 0.f);
     }
     if (shared_gate != nullptr && warp == n_warps - 1) {
         const float v = warp_dot(row, shared_gate, width, lane);
@@ -95,7 +95,7 @@ route_kernel(const TA* __restrict__ h, int h_stride, const TW* __restrict__ rout
         for (int e = 0; e < n_routed; ++e) { z[e] = expf(z[e] - m); sum += z[e]; }
         for (int e = 0; e < n_routed; ++e) z[e] = z[e] / sum;
     }
-    for (int e = 0; e < n_routed; ++e) c[e] = z[e] + (correction ? to_float(correction[e]) : 0.f);   // z: s; c: choice score
+    for (int e = 0; e < n_routed; ++e) c[e] = z[e] + (correction && !logit_bias ? to_float(correction[e]) : 0.f);   // z: s; c: choice score
     if (n_groups > 1 && keep_groups < n_groups) {
         const int per = n_routed / n_groups;
         // the best group not yet kept is looked for keep_groups times (ties: the lower number); a bit per group
@@ -446,8 +446,9 @@ extern "C" {
 
 int mdma_route(const void* h, int h_dtype, int h_stride, const void* router, int w_dtype, const void* correction,
                int c_dtype, const void* shared_gate, int n_tokens, int width, int n_routed, int top, int n_groups,
-               int keep_groups, int scoring, int group_top, int renormalize, int* chosen, float* weights,
+               int keep_groups, int scoring, int group_top, int renormalize, int logit_bias, int* chosen, float* weights,
                float* shared_scale, cudaStream_t stream) {
+    MDMA_REQUIRE(!logit_bias || correction, "route: a bias on the logits needs its numbers");
     MDMA_REQUIRE(scoring >= 0 && scoring <= 1 && group_top >= 1 && group_top <= kMaxGroupTop,
                  "route: scoring %d, a group's score over its %d largest (at most %d)", scoring, group_top, kMaxGroupTop);
     MDMA_REQUIRE(n_tokens >= 0 && width > 0, "route: bad sizes");
@@ -461,7 +462,7 @@ int mdma_route(const void* h, int h_dtype, int h_stride, const void* router, int
         MDMA_DISPATCH_DTYPE(c_dtype, TC,
             launch_chained(route_kernel<TA, TW, TC>, dim3(n_tokens), dim3(256), 0, stream, (const TA*)h, h_stride,
                            (const TW*)router, (const TC*)correction, (const TW*)shared_gate, width, n_routed, top,
-                           n_groups, keep_groups, scoring, group_top, renormalize, chosen, weights, shared_scale)));
+                           n_groups, keep_groups, scoring, group_top, renormalize, logit_bias, chosen, weights, shared_scale)));
     MDMA_LAUNCH_OK("route");
     return 0;
 }

@@ -160,6 +160,8 @@ class DecoderModel:
         and into it; write logits of ctx.want_rows into `logits` [n_want, vocab]."""
         x = ctx.buf("x", self.spec.hidden_size, torch.float32)
         self.embedding.forward(ctx, ctx.ids, x)
+        # whether the block before left a copy of x in the compute dtype (`leaves_stream_copy`)
+        ctx.stream_copied = False
         x0 = None
         if self.keeps_embedding:
             x0 = ctx.buf("x_embedded", self.spec.hidden_size, torch.float32)
@@ -172,17 +174,20 @@ class DecoderModel:
                     from .. import ops_tensor
                     ops_tensor.flush_pending(x.device, ctx.rt.tc)
                 self.junctions[entry.junction].forward(ctx, x, x0, entry.junction_arg)
+                ctx.stream_copied = False
             if ctx.rt.gemm == "tensor" and not getattr(block, "handles_pending", False):
                 # a product of the block before may have left partial sums of x for a norm to add up; an
                 # arrangement that does not know of that gets x complete
                 from .. import ops_tensor
                 ops_tensor.flush_pending(x.device, ctx.rt.tc)
             block.forward(ctx, x, cache.view(site, state_site=n), owns_cache=entry.cache is None)
+            ctx.stream_copied = getattr(block, "leaves_stream_copy", False)
             if entry.after is not None:
                 if ctx.rt.gemm == "tensor":
                     from .. import ops_tensor
                     ops_tensor.flush_pending(x.device, ctx.rt.tc)
                 self.junctions[entry.after].forward(ctx, x, x0, n)
+                ctx.stream_copied = False
             if self.on_layer is not None:
                 if ctx.rt.gemm == "tensor":
                     from .. import ops_tensor

@@ -548,11 +548,14 @@ def attention_distance(q, k_cache, v_cache, ctx, page_table, max_pages: int, pag
 
 # ---- routed feed-forward (csrc/routed_ffn.cu) -----------------------------------------------------------------------
 def route(h, router, correction, shared_gate, n_tokens: int, top: int, n_groups: int, keep_groups: int, chosen, weights,
-          shared_scale, scoring: str = "softmax", group_top: int = 1, renormalize: bool = True) -> None:
+          shared_scale, scoring: str = "softmax", group_top: int = 1, renormalize: bool = True, logit_bias=None) -> None:
     """Per token: scores over the router's logits (`scoring`: "softmax" over all, or "sigmoid" of each), choice among the
     best groups (a group's score: the sum of its `group_top` largest), `top` experts and their weights (their scores,
-    divided by their sum if `renormalize`); with `shared_gate` [width] also sigmoid(shared_gate . h) into `shared_scale`."""
-    assert scoring in ("softmax", "sigmoid")
+    divided by their sum if `renormalize`); with `shared_gate` [width] also sigmoid(shared_gate . h) into `shared_scale`.
+    `logit_bias` [n_routed] (in the place of `correction`) joins the logits themselves."""
+    assert scoring in ("softmax", "sigmoid") and (correction is None or logit_bias is None)
+    biased = logit_bias is not None
+    correction = logit_bias if biased else correction
     _need_cuda(h, router, correction, shared_gate, chosen, weights, shared_scale)
     n_routed, width = router.shape
     assert h.stride(1) == 1 and h.shape[1] == width and router.is_contiguous()
@@ -562,7 +565,7 @@ def route(h, router, correction, shared_gate, n_tokens: int, top: int, n_groups:
     _call("core", "mdma_route", _ptr(h), _i(dtype_code(h.dtype)), _i(h.stride(0)), _ptr(router), _i(dtype_code(router.dtype)),
           _ptr(correction), _i(dtype_code(correction.dtype) if correction is not None else F32), _ptr(shared_gate),
           _i(n_tokens), _i(width), _i(n_routed), _i(top), _i(n_groups), _i(keep_groups), _i(int(scoring == "sigmoid")),
-          _i(group_top), _i(int(renormalize)), _ptr(chosen), _ptr(weights), _ptr(shared_scale), _stream())
+          _i(group_top), _i(int(renormalize)), _i(int(biased)), _ptr(chosen), _ptr(weights), _ptr(shared_scale), _stream())
 
 
 def experts(h, gate_w, up_w, down_w, chosen, weights, n_tokens: int, n_experts: int, top: int, ff: int, act, x,
@@ -646,15 +649,27 @@ def head_gate(out: torch.Tensor, gate: Optional[torch.Tensor], n_rows: int, n_he
 
 
 def rmsnorm_add(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, n_rows: int,
-                partial: Optional[torch.Tensor] = None, splits: int = 0, split_stride: int = 0) -> None:
+                partial: Optional[torch.Tensor] = None, splits: int = 0, split_stride: int = 0, only_partial: bool = False,
+                copy: Optional[torch.Tensor] = None) -> None:
     """x[t] += y[t] / sqrt(mean(y[t]^2) + eps) * w; x and y float rows.  With `partial` [splits, rows, width], y is first
-    completed by those sums (a K-split product not yet added up)."""
-    _need_cuda(x, y, w, partial)
+    completed by those sums (a K-split product not yet added up), or is their sum (`only_partial`).  `copy`: the new rows
+    of x in the compute dtype as well."""
+    _need_cuda(x, y, w, partial, copy)
+    assert copy is None or (copy.is_contiguous() and copy.shape[1] == x.shape[1] and copy.shape[0] >= n_rows)
     width = x.shape[1]
     assert x.dtype == y.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous() and y.shape[1] == width
     assert w.numel() == width and w.is_contiguous()
     _call("core", "mdma_rmsnorm_add", _ptr(x), _ptr(y), _ptr(partial), _i(splits if partial is not None else 0),
-          ctypes.c_long(split_stride), _ptr(w), _i(dtype_code(w.dtype)), _i(n_rows), _i(width), _f(eps), _stream())
+          ctypes.c_long(split_stride), _i(int(only_partial)), _ptr(w), _i(dtype_code(w.dtype)), _i(n_rows), _i(width), _f(eps),
+          _ptr(copy), _i(dtype_code(copy.dtype) if copy is not None else F32), _stream())
+
+
+def copy_rows(x: torch.Tensor, out: torch.Tensor, n_rows: int) -> None:
+    """out[:n_rows] (bfloat16) = x[:n_rows] (float)."""
+    _need_cuda(x, out)
+    assert x.dtype == torch.float32 and out.dtype == torch.bfloat16 and x.is_contiguous() and out.is_contiguous()
+    assert x.shape[1] == out.shape[1]
+    _call("core", "mdma_copy_rows", _ptr(x), _ptr(out), ctypes.c_long(n_rows * x.shape[1]), _stream())
 
 
 def add_scaled(y: torch.Tensor, z: torch.Tensor, a: float, n_rows: int) -> None:
@@ -673,9 +688,11 @@ def linear_attention_fits(dim: int, vdim: int, chunked: bool = False) -> bool:
 
 def linear_attention(proj, q_col: int, k_col: int, v_col: int, decay, seq_start, seq_slot, state, out, n_seqs: int,
                      heads: int, dim: int, vdim: int, chunked: bool = False, run_rows: int = 0, max_runs: int = 1,
-                     scratch=None, single: bool = False) -> None:
-    """S = decay_h S + k v^T, o = S^T q per head over each sequence's rows, q, k, v = SiLU of the columns q_col.., k_col..,
-    v_col.. of `proj`; state [slots, heads * dim * vdim] floats is read and brought up to date; out [T, heads * vdim]
+                     scratch=None, single: bool = False, silu: bool = True, k_scale: float = 1.0, inv_freq=None,
+                     rotary_dim: int = 0, interleaved: bool = False, tok_pos=None) -> None:
+    """S = decay_h S + k v^T, o = S^T q per head over each sequence's rows, q, k, v = the columns q_col.., k_col..,
+    v_col.. of `proj`, through SiLU if `silu`, then the first `rotary_dim` numbers of every q and k head turned by the
+    token's position, then k times `k_scale`, all in float; state [slots, heads * dim * vdim] floats is read and brought up to date; out [T, heads * vdim]
     floats.  `chunked`: the walk a chunk of rows at a time, and with `run_rows` > 0 in runs of that many rows side by
     side (`max_runs`: the most runs of a sequence; `scratch`: n_seqs * max_runs * heads * dim * vdim floats); `single`:
     the kernel for steps in which no sequence brings more than one row.  Equal up to rounding."""
@@ -686,12 +703,15 @@ def linear_attention(proj, q_col: int, k_col: int, v_col: int, decay, seq_start,
     assert proj.shape[1] >= max(q_col + heads * dim, k_col + heads * dim, v_col + heads * vdim)
     assert run_rows == 0 or (chunked and scratch is not None and scratch.dtype == torch.float32 and scratch.is_contiguous())
     assert not (single and chunked)
+    _need_cuda(inv_freq, tok_pos)
+    assert rotary_dim == 0 or (inv_freq.dtype == torch.float32 and inv_freq.numel() >= rotary_dim // 2 and tok_pos is not None)
     sp, ss = _state(state)
     assert state.shape[1] >= heads * dim * vdim
     _call("core", "mdma_linear_attention", _ptr(proj), _i(dtype_code(proj.dtype)), _i(proj.stride(0)), _i(q_col), _i(k_col),
           _i(v_col), _ptr(decay), _ptr(seq_start), _ptr(seq_slot), sp, ss, _ptr(out), _i(n_seqs), _i(heads), _i(dim),
           _i(vdim), _i(2 if single else int(chunked)), _i(run_rows), _i(max_runs), _ptr(scratch),
-          ctypes.c_long(scratch.numel() if scratch is not None else 0), _stream(), launches=2 if run_rows > 0 else 1)
+          ctypes.c_long(scratch.numel() if scratch is not None else 0), _i(int(silu)), _i(rotary_dim), _i(int(interleaved)),
+          _ptr(inv_freq), _ptr(tok_pos), _f(k_scale), _stream(), launches=2 if run_rows > 0 else 1)
 
 
 def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_rows: int, eps: float,
@@ -825,3 +845,68 @@ def talking_attention(q, k_cache, v_cache, talk, sinks, ctx, page_table, max_pag
           _ptr(talk), _ptr(sinks), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(ctx.seq_slot), _ptr(page_table), _i(max_pages),
           _i(page_size), _ptr(out), _i(ctx.n_tokens), _i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim), _i(window), _f(scale),
           _stream())
+
+
+# ---- the gated delta rule with a decay per key channel (csrc/delta_rule.cu) ---------------------------------------------
+def delta_prepare(proj, raw, conv_w, taps: int, a_log, dt_bias, ctx, conv_state, q, k, v, lg, beta, heads: int,
+                  kv_heads: int, dim: int, vdim: int, unit_eps: float, q_scale: float) -> None:
+    """From float projection rows [q | k | v | b] and the decays' inputs `raw` [T, heads * dim] to what enters the
+    recurrence, float rows: q, k [T, kv_heads * dim] unit vectors (q times `q_scale`), v [T, heads * vdim], the decays'
+    logarithms lg [T, heads * dim], the step sizes beta [T, heads].  `conv_state` [slots, (taps - 1) * channels], the
+    convolutions' last inputs, is read and brought up to date."""
+    _need_cuda(proj, raw, conv_w, a_log, dt_bias, conv_state, q, k, v, lg, beta)
+    channels = 2 * kv_heads * dim + heads * vdim
+    assert proj.dtype == raw.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= channels + heads
+    assert raw.is_contiguous() and raw.shape[1] == heads * dim and conv_w.is_contiguous() and tuple(conv_w.shape) == (channels, taps)
+    assert a_log.numel() == heads and dt_bias.numel() == heads * dim
+    for t, c in ((q, kv_heads * dim), (k, kv_heads * dim), (v, heads * vdim), (lg, heads * dim), (beta, heads)):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape[1] == c and t.shape[0] >= ctx.n_tokens
+    sp, ss = _state(conv_state) if taps > 1 else (_ptr(None), ctypes.c_long(0))
+    assert taps == 1 or conv_state.shape[1] >= (taps - 1) * channels
+    _call("core", "mdma_delta_prepare", _ptr(proj), _i(proj.stride(0)), _ptr(raw), _ptr(conv_w), _i(dtype_code(conv_w.dtype)),
+          _i(taps), _ptr(a_log), _ptr(dt_bias), _i(_same_dtype(a_log, dt_bias)), _ptr(ctx.tok_seq), _ptr(ctx.seq_start),
+          _ptr(ctx.seq_slot), sp, ss, _ptr(q), _ptr(k), _ptr(v), _ptr(lg), _ptr(beta), _i(ctx.n_tokens), _i(ctx.n_seqs),
+          _i(heads), _i(kv_heads), _i(dim), _i(vdim), _f(unit_eps), _f(q_scale), _stream(), launches=2 if taps > 1 else 1)
+
+
+def delta_scan(q, k, v, lg, beta, ctx, state, out, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
+    """S = exp(lg) S; u = beta (v - S^T k); S += k u^T; o = S^T q per head over each sequence's rows, row by row in one
+    fixed order; state [slots, heads * dim * vdim] floats is read and brought up to date; out [T, heads * vdim] floats."""
+    _need_cuda(q, k, v, lg, beta, state, out)
+    for t, c in ((q, kv_heads * dim), (k, kv_heads * dim), (v, heads * vdim), (lg, heads * dim), (beta, heads), (out, heads * vdim)):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape[1] == c
+    sp, ss = _state(state)
+    assert state.shape[1] >= heads * dim * vdim
+    _call("core", "mdma_delta_scan", _ptr(q), _ptr(k), _ptr(v), _ptr(lg), _ptr(beta), _ptr(ctx.seq_start), _ptr(ctx.seq_slot),
+          sp, ss, _ptr(out), _i(ctx.n_seqs), _i(heads), _i(kv_heads), _i(dim), _i(vdim), _stream())
+
+
+def gated_head_rmsnorm(o: torch.Tensor, gate: torch.Tensor, w: Optional[torch.Tensor], out: torch.Tensor, n_rows: int,
+                       heads: int, vdim: int, eps: float, gate_act: str = "sigmoid") -> None:
+    """out = o_h / sqrt(mean(o_h^2) + eps) * w * act(gate) head by head; o float rows of heads * vdim, `w` [vdim] shared by
+    the heads (None: no weight), gate may be a view of wider rows; act "sigmoid" or "silu"."""
+    _need_cuda(o, gate, w, out)
+    width = heads * vdim
+    assert o.dtype == torch.float32 and o.is_contiguous() and out.is_contiguous() and o.shape[1] == out.shape[1] == width
+    assert gate.stride(1) == 1 and gate.shape[1] >= width and (w is None or (w.numel() == vdim and w.is_contiguous()))
+    assert gate_act in ("sigmoid", "silu")
+    _call("core", "mdma_gated_head_rmsnorm", _ptr(o), _ptr(gate), _i(dtype_code(gate.dtype)), _i(gate.stride(0)), _ptr(w),
+          _i(dtype_code(w.dtype) if w is not None else F32), _ptr(out), _i(dtype_code(out.dtype)), _i(n_rows), _i(heads),
+          _i(vdim), _f(eps), _i(int(gate_act == "silu")), _stream())
+
+
+# ---- attention whose heads' weights are mixed after the softmax (csrc/attention_mixed_weights.cu) ------------------------
+def mixed_weights_attention(q, k_cache, v_cache, mix, factor, softcap: float, ctx, page_table, max_pages: int, page_size: int,
+                            out, n_heads: int, n_kv_heads: int, dim: int, v_dim: int, window: int, keep_first: int) -> None:
+    """out[t, h] = sum_j w'_hj v_j with w'_h = sum_g mix[h, g] w_g and w_g the softmax over the visible keys of
+    factor[g] (q_g . k_j), through softcap tanh(. / softcap) if `softcap` > 0; a key is visible up to the token's position
+    if it lies within `window` (0: always) or is one of the first `keep_first`.  A block per token, keys in order."""
+    _need_cuda(q, k_cache, v_cache, mix, factor, page_table, out)
+    assert q.stride(1) == 1 and out.is_contiguous() and out.dtype == q.dtype == k_cache.dtype == v_cache.dtype
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and out.shape[1] == n_heads * v_dim and out.shape[0] >= ctx.n_tokens
+    assert mix.dtype == factor.dtype == torch.float32 and mix.is_contiguous() and mix.numel() == n_heads * n_heads
+    assert factor.is_contiguous() and factor.numel() == n_heads
+    _call("core", "mdma_mixed_weights", _ptr(q), _i(dtype_code(q.dtype)), _i(q.stride(0)), _ptr(k_cache), _ptr(v_cache),
+          _ptr(mix), _ptr(factor), _f(softcap), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(ctx.seq_slot), _ptr(page_table),
+          _i(max_pages), _i(page_size), _ptr(out), _i(ctx.n_tokens), _i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim),
+          _i(window), _i(keep_first), _stream())

@@ -4,13 +4,16 @@ feed_forward(norm(x)), the residual stream x kept in float
 in front of the mixer and a learned gate on each sublayer's result.  "parallel":
 one norm whose output both sublayers read, x += mixer(h) + feed_forward(h).
 "sandwich": a norm in front of each sublayer and one on its result,
-x += norm_b(mixer(norm_a(x))); x += norm_d(feed_forward(norm_c(x)))."""
+x += norm_b(mixer(norm_a(x))); x += norm_d(feed_forward(norm_c(x))).
+"postnorm": a norm on each sublayer's result only, x += norm_a(mixer(x));
+x += norm_b(feed_forward(x))."""
 from __future__ import annotations
 
 import dataclasses
 
 import torch
 
+from .. import ops
 from ..registry import AUXILIARIES, BLOCKS, FEED_FORWARDS, MIXERS, NORMS
 from ..spec import LayerSpec
 
@@ -211,3 +214,61 @@ class SandwichBlock:
         y[:n].zero_()
         self.ffn.forward(ctx, h, y)
         self.ffn_post.add_normed(ctx, y, x)
+
+
+@BLOCKS.register("postnorm")
+class PostNormBlock:
+    """The sublayers read the residual stream itself; a norm lies on each one's result only:
+
+        x += post1(mixer(x));   x += post2(feed_forward(x))       (if the layer has one)
+
+    The norms come from `LayerSpec.extras`: "mixer_post_norm" and "ffn_post_norm"; they must offer `add_normed`.  A
+    sublayer that offers `produce` stores its result (partial sums of a K-split product are left for the norm), any other
+    adds it into a zeroed buffer.  Where the engine computes in bfloat16, sublayers read a copy of the stream in that
+    dtype; the kernel that adds a normed result leaves the copy of the new rows behind, and the next layer of this
+    arrangement takes it over (`ctx.stream_copied`)."""
+    leaves_stream_copy = True
+
+    def __init__(self, spec: LayerSpec):
+        self.spec = spec
+        self.mixer = MIXERS.get(spec.mixer.kind)(spec.mixer)
+        self.mixer_post = NORMS.get(spec.extras["mixer_post_norm"].kind)(spec.extras["mixer_post_norm"])
+        self.width = int(spec.extras["mixer_post_norm"].params["width"])
+        self.ffn = self.ffn_post = None
+        if spec.mixer_norm is not None or spec.ffn_norm is not None:
+            raise ValueError("this arrangement has no norms in front of its sublayers")
+        if spec.ffn is not None:
+            self.ffn = FEED_FORWARDS.get(spec.ffn.kind)(spec.ffn)
+            self.ffn_post = NORMS.get(spec.extras["ffn_post_norm"].kind)(spec.extras["ffn_post_norm"])
+        for norm in (self.mixer_post, self.ffn_post):
+            if norm is not None and not hasattr(norm, "add_normed"):
+                raise ValueError(f"norm {norm.spec.kind!r} cannot follow a sublayer: it has no `add_normed`")
+
+    def parts(self):
+        return [p for p in (self.mixer, self.mixer_post, self.ffn, self.ffn_post) if p is not None]
+
+    def workspace(self):
+        return {"stream": (self.width, "act"), "sublayer": (self.width, "f32")}
+
+    def forward(self, ctx, x, view, owns_cache=True):
+        y = ctx.buf("sublayer", self.width, torch.float32)
+        copy = h = None
+        if ctx.rt.dtype == torch.float32:
+            h = x                                        # the stream itself is in the compute dtype
+        else:
+            copy = h = ctx.buf("stream", self.width)
+            if not getattr(ctx, "stream_copied", False):
+                ops.copy_rows(x, copy, ctx.n_tokens)
+        self._sublayer(ctx, self.mixer, self.mixer_post, h, x, y, copy, view, owns_cache)
+        if self.ffn is not None:
+            self._sublayer(ctx, self.ffn, self.ffn_post, h, x, y, copy)
+
+    @staticmethod
+    def _sublayer(ctx, part, norm, h, x, y, copy, *more):
+        if hasattr(part, "produce"):
+            part.produce(ctx, h, y, *more, defer=True)
+            norm.add_normed(ctx, y, x, stored=True, copy=copy)
+        else:
+            y[:ctx.n_tokens].zero_()
+            part.forward(ctx, h, y, *more)
+            norm.add_normed(ctx, y, x, copy=copy)

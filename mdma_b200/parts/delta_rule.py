@@ -1,0 +1,163 @@
+"""The gated delta rule with a decay per key channel (`channel_delta`).
+
+q, k = h Wq^T, h Wk^T [kv_heads x dim], v = h Wv^T [heads x v_dim]; head h uses q/k head h // (heads / kv_heads).  Each
+passes a short causal convolution over time per channel (`q.conv`, `k.conv`, `v.conv` [channels, taps], the last column
+is the current token's, zeros before the start) and SiLU; q and k become unit vectors per head, x / sqrt(sum(x^2) +
+unit_eps), and q is multiplied by dim^-1/2.  b = sigmoid(h Wb^T), one per head; g = exp(-exp(A_log_h) softplus(a2 a1 h +
+dt_bias)), one per head and key channel.  Per head, S [dim, v_dim]:
+
+    S <- diag(g) S;   u = b (v - S^T k);   S <- S + k u^T;   o = S^T q.
+
+Each head's o is divided by its root mean square, multiplied by the weight `norm` (shared by the heads) and by
+sigmoid(g2 g1 h), and the heads side by side go through Wo.
+
+State per sequence: S (floats) and the convolutions' last taps-1 inputs.  Everything that enters the recurrence is float
+in both engines (the projections write float rows); the inner rows of the two low-rank projections are in the compute
+dtype.  The 32-bit engine and short portions walk row by row in one fixed order.
+"""
+from __future__ import annotations
+
+import torch
+
+from .. import ops
+from ..cache import StateNeed
+from ..registry import MIXERS
+from ..spec import TensorSpec
+from .base import Part
+from .linear import Linear
+
+
+@MIXERS.register("channel_delta")
+class ChannelDelta(Part):
+    graph_safe = True
+    MAX_DIM, MAX_TAPS = 256, 16          # the kernels' limits
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = self.params
+        self.hidden = int(p["hidden_size"])
+        self.heads, self.kv_heads = int(p["num_heads"]), int(p.get("num_kv_heads") or p["num_heads"])
+        self.dim = int(p["head_dim"])
+        self.v_dim = int(p.get("v_dim") or self.dim)
+        self.taps = int(p["conv"])
+        self.decay_rank, self.gate_rank = int(p["decay_rank"]), int(p["gate_rank"])
+        self.eps, self.unit_eps = float(p["eps"]), float(p.get("unit_eps", 1e-6))
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} heads do not divide over {self.kv_heads} kv heads")
+        self.qk_width, self.k_width, self.v_width = self.kv_heads * self.dim, self.heads * self.dim, self.heads * self.v_dim
+        self.channels = 2 * self.qk_width + self.v_width            # what the convolutions see
+        self.row_width = self.channels + self.heads
+        self.row_pitch = -(-self.row_width // 8) * 8
+        # the two inner rows lie side by side when the second then starts on a 16-byte boundary
+        self.inner_fused = self.decay_rank % 8 == 0
+        self.inner_width = self.decay_rank + self.gate_rank
+        self.state_floats = self.heads * self.dim * self.v_dim
+        self.conv_at = -(-self.state_floats // 4) * 4
+        self.conv_floats = (self.taps - 1) * self.channels
+
+    def check_limits(self, rt):
+        if self.dim > self.MAX_DIM:
+            raise ValueError(f"delta-rule heads of {self.dim} are beyond the kernels' limit of {self.MAX_DIM}")
+        if not 1 <= self.taps <= self.MAX_TAPS:
+            raise ValueError(f"a convolution of {self.taps} taps is outside the kernel's 1..{self.MAX_TAPS}")
+
+    def tensor_specs(self):
+        W = self.hidden
+        return {"q": TensorSpec((self.qk_width, W)), "q.conv": TensorSpec((self.qk_width, self.taps)),
+                "k": TensorSpec((self.qk_width, W)), "k.conv": TensorSpec((self.qk_width, self.taps)),
+                "v": TensorSpec((self.v_width, W)), "v.conv": TensorSpec((self.v_width, self.taps)),
+                "b": TensorSpec((self.heads, W)), "A_log": TensorSpec((self.heads,), "vector", "normal"),
+                "norm": TensorSpec((self.v_dim,), "vector"),
+                "a1": TensorSpec((self.decay_rank, W)), "a2": TensorSpec((self.k_width, self.decay_rank)),
+                "dt_bias": TensorSpec((self.k_width,), "vector", "normal"),
+                "g1": TensorSpec((self.gate_rank, W)), "g2": TensorSpec((self.v_width, self.gate_rank)),
+                "o": TensorSpec((W, self.v_width))}
+
+    def fused_tensors(self):
+        fused = {"qkvb": ("q", "k", "v", "b"), "conv": ("q.conv", "k.conv", "v.conv")}
+        if self.inner_fused:
+            fused["a1g1"] = ("a1", "g1")
+        return fused
+
+    def kv_need(self):
+        return None
+
+    def state_need(self):
+        return StateNeed((self.conv_at + self.conv_floats,), torch.float32)
+
+    def _names(self):
+        tag = f"{self.heads}_{self.kv_heads}_{self.dim}_{self.v_dim}"
+        return {n: f"delta_{n}_{tag}" for n in ("proj", "q", "k", "v", "lg", "beta", "raw", "gate", "sum", "out")}
+
+    def workspace(self):
+        n = self._names()
+        ws = {n["proj"]: (self.row_pitch, "f32"), n["q"]: (self.qk_width, "f32"), n["k"]: (self.qk_width, "f32"),
+              n["v"]: (self.v_width, "f32"), n["lg"]: (self.k_width, "f32"), n["beta"]: (self.heads, "f32"),
+              n["raw"]: (self.k_width, "f32"), n["gate"]: (self.v_width, "act"), n["sum"]: (self.v_width, "f32"),
+              n["out"]: (self.v_width, "act")}
+        if self.inner_fused:
+            ws[f"delta_inner_{self.inner_width}"] = (-(-self.inner_width // 8) * 8, "act")
+        else:
+            ws[f"delta_a1_{self.decay_rank}"] = (-(-self.decay_rank // 8) * 8, "act")
+            ws[f"delta_g1_{self.gate_rank}"] = (-(-self.gate_rank // 8) * 8, "act")
+        return ws
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+
+        def whole(name, pieces):
+            t = tensors.get(name)
+            return t if t is not None else torch.cat([tensors[n] for n in pieces], dim=0).contiguous()
+        self.proj = Linear(whole("qkvb", ("q", "k", "v", "b")), rt)
+        self.conv = whole("conv", ("q.conv", "k.conv", "v.conv"))
+        if self.inner_fused:
+            self.inner = Linear(whole("a1g1", ("a1", "g1")), rt)
+        else:
+            self.a1, self.g1 = Linear(tensors["a1"], rt), Linear(tensors["g1"], rt)
+        self.a2, self.g2, self.o = Linear(tensors["a2"], rt), Linear(tensors["g2"], rt), Linear(tensors["o"], rt)
+        self.a_log, self.dt_bias, self.norm = tensors["A_log"], tensors["dt_bias"], tensors["norm"]
+
+    def _low_rank(self, ctx, h, raw, gate):
+        """raw = a2 a1 h (float rows), gate = g2 g1 h."""
+        n = ctx.n_tokens
+        if self.inner_fused:
+            inner = ctx.buf(f"delta_inner_{self.inner_width}", -(-self.inner_width // 8) * 8)
+            self.inner.store(h, inner[:, :self.inner_width], n)
+            a, g = inner[:, :self.decay_rank], inner[:, self.decay_rank:self.inner_width]
+        else:
+            a = ctx.buf(f"delta_a1_{self.decay_rank}", -(-self.decay_rank // 8) * 8)[:, :self.decay_rank]
+            g = ctx.buf(f"delta_g1_{self.gate_rank}", -(-self.gate_rank // 8) * 8)[:, :self.gate_rank]
+            self.a1.store(h, a, n)
+            self.g1.store(h, g, n)
+        self.a2.store(a, raw, n)
+        self.g2.store(g, gate, n)
+
+    def _run(self, ctx, h, view):
+        n = ctx.n_tokens
+        names = self._names()
+        f32 = torch.float32
+        proj = ctx.buf(names["proj"], self.row_pitch, f32)
+        raw, gate = ctx.buf(names["raw"], self.k_width, f32), ctx.buf(names["gate"], self.v_width)
+        q, k = ctx.buf(names["q"], self.qk_width, f32), ctx.buf(names["k"], self.qk_width, f32)
+        v, lg = ctx.buf(names["v"], self.v_width, f32), ctx.buf(names["lg"], self.k_width, f32)
+        beta, sums = ctx.buf(names["beta"], self.heads, f32), ctx.buf(names["sum"], self.v_width, f32)
+        out = ctx.buf(names["out"], self.v_width)
+        state = view.state[:, :self.state_floats]
+        conv_state = view.state[:, self.conv_at:self.conv_at + self.conv_floats] if self.taps > 1 else None
+        self.proj.store(h, proj[:, :self.row_width], n)
+        self._low_rank(ctx, h, raw, gate)
+        ops.delta_prepare(proj, raw, self.conv, self.taps, self.a_log, self.dt_bias, ctx, conv_state, q, k, v, lg, beta,
+                          self.heads, self.kv_heads, self.dim, self.v_dim, self.unit_eps, self.dim ** -0.5)
+        ops.delta_scan(q, k, v, lg, beta, ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
+        ops.gated_head_rmsnorm(sums, gate, self.norm, out, n, self.heads, self.v_dim, self.eps)
+        return out
+
+    def forward(self, ctx, h, x, view, owns_cache=True):
+        self.o.accumulate(self._run(ctx, h, view), x, ctx.n_tokens, defer=False)
+
+    def produce(self, ctx, h, out, view, owns_cache=True, defer=False):
+        self.o.store(self._run(ctx, h, view), out, ctx.n_tokens, defer=defer)
+
+    def resident_tensors(self):
+        ts = [self.proj.w, self.conv, self.a2.w, self.g2.w, self.o.w, self.a_log, self.dt_bias, self.norm]
+        return ts + ([self.inner.w] if self.inner_fused else [self.a1.w, self.g1.w])

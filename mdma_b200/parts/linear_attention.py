@@ -7,7 +7,9 @@ Linear attention.  q = silu(Wq h), k = silu(Wk h) [heads x dim], v = silu(Wv h) 
 
 S [dim, v_dim] starting at zero, kept in float per sequence (the site's state) and carried from step to step.
 The heads side by side are RMS-normed together with the weight `norm`, multiplied by sigmoid(Wg h), by the
-constant `out_scale`, and projected by Wo.  The decays are parameters (one per head).  The activations, the state, the
+constant `out_scale`, and projected by Wo.  Options: `activation` "none" leaves out the SiLU on q, k and v; `position`, a
+rotation by a frequency table, turns q and k (not v); `k_scale` multiplies k after it; `norm` "head" divides every head by
+its own root mean square, without a weight; `gate` "silu" multiplies by silu(Wg h).  The decays are parameters (one per head).  The activations, the rotation, the state, the
 sums over it, the norm and the gate are float in both engines; the projections are one product in the compute dtype.
 The 32-bit engine and short portions walk row by row in one fixed order; single tokens in the serving engine update
 the state row in place without staging it; the serving engine walks portions of
@@ -28,7 +30,7 @@ import torch
 
 from .. import ops
 from ..cache import StateNeed
-from ..registry import MIXERS
+from ..registry import MIXERS, POSITIONS
 from ..spec import PartSpec, TensorSpec
 from .base import Part
 from .linear import Linear
@@ -50,11 +52,24 @@ class LinearAttention(Part):
         self.decay = [float(d) for d in p["decay"]]
         self.eps = float(p["eps"])
         self.out_scale = float(p.get("out_scale", 1.0))
+        self.activation, self.gate = str(p.get("activation", "silu")), str(p.get("gate", "sigmoid"))
+        self.k_scale, self.norm_kind = float(p.get("k_scale", 1.0)), str(p.get("norm", "row"))
+        if self.activation not in ("silu", "none") or (self.norm_kind, self.gate) not in (("row", "sigmoid"), ("head", "sigmoid"), ("head", "silu")):
+            raise ValueError(f"linear attention with activation {self.activation!r}, norm {self.norm_kind!r} and gate {self.gate!r} is not implemented")
+        if self.norm_kind == "head" and self.out_scale != 1.0:
+            raise ValueError("a norm per head does not go with out_scale")
+        pos = p.get("position")
+        self.position = POSITIONS.get(pos.kind)(pos) if pos is not None else None
+        if self.position is not None and (not hasattr(self.position, "rotary_table") or getattr(self.position, "magnitude", 1.0) != 1.0):
+            raise ValueError("linear attention takes a rotation by a frequency table without a factor on cos and sin, or none")
         if len(self.decay) != self.heads:
             raise ValueError(f"{len(self.decay)} decays for {self.heads} heads")
         self.qk_width, self.v_width = self.heads * self.dim, self.heads * self.v_dim
         self.k_col, self.v_col, self.g_col = self.qk_width, 2 * self.qk_width, 2 * self.qk_width + self.v_width
         self.row_width = self.g_col + self.v_width
+
+    def children(self):
+        return [self.position] if self.position is not None else []
 
     def check_limits(self, rt):
         if self.v_dim > 256 or self.dim > 4096:
@@ -62,9 +77,12 @@ class LinearAttention(Part):
 
     def tensor_specs(self):
         W = self.hidden
-        return {"q": TensorSpec((self.qk_width, W)), "k": TensorSpec((self.qk_width, W)), "v": TensorSpec((self.v_width, W)),
-                "g": TensorSpec((self.v_width, W)), "norm": TensorSpec((self.v_width,), "vector"),
-                "o": TensorSpec((W, self.v_width))}
+        specs = {"q": TensorSpec((self.qk_width, W)), "k": TensorSpec((self.qk_width, W)), "v": TensorSpec((self.v_width, W)),
+                 "g": TensorSpec((self.v_width, W))}
+        if self.norm_kind == "row":
+            specs["norm"] = TensorSpec((self.v_width,), "vector")
+        specs["o"] = TensorSpec((W, self.v_width))
+        return specs
 
     def fused_tensors(self):
         return {"qkvg": ("q", "k", "v", "g")}
@@ -89,18 +107,20 @@ class LinearAttention(Part):
 
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
+        if self.position is not None:
+            self.position.bind({}, rt)
         fused = tensors.get("qkvg")
         if fused is None:
             fused = torch.cat([tensors[n] for n in ("q", "k", "v", "g")], dim=0).contiguous()
         self.proj = Linear(fused, rt)
-        self.norm = tensors["norm"]
+        self.norm = tensors.get("norm")
         self.o = Linear(tensors["o"], rt)
         self.decay_dev = rt.derived(torch.tensor(self.decay, dtype=torch.float64).to(torch.float32))
         if not ops.linear_attention_fits(self.dim, self.v_dim):
             raise ValueError(f"linear attention heads of {self.dim} x {self.v_dim} do not fit the kernels' shared memory")
         self.chunks_fit = ops.linear_attention_fits(self.dim, self.v_dim, chunked=True)
 
-    def forward(self, ctx, h, x, view, owns_cache=True):
+    def _run(self, ctx, h, view):
         n = ctx.n_tokens
         tag = f"{self.row_width}_{self.v_width}"
         proj = ctx.buf(f"lin_proj_{tag}", self.row_width)
@@ -117,14 +137,27 @@ class LinearAttention(Part):
             most = -(-ctx.max_new // self.RUN_ROWS)
             if ctx.n_seqs * most * self.heads * self.dim * self.v_dim <= runs.numel():
                 run_rows, max_runs, scratch = self.RUN_ROWS, most, runs
+        inv_freq, rotary_dim, interleaved = self.position.rotary_table() if self.position is not None else (None, 0, False)
         ops.linear_attention(proj, 0, self.k_col, self.v_col, self.decay_dev, ctx.seq_start, ctx.seq_slot, view.state, sums,
                              ctx.n_seqs, self.heads, self.dim, self.v_dim, chunked, run_rows, max_runs, scratch,
-                             single=ctx.max_new == 1 and proj.dtype != torch.float32)
-        ops.gated_rmsnorm(sums, proj[:, self.g_col:], self.norm, out, n, self.eps, self.out_scale)
-        self.o.accumulate(out, x, n, defer=False)
+                             single=ctx.max_new == 1 and proj.dtype != torch.float32, silu=self.activation == "silu",
+                             k_scale=self.k_scale, inv_freq=inv_freq, rotary_dim=rotary_dim, interleaved=interleaved,
+                             tok_pos=ctx.tok_pos)
+        if self.norm_kind == "head":
+            ops.gated_head_rmsnorm(sums, proj[:, self.g_col:], None, out, n, self.heads, self.v_dim, self.eps, self.gate)
+        else:
+            ops.gated_rmsnorm(sums, proj[:, self.g_col:], self.norm, out, n, self.eps, self.out_scale)
+        return out
+
+    def forward(self, ctx, h, x, view, owns_cache=True):
+        self.o.accumulate(self._run(ctx, h, view), x, ctx.n_tokens, defer=False)
+
+    def produce(self, ctx, h, out, view, owns_cache=True, defer=False):
+        """`defer`: the last product may leave K-split partial sums of `out` for the caller's next kernel."""
+        self.o.store(self._run(ctx, h, view), out, ctx.n_tokens, defer=defer)
 
     def resident_tensors(self):
-        return [self.proj.w, self.norm, self.o.w]
+        return [t for t in (self.proj.w, self.norm, self.o.w) if t is not None]
 
 
 @MIXERS.register("side_by_side")

@@ -41,7 +41,7 @@ class GatedMLP(Part):
         return specs
 
     def workspace(self):
-        return {"act": (self.inner, "act")}
+        return {"act": (-(-self.inner // 8) * 8, "act")}         # layers of several sizes share it: rows start on 16 bytes
 
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
@@ -53,6 +53,13 @@ class GatedMLP(Part):
         act = ctx.buf("act", self.inner)
         self.gate_up.gated(h, act, ctx.n_tokens)
         self.down.accumulate(act, x, ctx.n_tokens)
+
+    def produce(self, ctx, h, out, defer=False):
+        """The result as float rows; `defer`: the second product may leave K-split partial sums of `out` for the caller's
+        next kernel."""
+        act = ctx.buf("act", self.inner)
+        self.gate_up.gated(h, act, ctx.n_tokens)
+        self.down.store(act, out, ctx.n_tokens, defer=defer)
 
     def resident_tensors(self):
         return [t for t in (self.gate_up.w, self.gate_up.w2, self.down.w, self.gate_up.bias, self.gate_up.bias2,

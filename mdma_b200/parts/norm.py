@@ -58,21 +58,26 @@ class RMSNorm(Part):
             ops_tensor.flush_pending(x.device, self.rt.tc)
         ops.rmsnorm(x, self.weight, self.eps, out, rows, n)
 
-    def add_normed(self, ctx, y, x):
+    def add_normed(self, ctx, y, x, stored: bool = False, copy=None):
         """x += norm(y), both float rows: the norm on a sublayer's result.  Partial sums that a K-split product left
-        of y are added up on the way."""
-        partial, splits, stride = None, 0, 0
+        of y are added up on the way (`stored`: the product was to be stored into y, so y is their sum alone).  `copy`:
+        the new x in the compute dtype as well, in the same pass."""
+        partial, splits, stride, only = None, 0, 0, False
         if self.rt.gemm == "tensor":
             from .. import ops_tensor
-            pend = ops_tensor.take_pending(y, ops.GEMM_ACCUMULATE, ctx.n_tokens, self.rt.tc)
+            mode = ops.GEMM_STORE if stored else ops.GEMM_ACCUMULATE
+            pend = ops_tensor.take_pending(y, mode, ctx.n_tokens, self.rt.tc) if not (stored and self.groups > 1) else None
             if pend is not None:
                 partial, splits, stride = pend
+                only = stored
             else:
                 ops_tensor.flush_pending(y.device, self.rt.tc)
         if self.groups > 1:
+            if copy is not None:
+                raise ValueError("the norm in groups leaves no copy of the stream")
             ops.group_rmsnorm_add(x, y, self.weight, self.eps, self.groups, ctx.n_tokens, partial, splits, stride)
             return
-        ops.rmsnorm_add(x, y, self.weight, self.eps, ctx.n_tokens, partial, splits, stride)
+        ops.rmsnorm_add(x, y, self.weight, self.eps, ctx.n_tokens, partial, splits, stride, only, copy)
 
     def resident_tensors(self):
         return [self.weight]

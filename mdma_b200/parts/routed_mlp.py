@@ -1,6 +1,6 @@
 """A feed-forward of many small gated feed-forwards of which each token uses a few (`routed_mlp`).
 
-Router, in float:  z = R h over all routed outputs, s = softmax(z) (`scoring` "sigmoid": s = sigmoid(z), each
+Router, in float:  z = R h over all routed outputs (plus `router.b` with `logit_bias`), s = softmax(z) (`scoring` "sigmoid": s = sigmoid(z), each
 on its own), choice scores c = s + correction (`correction` off: c = s).
 The routed outputs form `groups` equal groups of neighbours; a group's score is the sum of its `group_top`
 largest c (1, the default: its largest), and only
@@ -13,7 +13,7 @@ the last `identity` ones have no matrices and return h itself.  The result is th
 shared expert of the same form (`shared_ff` > 0) runs for every token and is added, multiplied by
 sigmoid(g . h), one number per token (`shared_gate`).
 
-Tensors: `e<i>.gate|up|down`, `router` [experts + identity, width], `correction` [experts + identity],
+Tensors: `e<i>.gate|up|down`, `router` [experts + identity, width], `correction` or `router.b` [experts + identity],
 `shared.gate|up|down`, `shared.sg` [1, width].  The experts' matrices are laid out as three stacked
 matrices, so that a kernel finds expert e at a row offset.
 
@@ -53,6 +53,9 @@ class RoutedMLP(Part):
         self.shared_ff = int(p.get("shared_ff", 0) or 0)
         self.shared_gate = bool(p.get("shared_gate", True)) and self.shared_ff > 0
         self.correction = bool(p.get("correction", True))
+        self.logit_bias = bool(p.get("logit_bias", False))
+        if self.logit_bias and self.correction:
+            raise ValueError("a bias on the router's logits and a correction of its scores do not go together")
         self.scoring = str(p.get("scoring", "softmax"))
         self.group_top = int(p.get("group_top", 1) or 1)
         self.renormalize = bool(p.get("renormalize", True))
@@ -80,6 +83,8 @@ class RoutedMLP(Part):
         specs["router"] = TensorSpec((self.n_routed, W))
         if self.correction:
             specs["correction"] = TensorSpec((self.n_routed,), "vector", "zeros")
+        if self.logit_bias:
+            specs["router.b"] = TensorSpec((self.n_routed,), "vector", "normal")
         if self.shared_ff:
             specs["shared.gate"] = TensorSpec((self.shared_ff, W))
             specs["shared.up"] = TensorSpec((self.shared_ff, W))
@@ -123,7 +128,7 @@ class RoutedMLP(Part):
                 stacked[part] = t
             self.w_gate, self.w_up, self.w_down = stacked["gate"], stacked["up"], stacked["down"]
         self.router = tensors["router"]
-        self.correction_values = tensors.get("correction")
+        self.correction_values, self.bias_values = tensors.get("correction"), tensors.get("router.b")
         self.shared_up = self.shared_down = self.sg = None
         if self.shared_ff:
             self.shared_up = Linear(tensors["shared.gate"], rt, tensors["shared.up"], activation=self.activation,
@@ -138,7 +143,17 @@ class RoutedMLP(Part):
             from .. import ops_tensor
             self.by_products = (ops_tensor.gemm_supported(self.ff, self.hidden) and ops_tensor.gemm_supported(self.hidden, self.ff))
 
-    def forward(self, ctx, h, x):
+    def produce(self, ctx, h, out, defer=False):
+        """The result as float rows (an arrangement that norms it before it joins the stream): the shared expert's product
+        is stored, what the routed experts add comes on top."""
+        if self.shared_ff and self.sg is None:
+            self._shared(ctx, h, out, None, store=True)
+            self.forward(ctx, h, out, shared=False)
+            return
+        out[:ctx.n_tokens].zero_()
+        self.forward(ctx, h, out)
+
+    def forward(self, ctx, h, x, shared: bool = True):
         n = ctx.n_tokens
         if self.rt.gemm == "tensor":
             from .. import ops_tensor
@@ -149,11 +164,12 @@ class RoutedMLP(Part):
         act = ctx.buf(names[3], self.top * self.ff)
         scale = ctx.buf(names[6], 1, torch.float32)
         ops.route(h, self.router, self.correction_values, self.sg, n, self.top, self.groups, self.keep_groups, chosen,
-                  weight, scale if self.sg is not None else None, self.scoring, self.group_top, self.renormalize)
+                  weight, scale if self.sg is not None else None, self.scoring, self.group_top, self.renormalize, self.bias_values)
         if (self.by_products and n >= self.PRODUCTS_FROM and not getattr(ctx, "decode_only", False)
                 and not torch.cuda.is_current_stream_capturing()):
             self._experts_by_products(ctx, h, x, chosen, weight, act, names)
-            self._shared(ctx, h, x, scale)
+            if shared:
+                self._shared(ctx, h, x, scale)
             return
         # the 32-bit engine keeps ONE order of additions whatever the step's size: always expert by expert
         scratch = None
@@ -162,7 +178,8 @@ class RoutedMLP(Part):
             scratch = (self.first, order, ctx.buf(names[4], self.top * self.hidden, torch.float32))
         ops.experts(h, self.w_gate, self.w_up, self.w_down, chosen, weight, n, self.n_experts, self.top, self.ff,
                     act.view(-1, self.ff), x, scratch, self.pair_act, self.act_limit, self.act_alpha)
-        self._shared(ctx, h, x, scale)
+        if shared:
+            self._shared(ctx, h, x, scale)
 
     def _experts_by_products(self, ctx, h, x, chosen, weight, act, names):
         n = ctx.n_tokens
@@ -179,17 +196,17 @@ class RoutedMLP(Part):
         ops_tensor.gemm_runs(act, self.w_down, y, first, self.hidden, ops.GEMM_STORE, st=self.rt.tc)
         ops.experts_combine(y, h, chosen, weight, where, n, self.n_experts, self.top, x)
 
-    def _shared(self, ctx, h, x, scale):
+    def _shared(self, ctx, h, x, scale, store: bool = False):
         n = ctx.n_tokens
         if self.shared_ff:
             sact = ctx.buf(self._names()[5], self.shared_ff)
             self.shared_up.gated(h, sact, n)
             if self.sg is not None:
                 ops.scale_rows(sact, scale.view(-1), n)      # the down product is linear: scaling its input scales its result
-            self.shared_down.accumulate(sact, x, n, defer=False)
+            (self.shared_down.store if store else self.shared_down.accumulate)(sact, x, n, defer=False)
 
     def resident_tensors(self):
-        ts = [self.w_gate, self.w_up, self.w_down, self.router, self.correction_values, self.sg]
+        ts = [self.w_gate, self.w_up, self.w_down, self.router, self.correction_values, self.bias_values, self.sg]
         if self.shared_ff:
             ts += [self.shared_up.w, self.shared_up.w2, self.shared_down.w]
         return [t for t in ts if t is not None]

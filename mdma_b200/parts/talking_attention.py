@@ -1,4 +1,4 @@
-"""Grouped-query causal attention whose heads' scores are mixed before the softmax.
+"""Grouped-query causal attention whose heads' scores are mixed before the softmax, or their weights after it.
 
 q, k, v = h Wq^T (+ bq), h Wk^T (+ bk), h Wv^T (+ bv) with `bias`; with `qk_norm` every query and key head is divided
 by its root mean square, x / sqrt(mean(x^2) + eps), and multiplied by a weight of `head_dim` numbers that all heads
@@ -8,6 +8,11 @@ its own sequence, kv head = q head // (heads / kv heads).  With `talk`, the raw 
 query heads are mixed by a learned matrix T [heads, heads], s'_h = sum_g T[h, g] s_g, and head h takes the softmax of
 s'_h.  `denominator_extra` c > 0 adds c to every softmax denominator (a key with score ln c and no value; 1 is a sink
 whose score is 0).  The heads' results, concatenated, times Wo^T are added to the residual stream.
+
+With `talk` "weights" the scores stay each head's own and the heads' softmax weights are mixed instead, w'_h = sum_g
+T[h, g] w_g, before they meet the values of head h's own kv head.  Then also: `temp`, a learned number per head (tensor
+`temp`) that the scores are multiplied by; `softcap` c > 0, score <- c tanh(score / c) after that; `window` n > 0, a query
+at position i sees key j if i - j < n, and with `keep_first` m also if j < m (kept tokens keep their true positions).
 
 Scores, mixing and softmax are float in both engines.  Where the serving engine's tensor-core kernel takes the sizes,
 the mixing is moved onto the queries: heads of one group share their key head, so s'_h = sum_c x_h,c . k_c with
@@ -44,9 +49,16 @@ class TalkingAttention(Part):
         self.scale, self.eps = float(p["scale"]), float(p.get("eps", 0.0))
         self.window = int(p.get("window", 0) or 0)
         self.bias, self.qk_norm, self.talk = bool(p.get("bias", False)), bool(p.get("qk_norm", False)), bool(p.get("talk", False))
+        self.mixes_weights = p.get("talk") == "weights"
+        self.temp, self.softcap = bool(p.get("temp", False)), float(p.get("softcap", 0.0) or 0.0)
+        self.keep_first = int(p.get("keep_first", 0) or 0) if self.window else 0
+        if not self.mixes_weights and (self.temp or self.softcap or self.keep_first):
+            raise ValueError("temp, softcap and keep_first go with mixed weights only")
         self.extra = float(p.get("denominator_extra", 0.0) or 0.0)
         if self.extra < 0:
             raise ValueError("denominator_extra must not be negative")
+        if self.extra and self.mixes_weights:
+            raise ValueError("denominator_extra does not go with mixed weights")
         if self.n_heads % self.n_kv_heads:
             raise ValueError(f"{self.n_heads} heads do not divide over {self.n_kv_heads} kv heads")
         pos = p.get("position")
@@ -61,7 +73,7 @@ class TalkingAttention(Part):
         # the tensor-core kernel works on queries mixed per kv group, side by side: kv_heads * dim numbers a head
         from ..ops_tensor import talking_attention_mma_warps
         self.mixed_width = self.n_heads * self.n_kv_heads * self.head_dim
-        self._mma_shape = self.talk and talking_attention_mma_warps(self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim) > 0
+        self._mma_shape = self.talk and not self.mixes_weights and talking_attention_mma_warps(self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim) > 0
 
     def children(self):
         return [self.position] if self.position is not None else []
@@ -83,6 +95,8 @@ class TalkingAttention(Part):
             specs["k.norm"] = TensorSpec((self.head_dim,), "vector")
         if self.talk:
             specs["talk"] = TensorSpec((self.n_heads, self.n_heads), "vector", "normal")
+        if self.temp:
+            specs["temp"] = TensorSpec((self.n_heads,), "vector")
         specs["o"] = TensorSpec((self.hidden, self.out_width))
         return specs
 
@@ -96,13 +110,16 @@ class TalkingAttention(Part):
         out = {}
         if self.talk:
             out["talk_f32"] = ((self.n_heads, self.n_heads), torch.float32)
+        if self.mixes_weights:
+            out["factor"] = ((self.n_heads,), torch.float32)
         if self.extra > 0:
             out["sinks"] = ((self.n_heads,), torch.float32)
             out["sinks_log2"] = ((self.n_heads,), torch.float32)
         return out
 
     def kv_need(self):
-        return KVNeed(self.n_kv_heads, self.head_dim, self.window, v_dim=0 if self.v_dim == self.head_dim else self.v_dim)
+        return KVNeed(self.n_kv_heads, self.head_dim, self.window, v_dim=0 if self.v_dim == self.head_dim else self.v_dim,
+                      keep_first=self.keep_first)
 
     def state_need(self):
         return None
@@ -134,6 +151,13 @@ class TalkingAttention(Part):
         if self.talk:
             self.talk_f32 = take((self.n_heads, self.n_heads), torch.float32)      # the mixing is done in float
             self.talk_f32.copy_(self.talk_values.float())
+        self.factor = self.temp_values = None
+        if self.mixes_weights:
+            self.factor = take((self.n_heads,), torch.float32)         # what a head's raw scores are multiplied by
+            self.temp_values = tensors.get("temp")
+            self.factor.fill_(self.scale)
+            if self.temp:
+                self.factor.mul_(self.temp_values.float())
         if self.extra > 0:
             self.sinks = take((self.n_heads,), torch.float32)
             self.sinks.fill_(math.log(self.extra))
@@ -141,7 +165,7 @@ class TalkingAttention(Part):
             self.sinks_log2.fill_(math.log2(self.extra))
         self._tiled_ok = ops.talking_attention_tiled_fits(self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim)
 
-    def forward(self, ctx, h, x, view, owns_cache=True):
+    def _run(self, ctx, h, view, owns_cache):
         n = ctx.n_tokens
         row = ctx.buf(f"tqkv_{self.row_pitch}", self.row_pitch)
         out = ctx.buf(f"tattn_{self.out_width}", self.out_width)
@@ -155,6 +179,11 @@ class TalkingAttention(Part):
                            self.q_weight, self.k_weight, self.qk_norm, self.eps, view.k, view.v, view.page_table,
                            view.max_pages, view.page_size, n, self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim,
                            rotary_dim, interleaved, owns_cache)
+        if self.mixes_weights:
+            ops.mixed_weights_attention(row, view.k, view.v, self.talk_f32, self.factor, self.softcap, ctx, view.page_table,
+                                        view.max_pages, view.page_size, out, self.n_heads, self.n_kv_heads, self.head_dim,
+                                        self.v_dim, self.window, self.keep_first)
+            return out
         if self._mma_shape and self.rt.attention == "fast" and row.dtype == torch.bfloat16:
             from .. import ops_tensor
             mixed = ctx.buf(f"tmixed_{self.mixed_width}", self.mixed_width)
@@ -174,15 +203,22 @@ class TalkingAttention(Part):
             ops_tensor.talking_attention_mma(ctx, row, self.talk_f32, mixed, view, self.sinks_log2, out, self.n_heads,
                                              self.n_kv_heads, self.head_dim, self.v_dim, self.window, self.scale, st=self.rt.tc,
                                              splits=splits, partial=partial)
-            self.o.accumulate(out, x, n)
-            return
+            return out
         # the 32-bit engine visits keys in position order, a block per token; the serving engine stages tiles
         tiled = self._tiled_ok and row.dtype != torch.float32
         ops.talking_attention(row, view.k, view.v, self.talk_f32, self.sinks, ctx, view.page_table, view.max_pages,
                               view.page_size, out, self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, self.window,
                               self.scale, tiled=tiled)
-        self.o.accumulate(out, x, n)
+        return out
+
+    def forward(self, ctx, h, x, view, owns_cache=True):
+        self.o.accumulate(self._run(ctx, h, view, owns_cache), x, ctx.n_tokens)
+
+    def produce(self, ctx, h, out, view, owns_cache=True, defer=False):
+        """The result as float rows; `defer`: the last product may leave K-split partial sums of `out`."""
+        self.o.store(self._run(ctx, h, view, owns_cache), out, ctx.n_tokens, defer=defer)
 
     def resident_tensors(self):
-        return [t for t in (self.qkv.w, self.qkv.bias, self.o.w, self.q_weight, self.k_weight, self.talk_values)
+        return [t for t in (self.qkv.w, self.qkv.bias, self.o.w, self.q_weight, self.k_weight, self.talk_values,
+                            self.temp_values)
                 if t is not None]

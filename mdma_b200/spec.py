@@ -45,7 +45,7 @@ class LayerSpec:
     more parts than these four (a norm on the queries and keys, norms after the mixer and the
     feed-forward, a second feed-forward) finds them by name in `extras`."""
     block: str
-    mixer_norm: PartSpec
+    mixer_norm: Optional[PartSpec]        # None: the arrangement has no norm in front of its mixer
     mixer: PartSpec
     ffn_norm: Optional[PartSpec]          # None with `ffn`: a layer without a feed-forward
     ffn: Optional[PartSpec]

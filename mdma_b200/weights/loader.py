@@ -178,3 +178,11 @@ def load_tensors(model_dir: str, expected: dict[str, TensorSpec], compute: torch
 def stored_dtypes(model_dir: str) -> dict:
     """name -> dtype as stored, from the headers alone."""
     return {n: e.dtype for sf in open_model_files(model_dir) for n, e in sf.entries.items()}
+
+
+def stored_shapes(model_dir: str) -> dict:
+    """name -> shape, from the headers alone; empty for a folder without weights."""
+    try:
+        return {n: tuple(e.shape) for sf in open_model_files(model_dir) for n, e in sf.entries.items()}
+    except CheckpointError:
+        return {}
