@@ -21,6 +21,9 @@ constexpr int kDeltaMaxDim = 256, kDeltaMaxTaps = 16;
 __device__ __forceinline__ float delta_silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float delta_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float delta_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// exp(x), x <= 0, rounded once where it lies near one: a slow channel's decays are multiplied over thousands of tokens,
+// and an error of a unit in the last place to one side would add up over them
+__device__ __forceinline__ float delta_decay(float x) { return x > -0.5f ? 1.0f + expm1f(x) : expf(x); }
 __device__ __forceinline__ float delta_weight(const void* w, int dtype, size_t e) {
     return dtype == kF32 ? reinterpret_cast<const float*>(w)[e] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(w)[e]);
 }
@@ -137,7 +140,7 @@ delta_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
         for (int d = threadIdx.x; d < dim; d += blockDim.x) {
             sq[d] = q[((size_t)t * kv_heads + hk) * dim + d];
             sk[d] = k[((size_t)t * kv_heads + hk) * dim + d];
-            sg[d] = expf(lg[((size_t)t * heads + h) * dim + d]);
+            sg[d] = delta_decay(lg[((size_t)t * heads + h) * dim + d]);
         }
         const float b = beta[(size_t)t * heads + h];
         const float vc = mine ? v[((size_t)t * heads + h) * vdim + c] : 0.f;
