@@ -461,3 +461,58 @@ def talking_attention_splits(most_seqs: int, n_heads: int, n_kv_heads: int, dim:
     blocks = max(1, most_seqs) * -(-n_heads // warps)
     return max(1, min(8, sms // blocks))
 
+
+
+# ---- attention with mixed weights on the tensor cores (csrc/attention_mixed_weights_mma.cu) -------------------------------
+def mixed_weights_supported(n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
+    """Whether the tensor-core kernels take this geometry (the same arithmetic as the library's; kept here so that a
+    memory plan needs no compiled library)."""
+    return (0 < n_heads <= 32 and n_kv_heads > 0 and n_heads % n_kv_heads == 0 and dim % 16 == 0 and 0 < dim <= 256
+            and v_dim > 0 and v_dim % 8 == 0 and n_kv_heads * v_dim % 16 == 0)
+
+
+def mixed_weights_step_fits(n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
+    lib = _build._loaded.get("tensor") or _build.load("tensor")
+    return bool(lib.mdma_mixed_weights_step_fits(_i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim)))
+
+
+def mixed_weights_splits(most_seqs: int, max_len: int, window: int, keep_first: int, sms: int) -> int:
+    """Into how many runs the keys of a single-token step are divided: from the engine's capacity and the context rounded
+    up to 1,024 (as the replayed decode graphs see it); a run has two chunks of 32 keys at least where there are as many."""
+    keys = -(-max(max_len, 1) // 1024) * 1024
+    if window:
+        keys = min(keys, window + keep_first)
+    return max(1, min(sms // max(1, most_seqs), -(-keys // 64), 32))
+
+
+def mixed_weights_attention(ctx, q: torch.Tensor, view, mix: torch.Tensor, factor: torch.Tensor, softcap: float,
+                            out: torch.Tensor, scratch: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, v_dim: int,
+                            window: int, keep_first: int, st: Optional[TensorState] = None, step: Optional[int] = None) -> None:
+    """`ops.mixed_weights_attention` in bfloat16 on the tensor cores.  `scratch`: floats; a step runs in slabs of as many
+    tokens as heads * kv_heads * v_dim floats a token fit in it.  `step`: the kernel for steps of one token a sequence,
+    keys divided into that many runs (sequences * runs * heads * (kv_heads * v_dim + 2) floats of scratch)."""
+    _need_cuda(q, view.k, view.v, mix, factor, out, scratch, view.page_table)
+    if q.dtype != torch.bfloat16 or view.k.dtype != torch.bfloat16:
+        raise KernelError("the tensor-core attention takes bfloat16")
+    total = n_kv_heads * v_dim
+    assert q.stride(1) == 1 and out.is_contiguous() and out.shape[1] == n_heads * v_dim and out.shape[0] >= ctx.n_tokens
+    assert view.k.is_contiguous() and view.v.is_contiguous() and view.k.shape[-1] == dim and view.v.shape[-1] == v_dim
+    assert mix.dtype == factor.dtype == scratch.dtype == torch.float32 and mix.is_contiguous() and mix.numel() == n_heads * n_heads
+    assert factor.is_contiguous() and factor.numel() == n_heads and scratch.is_contiguous()
+    flush_pending(q.device, st or _device_state(q.device))
+    if step is not None:
+        need = ctx.n_seqs * step * n_heads * (total + 2)
+        if ctx.max_new != 1 or scratch.numel() < need:
+            raise KernelError(f"single tokens over {step} runs of keys need {need} floats of scratch, {scratch.numel()} given")
+        _call("tensor", "mdma_mixed_weights_step", _ptr(q), _i(q.stride(0)), _ptr(view.k), _ptr(view.v), _ptr(mix), _ptr(factor),
+              _f(softcap), _ptr(ctx.tok_pos), _ptr(ctx.seq_slot), _ptr(view.page_table), _i(view.max_pages), _i(view.page_size),
+              _ptr(out), _ptr(scratch), _i(step), _i(ctx.n_seqs), _i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim), _i(window),
+              _i(keep_first), _stream(), launches=2)
+        return
+    slab = min(scratch.numel() // (n_heads * total), ctx.n_tokens)
+    if slab < 1:
+        raise KernelError(f"attention with mixed weights needs {n_heads * total} floats of scratch a token, {scratch.numel()} given")
+    _call("tensor", "mdma_mixed_weights_rows", _ptr(q), _i(q.stride(0)), _ptr(view.k), _ptr(view.v), _ptr(mix), _ptr(factor),
+          _f(softcap), _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(ctx.seq_slot), _ptr(view.page_table), _i(view.max_pages),
+          _i(view.page_size), _ptr(out), _ptr(scratch), _i(slab), _i(ctx.n_tokens), _i(ctx.n_seqs), _i(ctx.max_new), _i(n_heads),
+          _i(n_kv_heads), _i(dim), _i(v_dim), _i(window), _i(keep_first), _stream(), launches=2 * -(-ctx.n_tokens // slab))

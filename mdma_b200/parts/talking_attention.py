@@ -18,6 +18,8 @@ Scores, mixing and softmax are float in both engines.  Where the serving engine'
 the mixing is moved onto the queries: heads of one group share their key head, so s'_h = sum_c x_h,c . k_c with
 x_h,c = scale * sum_{g in group c} T[h, g] q_g, one dot product of kv_heads * dim numbers against the token's key heads
 side by side as the cache row holds them (x is formed in float and rounded once to bfloat16, the product sums in float).
+With mixed weights the tensor-core kernels let every head attend over all value heads of a token side by side and mix the
+finished float rows: o_h = sum_g T[h, g] sum_j w_g(j) v_c(h)(j).
 """
 from __future__ import annotations
 
@@ -75,6 +77,10 @@ class TalkingAttention(Part):
         self.mixed_width = self.n_heads * self.n_kv_heads * self.head_dim
         self._mma_shape = self.talk and not self.mixes_weights and talking_attention_mma_warps(self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim) > 0
 
+        from ..ops_tensor import mixed_weights_supported
+        self._mixes_on_tensor = self.mixes_weights and mixed_weights_supported(self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim)
+        self.wide_width = self.n_heads * self.n_kv_heads * self.v_dim      # a token's heads, each over all value heads
+
     def children(self):
         return [self.position] if self.position is not None else []
 
@@ -128,6 +134,9 @@ class TalkingAttention(Part):
         out = {f"tqkv_{self.row_pitch}": (self.row_pitch, "act"), f"tattn_{self.out_width}": (self.out_width, "act")}
         if self._mma_shape:
             out[f"tmixed_{self.mixed_width}"] = (self.mixed_width, "act")
+        if self._mixes_on_tensor:
+            # long steps run in slabs of tokens: an eighth of a step's at a time where a token takes many floats
+            out[f"twide_{self.wide_width}"] = (max(-(-self.wide_width // 8), min(self.wide_width, 4096)), "f32")
         return out
 
     def bind(self, tensors, rt):
@@ -163,6 +172,10 @@ class TalkingAttention(Part):
             self.sinks.fill_(math.log(self.extra))
             self.sinks_log2 = take((self.n_heads,), torch.float32)      # the tensor-core kernel works in powers of two
             self.sinks_log2.fill_(math.log2(self.extra))
+        self._step_ok = False
+        if self._mixes_on_tensor and self.rt.attention == "fast":
+            from .. import ops_tensor
+            self._step_ok = ops_tensor.mixed_weights_step_fits(self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim)
         self._tiled_ok = ops.talking_attention_tiled_fits(self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim)
 
     def _run(self, ctx, h, view, owns_cache):
@@ -180,6 +193,21 @@ class TalkingAttention(Part):
                            view.max_pages, view.page_size, n, self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim,
                            rotary_dim, interleaved, owns_cache)
         if self.mixes_weights:
+            if self._mixes_on_tensor and self.rt.attention == "fast" and row.dtype == torch.bfloat16:
+                from .. import ops_tensor
+                scratch = ctx.buf(f"twide_{self.wide_width}", max(-(-self.wide_width // 8), min(self.wide_width, 4096)), torch.float32).view(-1)
+                step = None
+                if ctx.max_new == 1 and self._step_ok:
+                    most = int(getattr(ctx, "most_seqs", None) or ctx.n_seqs)
+                    sms = self.rt.tc.sms if self.rt.tc is not None else 148
+                    a_run = most * self.n_heads * (self.n_kv_heads * self.v_dim + 2)          # floats of one run of keys
+                    step = min(ops_tensor.mixed_weights_splits(most, ctx.max_len, self.window, self.keep_first, sms),
+                               scratch.numel() // a_run) or None
+                if step is not None or scratch.numel() >= self.wide_width:
+                    ops_tensor.mixed_weights_attention(ctx, row, view, self.talk_f32, self.factor, self.softcap, out, scratch,
+                                                       self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, self.window,
+                                                       self.keep_first, st=self.rt.tc, step=step)
+                    return out
             ops.mixed_weights_attention(row, view.k, view.v, self.talk_f32, self.factor, self.softcap, ctx, view.page_table,
                                         view.max_pages, view.page_size, out, self.n_heads, self.n_kv_heads, self.head_dim,
                                         self.v_dim, self.window, self.keep_first)
