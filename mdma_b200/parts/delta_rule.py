@@ -13,7 +13,8 @@ sigmoid(g2 g1 h), and the heads side by side go through Wo.
 
 State per sequence: S (floats) and the convolutions' last taps-1 inputs.  Everything that enters the recurrence is float
 in both engines (the projections write float rows); the inner rows of the two low-rank projections are in the compute
-dtype.  The 32-bit engine and short portions walk row by row in one fixed order.
+dtype.  The 32-bit engine and short portions walk row by row in one fixed order; the serving engine walks portions of
+`CHUNKS_FROM` rows or more a chunk of rows at a time (csrc/delta_chunk.cu).
 """
 from __future__ import annotations
 
@@ -31,6 +32,7 @@ from .linear import Linear
 class ChannelDelta(Part):
     graph_safe = True
     MAX_DIM, MAX_TAPS = 256, 16          # the kernels' limits
+    CHUNKS_FROM = 16                     # rows of a sequence in a step from which the serving engine walks chunk by chunk
 
     def __init__(self, spec):
         super().__init__(spec)
@@ -53,6 +55,7 @@ class ChannelDelta(Part):
         self.inner_width = self.decay_rank + self.gate_rank
         self.state_floats = self.heads * self.dim * self.v_dim
         self.conv_at = -(-self.state_floats // 4) * 4
+        self.chunks_fit = self.dim % 4 == 0 and self.v_dim % 4 == 0
         self.conv_floats = (self.taps - 1) * self.channels
 
     def check_limits(self, rt):
@@ -87,7 +90,7 @@ class ChannelDelta(Part):
 
     def _names(self):
         tag = f"{self.heads}_{self.kv_heads}_{self.dim}_{self.v_dim}"
-        return {n: f"delta_{n}_{tag}" for n in ("proj", "q", "k", "v", "lg", "beta", "raw", "gate", "sum", "out")}
+        return {n: f"delta_{n}_{tag}" for n in ("proj", "q", "k", "v", "lg", "beta", "raw", "gate", "sum", "out", "qg", "kd", "bm")}
 
     def workspace(self):
         n = self._names()
@@ -95,6 +98,8 @@ class ChannelDelta(Part):
               n["v"]: (self.v_width, "f32"), n["lg"]: (self.k_width, "f32"), n["beta"]: (self.heads, "f32"),
               n["raw"]: (self.k_width, "f32"), n["gate"]: (self.v_width, "act"), n["sum"]: (self.v_width, "f32"),
               n["out"]: (self.v_width, "act")}
+        if self.chunks_fit:
+            ws.update({n["qg"]: (self.k_width, "f32"), n["kd"]: (self.k_width, "f32"), n["bm"]: (16 * self.heads, "f32")})
         if self.inner_fused:
             ws[f"delta_inner_{self.inner_width}"] = (-(-self.inner_width // 8) * 8, "act")
         else:
@@ -148,7 +153,12 @@ class ChannelDelta(Part):
         self._low_rank(ctx, h, raw, gate)
         ops.delta_prepare(proj, raw, self.conv, self.taps, self.a_log, self.dt_bias, ctx, conv_state, q, k, v, lg, beta,
                           self.heads, self.kv_heads, self.dim, self.v_dim, self.unit_eps, self.dim ** -0.5)
-        ops.delta_scan(q, k, v, lg, beta, ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
+        if self.chunks_fit and self.rt.dtype != f32 and ctx.max_new >= self.CHUNKS_FROM:
+            # (the decays' inputs are spent: their rows take the solved right sides)
+            ops.delta_chunks(q, k, v, lg, beta, raw, ctx.buf(names["qg"], self.k_width, f32), ctx.buf(names["kd"], self.k_width, f32),
+                             ctx.buf(names["bm"], 16 * self.heads, f32), ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
+        else:
+            ops.delta_scan(q, k, v, lg, beta, ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
         ops.gated_head_rmsnorm(sums, gate, self.norm, out, n, self.heads, self.v_dim, self.eps)
         return out
 
