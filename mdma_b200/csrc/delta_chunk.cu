@@ -6,7 +6,8 @@
 //     S   <- diag(e^(L_n)) S + sum_j (e^(L_n - L_j) k_j) u_j^T.
 // No exponent is ever above zero.
 //
-// delta_chunk_prepare, block = (chunk, head), all chunks side by side: everything that does not depend on S.  The
+// delta_chunk_prepare, block = (chunk, head), all chunks side by side: everything that does not depend on S, left in
+// scratch as one run of floats per (chunk, head), laid out as the walk's shared memory (`DcLayout`).  The
 // triangular system is solved for its two right sides, w_i = b_i (e^(L_i) k_i - sum A_ij w_j) and z_i = b_i (v_i - sum
 // A_ij z_j), so that u = z - S^T w; also e^(L_i) q_i, e^(L_n - L_j) k_j, B and e^(L_n).
 // delta_chunk_walk, block = (sequence, head, sixteen columns of S), 4 warps, chunks in order: S^T lies in the accumulators
@@ -19,74 +20,115 @@
 namespace mdma {
 
 constexpr int kDc = 16;                   // rows of a chunk
-constexpr int kDcMaxDim = 256;
+constexpr int kDcMaxDim = 256, kDcCols = 16;
 constexpr float kDcLog2e = 1.4426950408889634f;
+
+// One (chunk, head) in scratch: w, qg [16][dimP + 8], kd [16][dimP + 4], B [16][24], the whole decay [dimP], then z for every
+// sixteen columns [16][20].  dimP: the channels rounded up to a multiple of 32, zero beyond dim; rows beyond the chunk's zero.
+struct DcLayout {
+    int dimP, wp, kp, qg, kd, b, g, z, slices, floats;
+    __host__ __device__ DcLayout(int dim, int vdim) {
+        dimP = (dim + 31) / 32 * 32;
+        if (dimP > 128) dimP = 256;                       // the sizes the walk is compiled for
+        wp = dimP + 8; kp = dimP + 4;
+        qg = kDc * wp; kd = 2 * kDc * wp; b = kd + kDc * kp; g = b + kDc * 24; z = g + dimP;
+        slices = (vdim + kDcCols - 1) / kDcCols;
+        floats = z + slices * kDc * 20;
+    }
+};
+// chunk c of sequence s: chunks of different sequences never share a place
+__device__ __forceinline__ size_t dc_place(int seq_start, int s, int chunk) { return (size_t)(seq_start / kDc) + s + chunk; }
+
+__device__ __forceinline__ float dc_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float4 dc_ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void dc_st4(float* p, float a, float b, float c, float d) { *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d); }
 
 // ---------------------------------------------------------------- what does not depend on S
 constexpr int kDcTiles = 36, kDcSlices = 7;          // 2 x 2 tiles on and below the diagonal; parts of the channels
-static size_t dc_prepare_smem(int dim) {
-    return sizeof(float) * ((size_t)3 * kDc * (dim + 1) + 2 * kDc * (kDc + 4) + (size_t)kDcSlices * kDcTiles * 8 + kDc);
+static size_t dc_prepare_smem(int dim, int vdim) {
+    return sizeof(float) * ((size_t)3 * kDc * (dim + 4) + (size_t)kDc * vdim + 2 * kDc * (kDc + 4) + (size_t)kDcSlices * kDcTiles * 8 + kDc);
 }
 
 __global__ void __launch_bounds__(256, 2)
-delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict__ k, float* __restrict__ v, float* __restrict__ lg,
-                           const float* __restrict__ beta, float* __restrict__ w, float* __restrict__ qg, float* __restrict__ kd,
-                           float* __restrict__ bm, const int* __restrict__ seq_start, int heads, int kv_heads, int dim, int vdim,
-                           int max_chunks) {
+delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v,
+                           const float* __restrict__ lg, const float* __restrict__ beta, float* __restrict__ scratch,
+                           const int* __restrict__ seq_start, int heads, int kv_heads, int dim, int vdim, int max_chunks) {
     chain_release();
     chain_wait();
     extern __shared__ __align__(16) float dc_sm[];
-    const int s = blockIdx.x / max_chunks, h = blockIdx.y;
-    const int t0 = seq_start[s] + (int)(blockIdx.x % max_chunks) * kDc;
+    const int s = blockIdx.x / max_chunks, chunk = blockIdx.x - s * max_chunks, h = blockIdx.y;
+    const int start = seq_start[s], t0 = start + chunk * kDc;
     const int n = min(kDc, seq_start[s + 1] - t0);
     if (n <= 0) return;
-    const int hk = h / (heads / kv_heads), P = dim + 1, ap = kDc + 4;
-    float* sk = dc_sm;                        // [16][dim + 1]
+    const DcLayout lay(dim, vdim);
+    float* dst = scratch + (dc_place(start, s, chunk) * heads + h) * lay.floats;
+    const int hk = h / (heads / kv_heads), P = dim + 4, ap = kDc + 4, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* sk = dc_sm;                        // [16][dim + 4]
     float* sq = sk + kDc * P;
     float* sL = sq + kDc * P;                 // running sums of log2 decays
-    float* sA = sL + kDc * P + ((4 - (3 * kDc * P) % 4) & 3);        // [16][20], rows on 16-byte boundaries
+    float* sv = sL + kDc * P;                 // [16][vdim]
+    float* sA = sv + kDc * vdim;              // [16][20]
     float* sB = sA + kDc * ap;
     float* red = sB + kDc * ap;               // [slices][tiles][8]
     float* sb = red + kDcSlices * kDcTiles * 8;
-    for (int e = threadIdx.x; e < kDc * dim; e += blockDim.x) {
-        const int i = e / dim, d = e - i * dim;
+#pragma unroll
+    for (int it = 0; it < kDc / 8; ++it) {    // a warp a row
+        const int i = warp + 8 * it;
         const bool have = i < n;
-        sk[i * P + d] = have ? k[((size_t)(t0 + i) * kv_heads + hk) * dim + d] : 0.f;
-        sq[i * P + d] = have ? q[((size_t)(t0 + i) * kv_heads + hk) * dim + d] : 0.f;
-        sL[i * P + d] = have ? lg[((size_t)(t0 + i) * heads + h) * dim + d] * kDcLog2e : 0.f;
+        const float* kr = k + ((size_t)(t0 + i) * kv_heads + hk) * dim;
+        const float* qr = q + ((size_t)(t0 + i) * kv_heads + hk) * dim;
+        const float* lr = lg + ((size_t)(t0 + i) * heads + h) * dim;
+        const float* vr = v + ((size_t)(t0 + i) * heads + h) * vdim;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int d = 4 * lane; d < dim; d += 128) {
+            const float4 a = have ? dc_ld4(kr + d) : zero, b = have ? dc_ld4(qr + d) : zero, c = have ? dc_ld4(lr + d) : zero;
+            *reinterpret_cast<float4*>(sk + i * P + d) = a;
+            *reinterpret_cast<float4*>(sq + i * P + d) = b;
+            dc_st4(sL + i * P + d, c.x * kDcLog2e, c.y * kDcLog2e, c.z * kDcLog2e, c.w * kDcLog2e);
+        }
+        for (int d = 4 * lane; d < vdim; d += 128) *reinterpret_cast<float4*>(sv + i * vdim + d) = have ? dc_ld4(vr + d) : zero;
     }
     if (threadIdx.x < kDc) sb[threadIdx.x] = threadIdx.x < n ? beta[(size_t)(t0 + threadIdx.x) * heads + h] : 0.f;
+    for (int e = threadIdx.x; e < 2 * kDc * ap; e += 256) sA[e] = 0.f;              // A, then B
     __syncthreads();
-    for (int d = threadIdx.x; d < dim; d += blockDim.x) {
+    for (int d = threadIdx.x; d < dim; d += 256) {
         float acc = 0.f;
 #pragma unroll
         for (int i = 0; i < kDc; ++i) { acc += sL[i * P + d]; sL[i * P + d] = acc; }
     }
     __syncthreads();
     if (threadIdx.x < kDcTiles * kDcSlices) {
-        const int tile = threadIdx.x % kDcTiles, slice = threadIdx.x / kDcTiles;
+        const int slice = threadIdx.x / kDcTiles, tile = threadIdx.x - slice * kDcTiles;
         int ti = 0;
         while ((ti + 1) * (ti + 2) / 2 <= tile) ++ti;
         const int tj = tile - ti * (ti + 1) / 2;
-        const float *k0 = sk + 2 * ti * P, *k1 = k0 + P, *q0 = sq + 2 * ti * P, *q1 = q0 + P, *L0 = sL + 2 * ti * P, *L1 = L0 + P;
-        const float *x0 = sk + 2 * tj * P, *x1 = x0 + P, *M0 = sL + 2 * tj * P, *M1 = M0 + P;
+        const float *k0 = sk + 2 * ti * P, *q0 = sq + 2 * ti * P, *L0 = sL + 2 * ti * P, *x0 = sk + 2 * tj * P, *M0 = sL + 2 * tj * P;
         float a[4] = {0.f, 0.f, 0.f, 0.f}, b[4] = {0.f, 0.f, 0.f, 0.f};
         // pairs (i, j): (0,0) (0,1) (1,0) (1,1) of the tile; above the diagonal the exponent could be positive: cut off at zero
-        for (int d = slice; d < dim; d += kDcSlices) {
-            const float l0 = L0[d], l1 = L1[d], m0 = M0[d], m1 = M1[d];
-            const float e00 = x0[d] * exp2f(l0 - m0), e01 = x1[d] * exp2f(fminf(l0 - m1, 0.f));
-            const float e10 = x0[d] * exp2f(l1 - m0), e11 = x1[d] * exp2f(l1 - m1);
-            const float ka = k0[d], kb = k1[d], qa = q0[d], qb = q1[d];
-            a[0] = fmaf(ka, e00, a[0]); a[1] = fmaf(ka, e01, a[1]); a[2] = fmaf(kb, e10, a[2]); a[3] = fmaf(kb, e11, a[3]);
-            b[0] = fmaf(qa, e00, b[0]); b[1] = fmaf(qa, e01, b[1]); b[2] = fmaf(qb, e10, b[2]); b[3] = fmaf(qb, e11, b[3]);
+#define MDMA_DC_PAIRS(c)                                                                                                     \
+        {                                                                                                                    \
+            const float e00 = xa.c * dc_exp2(l0.c - m0.c), e01 = xb.c * dc_exp2(fminf(l0.c - m1.c, 0.f));                      \
+            const float e10 = xa.c * dc_exp2(l1.c - m0.c), e11 = xb.c * dc_exp2(l1.c - m1.c);                                 \
+            a[0] = fmaf(ka.c, e00, a[0]); a[1] = fmaf(ka.c, e01, a[1]); a[2] = fmaf(kb.c, e10, a[2]); a[3] = fmaf(kb.c, e11, a[3]); \
+            b[0] = fmaf(qa.c, e00, b[0]); b[1] = fmaf(qa.c, e01, b[1]); b[2] = fmaf(qb.c, e10, b[2]); b[3] = fmaf(qb.c, e11, b[3]); \
         }
+        for (int d = 4 * slice; d < dim; d += 4 * kDcSlices) {
+            const float4 l0 = dc_ld4(L0 + d), l1 = dc_ld4(L0 + P + d), m0 = dc_ld4(M0 + d), m1 = dc_ld4(M0 + P + d);
+            const float4 xa = dc_ld4(x0 + d), xb = dc_ld4(x0 + P + d);
+            const float4 ka = dc_ld4(k0 + d), kb = dc_ld4(k0 + P + d), qa = dc_ld4(q0 + d), qb = dc_ld4(q0 + P + d);
+            MDMA_DC_PAIRS(x) MDMA_DC_PAIRS(y) MDMA_DC_PAIRS(z) MDMA_DC_PAIRS(w)
+        }
+#undef MDMA_DC_PAIRS
         float* r = red + (slice * kDcTiles + tile) * 8;
-#pragma unroll
-        for (int e = 0; e < 4; ++e) { r[e] = a[e]; r[4 + e] = b[e]; }
+        dc_st4(r, a[0], a[1], a[2], a[3]);
+        dc_st4(r + 4, b[0], b[1], b[2], b[3]);
     }
-    for (int e = threadIdx.x; e < 2 * kDc * ap; e += blockDim.x) sA[e] = 0.f;        // A, then B
     __syncthreads();
-    for (int e = threadIdx.x; e < kDcTiles * 8; e += blockDim.x) {
+    for (int e = threadIdx.x; e < kDcTiles * 8; e += 256) {
         const int tile = e >> 3, x = e & 7;
         int ti = 0;
         while ((ti + 1) * (ti + 2) / 2 <= tile) ++ti;
@@ -99,17 +141,19 @@ delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict_
     }
     __syncthreads();
     // the triangular system: a thread per column of w (key channels) and z (value columns)
-    for (int c = threadIdx.x; c < dim + vdim; c += blockDim.x) {
-        const bool key = c < dim;
+    const int zcols = lay.slices * kDcCols;
+    for (int c = threadIdx.x; c < lay.dimP + zcols; c += 256) {
+        const bool key = c < lay.dimP;
+        const int cv = c - lay.dimP;
+        const bool real = key ? c < dim : cv < vdim;
         float u[kDc];
 #pragma unroll
         for (int i = 0; i < kDc; ++i) {
             float r = 0.f;
-            if (key) r = sk[i * P + c] * exp2f(sL[i * P + c]);
-            else if (i < n) r = v[((size_t)(t0 + i) * heads + h) * vdim + c - dim];
+            if (real) r = key ? sk[i * P + c] * dc_exp2(sL[i * P + c]) : sv[i * vdim + cv];
 #pragma unroll
             for (int j4 = 0; j4 < i; j4 += 4) {
-                const float4 a4 = *reinterpret_cast<const float4*>(sA + i * ap + j4);      // zero from the diagonal on
+                const float4 a4 = dc_ld4(sA + i * ap + j4);      // zero from the diagonal on
                 r = fmaf(-a4.x, u[j4], r);
                 if (j4 + 1 < i) r = fmaf(-a4.y, u[j4 + 1], r);
                 if (j4 + 2 < i) r = fmaf(-a4.z, u[j4 + 2], r);
@@ -117,27 +161,32 @@ delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict_
             }
             u[i] = sb[i] * r;
         }
+        float* to = key ? dst + c : dst + lay.z + (cv >> 4) * (kDc * 20) + (cv & 15);
+        const int pitch = key ? lay.wp : 20;
 #pragma unroll
-        for (int i = 0; i < kDc; ++i)
-            if (i < n) {
-                if (key) w[((size_t)(t0 + i) * heads + h) * dim + c] = u[i];
-                else v[((size_t)(t0 + i) * heads + h) * vdim + c - dim] = u[i];
-            }
+        for (int i = 0; i < kDc; ++i) to[i * pitch] = u[i];
     }
     const float* last = sL + (n - 1) * P;
-    for (int e = threadIdx.x; e < n * dim; e += blockDim.x) {
-        const int i = e / dim, d = e - i * dim;
-        const size_t at = ((size_t)(t0 + i) * heads + h) * dim + d;
-        qg[at] = sq[i * P + d] * exp2f(sL[i * P + d]);
-        kd[at] = sk[i * P + d] * exp2f(last[d] - sL[i * P + d]);
-        if (i == 0) lg[at] = exp2f(last[d]);              // the chunk's whole decay takes the place of its first row's
+#pragma unroll
+    for (int it = 0; it < kDc / 8; ++it) {
+        const int i = warp + 8 * it;
+        for (int d = 4 * lane; d < lay.dimP; d += 128) {
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
+            if (d < dim && i < n) {
+                const float4 L = dc_ld4(sL + i * P + d), E = dc_ld4(last + d), x = dc_ld4(sq + i * P + d), y = dc_ld4(sk + i * P + d);
+                a = make_float4(x.x * dc_exp2(L.x), x.y * dc_exp2(L.y), x.z * dc_exp2(L.z), x.w * dc_exp2(L.w));
+                b = make_float4(y.x * dc_exp2(E.x - L.x), y.y * dc_exp2(E.y - L.y), y.z * dc_exp2(E.z - L.z), y.w * dc_exp2(E.w - L.w));
+            }
+            *reinterpret_cast<float4*>(dst + lay.qg + i * lay.wp + d) = a;
+            *reinterpret_cast<float4*>(dst + lay.kd + i * lay.kp + d) = b;
+        }
     }
-    for (int e = threadIdx.x; e < n * kDc; e += blockDim.x)
-        bm[((size_t)(t0 + e / kDc) * heads + h) * kDc + e % kDc] = sB[(e / kDc) * ap + e % kDc];
+    for (int d = threadIdx.x; d < lay.dimP; d += 256) dst[lay.g + d] = d < dim ? dc_exp2(last[d]) : 0.f;
+    dst[lay.b + (threadIdx.x >> 4) * 24 + (threadIdx.x & 15)] = sB[(threadIdx.x >> 4) * ap + (threadIdx.x & 15)];
 }
 
 // ---------------------------------------------------------------- the walk
-constexpr int kDwCols = 16, kDwWarps = 4, kDwStages = 4;
+constexpr int kDwWarps = 4, kDwStages = 3;
 
 __device__ __forceinline__ void dw_mma(float* c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -152,29 +201,27 @@ __device__ __forceinline__ void dw_copy16(void* dst_shared, const void* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" :: "r"((uint32_t)__cvta_generic_to_shared(dst_shared)), "l"(src) : "memory");
 }
 
-// floats of one staged chunk: w, qg [16][dimP + 8]; kd [16][dimP + 4]; z [16][20]; B [16][24]; whole decay [dimP]
-static __host__ __device__ int dw_stage_floats(int dimP) { return kDc * (3 * dimP + 20 + 20 + 24) + dimP; }
+// floats of one staged chunk: everything of a (chunk, head) up to z, and z of the block's columns
+static __host__ __device__ constexpr int dw_stage_floats(int dimP) { return kDc * (3 * dimP + 20 + 24) + dimP + kDc * 20; }
 static size_t dw_smem(int dimP) { return sizeof(float) * ((size_t)kDwStages * dw_stage_floats(dimP) + kDwWarps * 16 * 32); }
 
 // NTD: tiles of eight key channels a warp has (dim up to 32 * NTD)
 template <int NTD>
 __global__ void __launch_bounds__(kDwWarps * 32)
-delta_chunk_walk_kernel(const float* __restrict__ w, const float* __restrict__ qg, const float* __restrict__ kd,
-                        const float* __restrict__ z, const float* __restrict__ bm, const float* __restrict__ whole,
-                        const int* __restrict__ seq_start, const int* __restrict__ seq_slot, float* __restrict__ state,
-                        size_t state_stride, float* __restrict__ out, int heads, int dim, int vdim) {
+delta_chunk_walk_kernel(const float* __restrict__ scratch, const int* __restrict__ seq_start, const int* __restrict__ seq_slot,
+                        float* __restrict__ state, size_t state_stride, float* __restrict__ out, int heads, int dim, int vdim) {
     chain_release();
     chain_wait();
     extern __shared__ __align__(16) float dw_sm[];
-    constexpr int dimP = 32 * NTD, wp = dimP + 8, kp = dimP + 4, zp = 20, bp = 24;
-    const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kDwCols, cw = min(kDwCols, vdim - c0);
+    constexpr int dimP = 32 * NTD, wp = dimP + 8, kp = dimP + 4, zp = 20, bp = 24, stage_floats = dw_stage_floats(dimP);
+    constexpr int common = stage_floats - kDc * zp;
+    const int s = blockIdx.x, h = blockIdx.y, c0 = blockIdx.z * kDcCols, cw = min(kDcCols, vdim - c0);
     const int t0 = seq_start[s], t1 = seq_start[s + 1];
     if (t1 <= t0) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lr = lane >> 2, lc = lane & 3;
-    const int stage_floats = dw_stage_floats(dimP);
     float* red = dw_sm + (size_t)kDwStages * stage_floats;       // [warp][16][32 lanes]
-    for (int e = threadIdx.x; e < kDwStages * stage_floats; e += blockDim.x) dw_sm[e] = 0.f;      // padding stays zero
-    const int chunks = (t1 - t0 + kDc - 1) / kDc, d4 = dim >> 2, c4 = cw >> 2;
+    const int chunks = (t1 - t0 + kDc - 1) / kDc;
+    const DcLayout lay(dim, vdim);
     float* st = state + (size_t)seq_slot[s] * state_stride + (size_t)h * dim * vdim;
     float S[NTD][4];                  // S^T: columns lr, lr + 8; channels warp * 8 NTD + 8 nt + 2 lc, + 1
 #pragma unroll
@@ -184,57 +231,38 @@ delta_chunk_walk_kernel(const float* __restrict__ w, const float* __restrict__ q
             const int c = lr + (e >> 1) * 8, d = warp * 8 * NTD + nt * 8 + 2 * lc + (e & 1);
             S[nt][e] = (c < cw && d < dim) ? st[(size_t)d * vdim + c0 + c] : 0.f;
         }
-    __syncthreads();
+    const size_t chunk_pitch = (size_t)heads * lay.floats;
+    const float* next = scratch + (dc_place(t0, s, 0) * heads + h) * lay.floats + 4 * threadIdx.x;
+    const int z_from = lay.z + (int)blockIdx.z * kDc * zp - common;        // the block's z, seen from where `common` ends
+    int fill = 0;                                                           // the stage that is filled next
     auto issue = [&](int chunk) {
         if (chunk < chunks) {
-            float* sw = dw_sm + (size_t)(chunk % kDwStages) * stage_floats;
-            float* sqg = sw + kDc * wp;
-            float* skd = sqg + kDc * wp;
-            float* sz = skd + kDc * kp;
-            float* sB = sz + kDc * zp;
-            float* sg = sB + kDc * bp;
-            const int r0 = t0 + chunk * kDc, n = min(kDc, t1 - r0);
-            for (int e = threadIdx.x; e < kDc * d4; e += blockDim.x) {
-                const int i = e / d4, p = (e - i * d4) << 2;
-                if (i < n) {
-                    const size_t at = ((size_t)(r0 + i) * heads + h) * dim + p;
-                    dw_copy16(sw + i * wp + p, w + at);
-                    dw_copy16(sqg + i * wp + p, qg + at);
-                    dw_copy16(skd + i * kp + p, kd + at);
-                } else {
-                    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-                    *reinterpret_cast<float4*>(sw + i * wp + p) = zero;
-                    *reinterpret_cast<float4*>(sqg + i * wp + p) = zero;
-                    *reinterpret_cast<float4*>(skd + i * kp + p) = zero;
-                }
-            }
-            for (int e = threadIdx.x; e < kDc * 4; e += blockDim.x) {
-                const int i = e >> 2, p = (e & 3) << 2;
-                const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (i < n) {
-                    if ((e & 3) < c4) dw_copy16(sz + i * zp + p, z + ((size_t)(r0 + i) * heads + h) * vdim + c0 + p);
-                    dw_copy16(sB + i * bp + p, bm + ((size_t)(r0 + i) * heads + h) * kDc + p);
-                } else {
-                    *reinterpret_cast<float4*>(sz + i * zp + p) = zero;
-                    *reinterpret_cast<float4*>(sB + i * bp + p) = zero;
-                }
-            }
-            for (int e = threadIdx.x; e < d4; e += blockDim.x) dw_copy16(sg + 4 * e, whole + ((size_t)r0 * heads + h) * dim + 4 * e);
+            float* to = dw_sm + fill * stage_floats + 4 * threadIdx.x;
+#pragma unroll
+            for (int e = 0; e < common; e += 4 * kDwWarps * 32)
+                if (e + 4 * (int)threadIdx.x < common) dw_copy16(to + e, next + e);
+            if (threadIdx.x < kDc * zp / 4) dw_copy16(to + common, next + common + z_from);
+            next += chunk_pitch;
+            fill = fill + 1 == kDwStages ? 0 : fill + 1;
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
 #pragma unroll
     for (int p = 0; p < kDwStages - 1; ++p) issue(p);
+    int stage = 0;
+    float* orow = out + ((size_t)(t0 + (warp & 1) * 8 + 2 * lc) * heads + h) * vdim + c0 + lr;       // warps 0 and 1
+    const size_t opitch = (size_t)heads * vdim;
     for (int chunk = 0; chunk < chunks; ++chunk) {
         asm volatile("cp.async.wait_group %0;" :: "n"(kDwStages - 2) : "memory");
         __syncthreads();                       // this chunk is there for everyone; the one before is done with
         issue(chunk + kDwStages - 1);
-        const float* sw = dw_sm + (size_t)(chunk % kDwStages) * stage_floats;
+        const float* sw = dw_sm + stage * stage_floats;
         const float* sqg = sw + kDc * wp;
         const float* skd = sqg + kDc * wp;
-        const float* sz = skd + kDc * kp;
-        const float* sB = sz + kDc * zp;
+        const float* sB = skd + kDc * kp;
         const float* sg = sB + kDc * bp;
+        const float* sz = sg + dimP;
+        stage = stage + 1 == kDwStages ? 0 : stage + 1;
         // this warp's channels of S^T w and S^T q: [matrix][rows 0-7 | 8-15][4]; the three partial products on their own
         float pa[2][2][4], pb[2][2][4];
 #pragma unroll
@@ -302,12 +330,16 @@ delta_chunk_walk_kernel(const float* __restrict__ w, const float* __restrict__ q
                 dw_mma(o, uh[r][0], uh[r][1], uh[r][2], uh[r][3], bl0, bl1);
                 dw_mma(o, uh[r][0], uh[r][1], uh[r][2], uh[r][3], bh0, bh1);
             }
-            const int i0 = chunk * kDc + warp * 8 + 2 * lc;
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int c = lr + (e >> 1) * 8, i = i0 + (e & 1);
-                if (c < cw && t0 + i < t1) out[((size_t)(t0 + i) * heads + h) * vdim + c0 + c] = o[e];
+            const int left = t1 - t0 - chunk * kDc - warp * 8 - 2 * lc;
+            if (lr < cw) {
+                if (left > 0) orow[0] = o[0];
+                if (left > 1) orow[opitch] = o[1];
             }
+            if (lr + 8 < cw) {
+                if (left > 0) orow[8] = o[2];
+                if (left > 1) orow[opitch + 8] = o[3];
+            }
+            orow += kDc * opitch;
         }
         // S^T <- S^T e^(L_n) + u^T kd
 #pragma unroll
@@ -344,38 +376,44 @@ using namespace mdma;
 
 extern "C" {
 
-// q, k [rows][kv_heads * dim], v [rows][heads * vdim] (becomes z), lg [rows][heads * dim] (a chunk's first row becomes its
-// whole decay), beta [rows][heads]; w, qg, kd [rows][heads * dim] and bm [rows][heads * 16] are scratch; out [rows][heads * vdim]
-int mdma_delta_chunks(const float* q, const float* k, float* v, float* lg, const float* beta, float* w, float* qg, float* kd,
-                      float* bm, const int* seq_start, const int* seq_slot, float* state, long state_stride, float* out,
+// Floats of scratch a step of n_rows rows in n_seqs sequences needs.
+long mdma_delta_chunks_scratch(int n_rows, int n_seqs, int heads, int dim, int vdim) {
+    return ((long)n_rows / kDc + n_seqs + 1) * heads * (long)DcLayout(dim, vdim).floats;
+}
+
+// q, k [rows][kv_heads * dim], v, out [rows][heads * vdim], lg [rows][heads * dim], beta [rows][heads], all floats
+int mdma_delta_chunks(const float* q, const float* k, const float* v, const float* lg, const float* beta, float* scratch,
+                      long scratch_floats, const int* seq_start, const int* seq_slot, float* state, long state_stride, float* out,
                       int n_rows, int n_seqs, int max_new, int heads, int kv_heads, int dim, int vdim, cudaStream_t stream) {
     MDMA_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0, "delta_chunks: bad sizes");
-    MDMA_REQUIRE(dim <= kDcMaxDim && dim % 4 == 0 && vdim % 4 == 0, "delta_chunks: heads of %d x %d are not a geometry this kernel takes", dim, vdim);
-    MDMA_REQUIRE((((uintptr_t)v | (uintptr_t)lg | (uintptr_t)w | (uintptr_t)qg | (uintptr_t)kd | (uintptr_t)bm) & 15) == 0, "delta_chunks: rows must start on 16 bytes");
+    MDMA_REQUIRE(dim <= kDcMaxDim && dim % 4 == 0 && vdim % 4 == 0 && vdim <= 512, "delta_chunks: heads of %d x %d are not a geometry this kernel takes", dim, vdim);
+    MDMA_REQUIRE((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)lg | (uintptr_t)scratch) & 15) == 0, "delta_chunks: rows must start on 16 bytes");
     if (n_rows == 0 || n_seqs == 0) return 0;
+    const long need = mdma_delta_chunks_scratch(n_rows, n_seqs, heads, dim, vdim);
+    MDMA_REQUIRE(scratch_floats >= need, "delta_chunks: %ld floats of scratch needed, %ld given", need, scratch_floats);
     const int max_chunks = (max_new + kDc - 1) / kDc;
     MDMA_REQUIRE((long)n_seqs * max_chunks <= 2147483647l && heads <= 65535, "delta_chunks: too many rows");
     static bool raised = false;
     if (!raised) {
-        cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+        cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
         raised = true;
     }
-    launch_chained(delta_chunk_prepare_kernel, dim3((unsigned)(n_seqs * max_chunks), heads), dim3(256), dc_prepare_smem(dim) + 16, stream,
-                   q, k, v, lg, beta, w, qg, kd, bm, seq_start, heads, kv_heads, dim, vdim, max_chunks);
+    launch_chained(delta_chunk_prepare_kernel, dim3((unsigned)(n_seqs * max_chunks), heads), dim3(256), dc_prepare_smem(dim, vdim), stream,
+                   q, k, v, lg, beta, scratch, seq_start, heads, kv_heads, dim, vdim, max_chunks);
     MDMA_LAUNCH_OK("delta_chunk_prepare");
-    dim3 grid(n_seqs, heads, (vdim + kDwCols - 1) / kDwCols);
+    const DcLayout lay(dim, vdim);
+    dim3 grid(n_seqs, heads, lay.slices);
 #define MDMA_DW(NTD)                                                                                                     \
     do {                                                                                                                 \
         static bool up = false;                                                                                          \
         if (!up) { cudaFuncSetAttribute(delta_chunk_walk_kernel<NTD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dw_smem(32 * NTD)); up = true; } \
-        launch_chained(delta_chunk_walk_kernel<NTD>, grid, dim3(kDwWarps * 32), dw_smem(32 * NTD), stream, (const float*)w,  \
-                       (const float*)qg, (const float*)kd, (const float*)v, (const float*)bm, (const float*)lg, seq_start, \
-                       seq_slot, state, (size_t)state_stride, out, heads, dim, vdim);                                    \
+        launch_chained(delta_chunk_walk_kernel<NTD>, grid, dim3(kDwWarps * 32), dw_smem(32 * NTD), stream, (const float*)scratch, \
+                       seq_start, seq_slot, state, (size_t)state_stride, out, heads, dim, vdim);                         \
     } while (0)
-    if (dim <= 32) MDMA_DW(1);
-    else if (dim <= 64) MDMA_DW(2);
-    else if (dim <= 96) MDMA_DW(3);
-    else if (dim <= 128) MDMA_DW(4);
+    if (lay.dimP == 32) MDMA_DW(1);
+    else if (lay.dimP == 64) MDMA_DW(2);
+    else if (lay.dimP == 96) MDMA_DW(3);
+    else if (lay.dimP == 128) MDMA_DW(4);
     else MDMA_DW(8);
 #undef MDMA_DW
     MDMA_LAUNCH_OK("delta_chunk_walk");

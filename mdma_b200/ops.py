@@ -881,16 +881,23 @@ def delta_scan(q, k, v, lg, beta, ctx, state, out, heads: int, kv_heads: int, di
           sp, ss, _ptr(out), _i(ctx.n_seqs), _i(heads), _i(kv_heads), _i(dim), _i(vdim), _stream())
 
 
-def delta_chunks(q, k, v, lg, beta, w, qg, kd, bm, ctx, state, out, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
-    """`delta_scan` a chunk of sixteen rows at a time (equal up to rounding; dim and vdim multiples of four).  v and lg are
-    overwritten; w, qg, kd [T, heads * dim] and bm [T, heads * 16] are scratch."""
-    _need_cuda(q, k, v, lg, beta, w, qg, kd, bm, state, out)
-    for t, c in ((q, kv_heads * dim), (k, kv_heads * dim), (v, heads * vdim), (lg, heads * dim), (beta, heads), (out, heads * vdim),
-                 (w, heads * dim), (qg, heads * dim), (kd, heads * dim), (bm, heads * 16)):
+def delta_chunk_floats(heads: int, dim: int, vdim: int) -> int:
+    """Floats of scratch of one chunk of sixteen rows (the layout of csrc/delta_chunk.cu; a step of T rows in B sequences
+    has T // 16 + B + 1 places)."""
+    padded = -(-dim // 32) * 32 if dim <= 128 else 256
+    return heads * (16 * (3 * padded + 44) + padded + -(-vdim // 16) * 320)
+
+
+def delta_chunks(q, k, v, lg, beta, scratch, ctx, state, out, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
+    """`delta_scan` a chunk of sixteen rows at a time (equal up to rounding; dim and vdim multiples of four).  `scratch`:
+    (T // 16 + sequences + 1) * `delta_chunk_floats` floats."""
+    _need_cuda(q, k, v, lg, beta, scratch, state, out)
+    for t, c in ((q, kv_heads * dim), (k, kv_heads * dim), (v, heads * vdim), (lg, heads * dim), (beta, heads), (out, heads * vdim)):
         assert t.dtype == torch.float32 and t.is_contiguous() and t.shape[1] == c and t.shape[0] >= ctx.n_tokens
+    assert scratch.dtype == torch.float32 and scratch.is_contiguous()
     sp, ss = _state(state)
     assert state.shape[1] >= heads * dim * vdim
-    _call("core", "mdma_delta_chunks", _ptr(q), _ptr(k), _ptr(v), _ptr(lg), _ptr(beta), _ptr(w), _ptr(qg), _ptr(kd), _ptr(bm),
+    _call("core", "mdma_delta_chunks", _ptr(q), _ptr(k), _ptr(v), _ptr(lg), _ptr(beta), _ptr(scratch), ctypes.c_long(scratch.numel()),
           _ptr(ctx.seq_start), _ptr(ctx.seq_slot), sp, ss, _ptr(out), _i(ctx.n_tokens), _i(ctx.n_seqs), _i(ctx.max_new),
           _i(heads), _i(kv_heads), _i(dim), _i(vdim), _stream(), launches=2)
 

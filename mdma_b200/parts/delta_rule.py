@@ -55,7 +55,7 @@ class ChannelDelta(Part):
         self.inner_width = self.decay_rank + self.gate_rank
         self.state_floats = self.heads * self.dim * self.v_dim
         self.conv_at = -(-self.state_floats // 4) * 4
-        self.chunks_fit = self.dim % 4 == 0 and self.v_dim % 4 == 0
+        self.chunks_fit = self.dim % 4 == 0 and self.v_dim % 4 == 0 and self.v_dim <= 512
         self.conv_floats = (self.taps - 1) * self.channels
 
     def check_limits(self, rt):
@@ -90,7 +90,7 @@ class ChannelDelta(Part):
 
     def _names(self):
         tag = f"{self.heads}_{self.kv_heads}_{self.dim}_{self.v_dim}"
-        return {n: f"delta_{n}_{tag}" for n in ("proj", "q", "k", "v", "lg", "beta", "raw", "gate", "sum", "out", "qg", "kd", "bm")}
+        return {n: f"delta_{n}_{tag}" for n in ("proj", "q", "k", "v", "lg", "beta", "raw", "gate", "sum", "out", "chunks")}
 
     def workspace(self):
         n = self._names()
@@ -99,13 +99,17 @@ class ChannelDelta(Part):
               n["raw"]: (self.k_width, "f32"), n["gate"]: (self.v_width, "act"), n["sum"]: (self.v_width, "f32"),
               n["out"]: (self.v_width, "act")}
         if self.chunks_fit:
-            ws.update({n["qg"]: (self.k_width, "f32"), n["kd"]: (self.k_width, "f32"), n["bm"]: (16 * self.heads, "f32")})
+            ws[n["chunks"]] = (self._chunk_columns(), "f32")
         if self.inner_fused:
             ws[f"delta_inner_{self.inner_width}"] = (-(-self.inner_width // 8) * 8, "act")
         else:
             ws[f"delta_a1_{self.decay_rank}"] = (-(-self.decay_rank // 8) * 8, "act")
             ws[f"delta_g1_{self.gate_rank}"] = (-(-self.gate_rank // 8) * 8, "act")
         return ws
+
+    def _chunk_columns(self) -> int:
+        # scratch of the chunks side by side: a row's share, and an eighth more for sequences' last, partial chunks
+        return -(-9 * ops.delta_chunk_floats(self.heads, self.dim, self.v_dim) // 128)
 
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
@@ -153,10 +157,14 @@ class ChannelDelta(Part):
         self._low_rank(ctx, h, raw, gate)
         ops.delta_prepare(proj, raw, self.conv, self.taps, self.a_log, self.dt_bias, ctx, conv_state, q, k, v, lg, beta,
                           self.heads, self.kv_heads, self.dim, self.v_dim, self.unit_eps, self.dim ** -0.5)
+        chunks = None
         if self.chunks_fit and self.rt.dtype != f32 and ctx.max_new >= self.CHUNKS_FROM:
-            # (the decays' inputs are spent: their rows take the solved right sides)
-            ops.delta_chunks(q, k, v, lg, beta, raw, ctx.buf(names["qg"], self.k_width, f32), ctx.buf(names["kd"], self.k_width, f32),
-                             ctx.buf(names["bm"], 16 * self.heads, f32), ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
+            # (room for them all, unless very many short sequences come with a long one)
+            chunks = ctx.buf(names["chunks"], self._chunk_columns(), f32).view(-1)
+            if (n // 16 + ctx.n_seqs + 1) * ops.delta_chunk_floats(self.heads, self.dim, self.v_dim) > chunks.numel():
+                chunks = None
+        if chunks is not None:
+            ops.delta_chunks(q, k, v, lg, beta, chunks, ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
         else:
             ops.delta_scan(q, k, v, lg, beta, ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
         ops.gated_head_rmsnorm(sums, gate, self.norm, out, n, self.heads, self.v_dim, self.eps)
