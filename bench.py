@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl reference]
     python bench.py --shape llama-2-7b | llama-3.2-1b [--batch B] [--prompt-len P] [--prefill-tokens T]
-    python bench.py --compare gevonex|mogevik|tubusun|fizadra [--compare-widths 1024,2048,4096] [--compare-layers 4]
+    python bench.py --compare gevonex|mogevik|tubusun|fizadra|degavik [--compare-widths 1024,2048,4096] [--compare-layers 4]
 
 Prints ONE JSON line.  The default run has the layer sizes of the
 Llama-3.1-8B shape with random bfloat16 weights, a batch of 8 sequences
@@ -35,6 +35,12 @@ and a Llama of the same width, depth and vocabulary.
 over a cached latent with a turned key part, attention whose heads' scores
 are mixed, grouped norms around every sublayer, a weighted sum over the
 depth) beside a Gevonex (the other model with a cached latent) and a Llama.
+
+`--compare degavik` does the same for the Degavik architecture (a gated delta
+rule, windowed attention whose heads' weights are mixed, retention, dense and
+routed feed-forwards, norms after the sublayers) beside a Tubusun (the other
+model with linear attention and routed experts), a Fizadra (the other one whose
+heads are mixed) and a Llama.
 """
 from __future__ import annotations
 
@@ -221,6 +227,26 @@ def fizadra_config(width: int, layers: int, vocab: int) -> dict:
     return {"architecture": "Fizadra", "vocab": vocab, "width": width, "norm": {"eps": 1e-5, "groups": 4}, "layers": out}
 
 
+def degavik_config(width: int, layers: int, vocab: int) -> dict:
+    """A Degavik of `layers` layers (delta rule, attention, retention, delta rule, ...) whose sizes follow the width:
+    heads of 128 x 128 throughout, four taps and low-rank projections of 128 for the delta rule; query heads in groups of
+    four over a window of 1,024 and the first four tokens, half of each head turned; retention decays from 0.97 to 0.9995;
+    dense feed-forwards of 8/3 x width (the parameters of 4 x width without a gate) and, in every second layer, sixteen
+    experts of width / 2, four per token, beside a shared one of width / 2."""
+    heads = max(1, width // 128)
+    mixers = {"channel_delta": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128,
+                                "gate_rank": 128},
+              "attention": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 0.09,
+                            "softcap": 30.0, "mask": {"size": 1024, "keep_first": 4}, "rot": {"dims": 64, "base": 10000.0}},
+              "retention": {"heads": heads, "dim": 128, "vdim": 128, "rot": {"dims": 128, "base": 10000.0},
+                            "decay": [1.0 - 0.03 * (1.0 / 60.0) ** (h / max(1, heads - 1)) for h in range(heads)]}}
+    kinds = ["channel_delta", "attention", "retention", "channel_delta"]
+    moe = {"kind": "moe", "expert": {"ff": width // 2}, "router": {"experts": 16, "top": 4}, "shared": {"ff": width // 2}}
+    dense = {"kind": "dense", "ff": (8 * width // 3 + 63) // 64 * 64}
+    return {"architecture": "Degavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "layers": [{"type": kinds[i % 4], "mixer": mixers[kinds[i % 4]], "mlp": moe if i % 2 else dense} for i in range(layers)]}
+
+
 def expert_share(cfg: dict, name: str, draws: int) -> float:
     """The share of an expert's matrix that a step of `draws` tokens reads (decode: distinct experts among the
     draws, chosen evenly) or, with draws = 0, the share of tokens that use it (prefill)."""
@@ -267,7 +293,7 @@ def compare(args) -> int:
                 n = 1
                 for d in ts.shape:
                     n *= d
-                routed = cfg.get("architecture") in ("Mogevik", "Tubusun")
+                routed = cfg.get("architecture") in ("Degavik", "Mogevik", "Tubusun")
                 matrix_bytes += 2 * n * (expert_share(cfg, name, batch) if routed else 1.0)
                 prefill_elements += n * (expert_share(cfg, name, 0) if routed else 1.0)
         # what a decode step moves besides the matrices: every live sequence's fixed-size state is read and written,
@@ -326,17 +352,19 @@ def compare(args) -> int:
     rows = []
     for width in [int(w) for w in args.compare_widths.split(",")]:
         row = {"width": width, "layers": args.compare_layers, "vocab": vocab, "batch": args.batch}
-        if args.compare == "fizadra":
+        if args.compare == "degavik":
+            row["degavik"] = measure(degavik_config(width, args.compare_layers, vocab), args.batch)
+        if args.compare in ("fizadra", "degavik"):
             row["fizadra"] = measure(fizadra_config(width, args.compare_layers, vocab), args.batch)
-        if args.compare == "tubusun":
+        if args.compare in ("tubusun", "degavik"):
             row["tubusun"] = measure(tubusun_config(width, args.compare_layers, vocab), args.batch)
         if args.compare in ("mogevik", "tubusun"):
             row["mogevik"] = measure(mogevik_config(width, args.compare_layers, vocab), args.batch)
-        if args.compare != "tubusun":
+        if args.compare not in ("tubusun", "degavik"):
             row["gevonex"] = measure(gevonex_config(width, args.compare_layers, vocab), args.batch)
         row["llama"] = measure(llama_like(width, args.compare_layers, vocab), args.batch)
         rows.append(row)
-    beside = {"fizadra": "fizadra beside gevonex and llama", "tubusun": "tubusun beside mogevik and llama", "mogevik": "mogevik beside gevonex and llama",
+    beside = {"degavik": "degavik beside tubusun, fizadra and llama", "fizadra": "fizadra beside gevonex and llama", "tubusun": "tubusun beside mogevik and llama", "mogevik": "mogevik beside gevonex and llama",
               "gevonex": "gevonex beside llama"}[args.compare]
     print(json.dumps({"compare": beside + " at equal width, depth and vocabulary", "dtype": args.dtype,
                       "prefill_tokens": T, "decode_after_prompts_of": prompt, "peaks": peak_src,
@@ -365,7 +393,7 @@ def main() -> int:
     ap.add_argument("--prefill-only", action="store_true", help="run only the 2,048-token prefill (profiling runs)")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
                     help="float32: the true 32-bit engine (CUDA-core kernels), for the record; the headline is bfloat16")
-    ap.add_argument("--compare", default=None, choices=["gevonex", "mogevik", "tubusun", "fizadra"],
+    ap.add_argument("--compare", default=None, choices=["gevonex", "mogevik", "tubusun", "fizadra", "degavik"],
                     help="another program: the named architecture beside a Llama of equal size (see the header)")
     ap.add_argument("--compare-widths", default="1024,2048,4096")
     ap.add_argument("--compare-layers", type=int, default=4)

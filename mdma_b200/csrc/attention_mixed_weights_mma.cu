@@ -452,16 +452,16 @@ mixed_merge_kernel(const float* __restrict__ partial, const float* __restrict__ 
     const float* src = partial + (size_t)s * splits * pitch;
     float* fac = msm;
     float* red = msm + splits * n_heads;
-    for (int h = threadIdx.x; h < n_heads; h += blockDim.x) {
-        float M = -INFINITY, L = 0.f;
-        for (int k = 0; k < splits; ++k) M = fmaxf(M, src[k * pitch + (size_t)n_heads * total + h]);
-        for (int k = 0; k < splits; ++k) {
-            const float e = exp2f(src[k * pitch + (size_t)n_heads * total + h] - M);          // 0 for a run without keys
-            fac[k * n_heads + h] = e;
-            L = fmaf(src[k * pitch + (size_t)n_heads * total + n_heads + h], e, L);
-        }
-        const float inv = 1.0f / L;
-        for (int k = 0; k < splits; ++k) fac[k * n_heads + h] *= inv;
+    // a warp per head, lanes over the runs: factors that turn each run's sums into parts of the normalised row
+    for (int h = threadIdx.x / 32; h < n_heads; h += kMergeCols * kMergeParts / 32) {
+        const int k0 = threadIdx.x & 31, k1 = k0 + 32;
+        const float* stat = src + (size_t)n_heads * total + h;
+        const float m0 = k0 < splits ? stat[k0 * pitch] : -INFINITY, m1 = k1 < splits ? stat[k1 * pitch] : -INFINITY;
+        const float l0 = k0 < splits ? stat[k0 * pitch + n_heads] : 0.f, l1 = k1 < splits ? stat[k1 * pitch + n_heads] : 0.f;
+        const float M = warp_max(fmaxf(m0, m1)), e0 = exp2f(m0 - M), e1 = exp2f(m1 - M);          // 0 for a run without keys
+        const float inv = 1.0f / warp_sum(fmaf(l0, e0, l1 * e1));
+        if (k0 < splits) fac[k0 * n_heads + h] = e0 * inv;
+        if (k1 < splits) fac[k1 * n_heads + h] = e1 * inv;
     }
     __syncthreads();
     const int lane = threadIdx.x % kMergeCols, part = threadIdx.x / kMergeCols;

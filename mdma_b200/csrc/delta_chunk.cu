@@ -7,7 +7,8 @@
 // No exponent is ever above zero.
 //
 // delta_chunk_prepare, block = (chunk, head), all chunks side by side: everything that does not depend on S, left in
-// scratch as one run of floats per (chunk, head), laid out as the walk's shared memory (`DcLayout`).  The
+// scratch as one run of floats per (chunk, head), laid out as the walk's shared memory (`DcLayout`).  It starts from the
+// projections: the short convolutions with silu, unit vectors, step sizes and the decays' logarithms are made here too.  The
 // triangular system is solved for its two right sides, w_i = b_i (e^(L_i) k_i - sum A_ij w_j) and z_i = b_i (v_i - sum
 // A_ij z_j), so that u = z - S^T w; also e^(L_i) q_i, e^(L_n - L_j) k_j, B and e^(L_n).
 // delta_chunk_walk, block = (sequence, head, sixteen columns of S), 4 warps, chunks in order: S^T lies in the accumulators
@@ -15,7 +16,7 @@
 // are; the warps' partial sums meet in shared memory once a chunk.  Products in float precision from tf32 pairs: every
 // number is split into the part the tensor core reads and the rest, and three of the four products are summed.
 // The next chunks' rows are on their way (cp.async) while a chunk is computed.
-#include "common.cuh"
+#include "delta_rule.cuh"
 
 namespace mdma {
 
@@ -53,10 +54,13 @@ static size_t dc_prepare_smem(int dim, int vdim) {
     return sizeof(float) * ((size_t)3 * kDc * (dim + 4) + (size_t)kDc * vdim + 2 * kDc * (kDc + 4) + (size_t)kDcSlices * kDcTiles * 8 + kDc);
 }
 
+template <int TAPS>      // the convolution's taps (shorter ones: zeros in front), or 0: any number, every input read again
 __global__ void __launch_bounds__(256, 2)
-delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v,
-                           const float* __restrict__ lg, const float* __restrict__ beta, float* __restrict__ scratch,
-                           const int* __restrict__ seq_start, int heads, int kv_heads, int dim, int vdim, int max_chunks) {
+delta_chunk_prepare_kernel(const float* __restrict__ proj, int proj_stride, const float* __restrict__ raw, const void* __restrict__ conv_w,
+                           int conv_dtype, int taps, const void* __restrict__ a_log, const void* __restrict__ dt_bias, int vec_dtype,
+                           const float* __restrict__ conv_state, size_t state_stride, float* __restrict__ scratch,
+                           const int* __restrict__ seq_start, const int* __restrict__ seq_slot, int heads, int kv_heads, int dim,
+                           int vdim, int max_chunks, float unit_eps, float q_scale) {
     chain_release();
     chain_wait();
     extern __shared__ __align__(16) float dc_sm[];
@@ -75,30 +79,67 @@ delta_chunk_prepare_kernel(const float* __restrict__ q, const float* __restrict_
     float* sB = sA + kDc * ap;
     float* red = sB + kDc * ap;               // [slices][tiles][8]
     float* sb = red + kDcSlices * kDcTiles * 8;
+    // convolutions with silu, a thread a channel: q's, k's and v's of this head
+    const int qk = kv_heads * dim, channels = 2 * qk + heads * vdim;
+    const float* kept = conv_state + (size_t)seq_slot[s] * state_stride;
+    for (int e = threadIdx.x; e < 2 * dim + vdim; e += 256) {
+        const int ch = e < dim ? hk * dim + e : e < 2 * dim ? qk + hk * dim + e - dim : 2 * qk + h * vdim + e - 2 * dim;
+        float* to = e < dim ? sq + e : e < 2 * dim ? sk + e - dim : sv + e - 2 * dim;
+        const int pitch = e < 2 * dim ? P : vdim;
+        const float* src = proj + (size_t)t0 * proj_stride + ch;
+        if (TAPS > 0) {
+            float w[TAPS > 0 ? TAPS : 1], x[kDc + (TAPS > 0 ? TAPS : 1) - 1];
 #pragma unroll
-    for (int it = 0; it < kDc / 8; ++it) {    // a warp a row
-        const int i = warp + 8 * it;
-        const bool have = i < n;
-        const float* kr = k + ((size_t)(t0 + i) * kv_heads + hk) * dim;
-        const float* qr = q + ((size_t)(t0 + i) * kv_heads + hk) * dim;
-        const float* lr = lg + ((size_t)(t0 + i) * heads + h) * dim;
-        const float* vr = v + ((size_t)(t0 + i) * heads + h) * vdim;
-        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int d = 4 * lane; d < dim; d += 128) {
-            const float4 a = have ? dc_ld4(kr + d) : zero, b = have ? dc_ld4(qr + d) : zero, c = have ? dc_ld4(lr + d) : zero;
-            *reinterpret_cast<float4*>(sk + i * P + d) = a;
-            *reinterpret_cast<float4*>(sq + i * P + d) = b;
-            dc_st4(sL + i * P + d, c.x * kDcLog2e, c.y * kDcLog2e, c.z * kDcLog2e, c.w * kDcLog2e);
+            for (int j = 0; j < TAPS; ++j) w[j] = j >= TAPS - taps ? delta_weight(conv_w, conv_dtype, (size_t)ch * taps + j - (TAPS - taps)) : 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) {
+                const int back = TAPS - 1 - j, at = t0 - back - start;           // rows before this step's first: kept inputs
+                x[j] = back > taps - 1 ? 0.f : at >= 0 ? src[-(ptrdiff_t)back * proj_stride] : kept[(size_t)(taps - 1 + at) * channels + ch];
+            }
+#pragma unroll
+            for (int i = 0; i < kDc; ++i) x[TAPS - 1 + i] = i < n ? src[(size_t)i * proj_stride] : 0.f;
+#pragma unroll
+            for (int i = 0; i < kDc; ++i) {
+                float acc = 0.f;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j], x[i + j], acc);
+                to[i * pitch] = i < n ? delta_silu(acc) : 0.f;
+            }
+        } else {
+            for (int i = 0; i < kDc; ++i)
+                to[i * pitch] = i < n ? delta_conv(proj, proj_stride, kept, conv_w, conv_dtype, taps, channels, t0 + i, start, ch) : 0.f;
         }
-        for (int d = 4 * lane; d < vdim; d += 128) *reinterpret_cast<float4*>(sv + i * vdim + d) = have ? dc_ld4(vr + d) : zero;
     }
-    if (threadIdx.x < kDc) sb[threadIdx.x] = threadIdx.x < n ? beta[(size_t)(t0 + threadIdx.x) * heads + h] : 0.f;
+    const float rate = -expf(delta_weight(a_log, vec_dtype, h)) * kDcLog2e;
+    for (int d = threadIdx.x; d < dim; d += 256) {
+        const float bias = delta_weight(dt_bias, vec_dtype, (size_t)h * dim + d);
+        const float* src = raw + ((size_t)t0 * heads + h) * dim + d;
+        float x[kDc], acc = 0.f;
+#pragma unroll
+        for (int i = 0; i < kDc; ++i) x[i] = i < n ? src[(size_t)i * heads * dim] : 0.f;
+#pragma unroll
+        for (int i = 0; i < kDc; ++i) {
+            if (i < n) acc = fmaf(rate, delta_softplus(x[i] + bias), acc);
+            sL[i * P + d] = acc;
+        }
+    }
+    if (threadIdx.x < kDc) sb[threadIdx.x] = threadIdx.x < n ? delta_sigmoid(proj[(size_t)(t0 + threadIdx.x) * proj_stride + channels + h]) : 0.f;
     for (int e = threadIdx.x; e < 2 * kDc * ap; e += 256) sA[e] = 0.f;              // A, then B
     __syncthreads();
-    for (int d = threadIdx.x; d < dim; d += 256) {
+#pragma unroll
+    for (int it = 0; it < kDc / 4; ++it) {    // unit vectors, a warp a row of q or k
+        float* row = (it & 1 ? sk : sq) + (warp + 8 * (it >> 1)) * P;
+        float4 x[2];
         float acc = 0.f;
 #pragma unroll
-        for (int i = 0; i < kDc; ++i) { acc += sL[i * P + d]; sL[i * P + d] = acc; }
+        for (int p = 0; p < 2; ++p) {
+            x[p] = 4 * lane + 128 * p < dim ? dc_ld4(row + 4 * lane + 128 * p) : make_float4(0.f, 0.f, 0.f, 0.f);
+            acc = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, fmaf(x[p].z, x[p].z, fmaf(x[p].w, x[p].w, acc))));
+        }
+        const float f = (it & 1 ? 1.0f : q_scale) / sqrtf(warp_sum(acc) + unit_eps);
+#pragma unroll
+        for (int p = 0; p < 2; ++p)
+            if (4 * lane + 128 * p < dim) dc_st4(row + 4 * lane + 128 * p, x[p].x * f, x[p].y * f, x[p].z * f, x[p].w * f);
     }
     __syncthreads();
     if (threadIdx.x < kDcTiles * kDcSlices) {
@@ -381,25 +422,33 @@ long mdma_delta_chunks_scratch(int n_rows, int n_seqs, int heads, int dim, int v
     return ((long)n_rows / kDc + n_seqs + 1) * heads * (long)DcLayout(dim, vdim).floats;
 }
 
-// q, k [rows][kv_heads * dim], v, out [rows][heads * vdim], lg [rows][heads * dim], beta [rows][heads], all floats
-int mdma_delta_chunks(const float* q, const float* k, const float* v, const float* lg, const float* beta, float* scratch,
+// proj rows [q | k | v | b | ..], raw [rows][heads * dim] the decays' inputs, out [rows][heads * vdim], all floats; the
+// convolutions' kept inputs are read, not brought up to date
+int mdma_delta_chunks(const float* proj, int proj_stride, const float* raw, const void* conv_w, int conv_dtype, int taps,
+                      const void* a_log, const void* dt_bias, int vec_dtype, const float* conv_state, float* scratch,
                       long scratch_floats, const int* seq_start, const int* seq_slot, float* state, long state_stride, float* out,
-                      int n_rows, int n_seqs, int max_new, int heads, int kv_heads, int dim, int vdim, cudaStream_t stream) {
+                      int n_rows, int n_seqs, int max_new, int heads, int kv_heads, int dim, int vdim, float unit_eps,
+                      float q_scale, cudaStream_t stream) {
     MDMA_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0, "delta_chunks: bad sizes");
     MDMA_REQUIRE(dim <= kDcMaxDim && dim % 4 == 0 && vdim % 4 == 0 && vdim <= 512, "delta_chunks: heads of %d x %d are not a geometry this kernel takes", dim, vdim);
-    MDMA_REQUIRE((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)lg | (uintptr_t)scratch) & 15) == 0, "delta_chunks: rows must start on 16 bytes");
+    MDMA_REQUIRE(taps >= 1 && taps <= kDeltaMaxTaps, "delta_chunks: %d taps, the kernel takes 1..%d", taps, kDeltaMaxTaps);
+    MDMA_REQUIRE(((uintptr_t)scratch & 15) == 0, "delta_chunks: scratch must start on 16 bytes");
     if (n_rows == 0 || n_seqs == 0) return 0;
     const long need = mdma_delta_chunks_scratch(n_rows, n_seqs, heads, dim, vdim);
     MDMA_REQUIRE(scratch_floats >= need, "delta_chunks: %ld floats of scratch needed, %ld given", need, scratch_floats);
     const int max_chunks = (max_new + kDc - 1) / kDc;
     MDMA_REQUIRE((long)n_seqs * max_chunks <= 2147483647l && heads <= 65535, "delta_chunks: too many rows");
-    static bool raised = false;
-    if (!raised) {
-        cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
-        raised = true;
-    }
-    launch_chained(delta_chunk_prepare_kernel, dim3((unsigned)(n_seqs * max_chunks), heads), dim3(256), dc_prepare_smem(dim, vdim), stream,
-                   q, k, v, lg, beta, scratch, seq_start, heads, kv_heads, dim, vdim, max_chunks);
+#define MDMA_DC_PREPARE(TAPS)                                                                                               \
+    do {                                                                                                                   \
+        static bool raised = false;                                                                                        \
+        if (!raised) { cudaFuncSetAttribute(delta_chunk_prepare_kernel<TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024); raised = true; } \
+        launch_chained(delta_chunk_prepare_kernel<TAPS>, dim3((unsigned)(n_seqs * max_chunks), heads), dim3(256),          \
+                       dc_prepare_smem(dim, vdim), stream, proj, proj_stride, raw, conv_w, conv_dtype, taps, a_log, dt_bias, \
+                       vec_dtype, conv_state, (size_t)state_stride, scratch, seq_start, seq_slot, heads, kv_heads, dim, vdim, \
+                       max_chunks, unit_eps, q_scale);                                                                     \
+    } while (0)
+    if (taps <= 4) MDMA_DC_PREPARE(4); else MDMA_DC_PREPARE(0);
+#undef MDMA_DC_PREPARE
     MDMA_LAUNCH_OK("delta_chunk_prepare");
     const DcLayout lay(dim, vdim);
     dim3 grid(n_seqs, heads, lay.slices);

@@ -848,25 +848,80 @@ def talking_attention(q, k_cache, v_cache, talk, sinks, ctx, page_table, max_pag
 
 
 # ---- the gated delta rule with a decay per key channel (csrc/delta_rule.cu) ---------------------------------------------
-def delta_prepare(proj, raw, conv_w, taps: int, a_log, dt_bias, ctx, conv_state, q, k, v, lg, beta, heads: int,
-                  kv_heads: int, dim: int, vdim: int, unit_eps: float, q_scale: float) -> None:
-    """From float projection rows [q | k | v | b] and the decays' inputs `raw` [T, heads * dim] to what enters the
-    recurrence, float rows: q, k [T, kv_heads * dim] unit vectors (q times `q_scale`), v [T, heads * vdim], the decays'
-    logarithms lg [T, heads * dim], the step sizes beta [T, heads].  `conv_state` [slots, (taps - 1) * channels], the
-    convolutions' last inputs, is read and brought up to date."""
-    _need_cuda(proj, raw, conv_w, a_log, dt_bias, conv_state, q, k, v, lg, beta)
+def _delta_inputs(proj, raw, conv_w, taps, a_log, dt_bias, heads, kv_heads, dim, vdim):
     channels = 2 * kv_heads * dim + heads * vdim
     assert proj.dtype == raw.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= channels + heads
     assert raw.is_contiguous() and raw.shape[1] == heads * dim and conv_w.is_contiguous() and tuple(conv_w.shape) == (channels, taps)
     assert a_log.numel() == heads and dt_bias.numel() == heads * dim
+    return (_ptr(proj), _i(proj.stride(0)), _ptr(raw), _ptr(conv_w), _i(dtype_code(conv_w.dtype)), _i(taps), _ptr(a_log),
+            _ptr(dt_bias), _i(_same_dtype(a_log, dt_bias)))
+
+
+def _kept(conv_state, taps: int, channels: int):
+    if taps == 1:
+        return _ptr(None), ctypes.c_long(0)
+    assert conv_state.shape[1] >= (taps - 1) * channels
+    return _state(conv_state)
+
+
+def delta_prepare(proj, raw, conv_w, taps: int, a_log, dt_bias, ctx, conv_state, q, k, v, lg, beta, heads: int,
+                  kv_heads: int, dim: int, vdim: int, unit_eps: float, q_scale: float) -> None:
+    """From float projection rows [q | k | v | b | ..] and the decays' inputs `raw` [T, heads * dim] to what enters the
+    recurrence, float rows: q, k [T, kv_heads * dim] unit vectors (q times `q_scale`), v [T, heads * vdim], the decays'
+    logarithms lg [T, heads * dim], the step sizes beta [T, heads].  `conv_state` [slots, (taps - 1) * channels]: the
+    convolutions' kept inputs, read only (`delta_conv_keep` brings them up to date)."""
+    _need_cuda(proj, raw, conv_w, a_log, dt_bias, conv_state, q, k, v, lg, beta)
     for t, c in ((q, kv_heads * dim), (k, kv_heads * dim), (v, heads * vdim), (lg, heads * dim), (beta, heads)):
         assert t.dtype == torch.float32 and t.is_contiguous() and t.shape[1] == c and t.shape[0] >= ctx.n_tokens
-    sp, ss = _state(conv_state) if taps > 1 else (_ptr(None), ctypes.c_long(0))
-    assert taps == 1 or conv_state.shape[1] >= (taps - 1) * channels
-    _call("core", "mdma_delta_prepare", _ptr(proj), _i(proj.stride(0)), _ptr(raw), _ptr(conv_w), _i(dtype_code(conv_w.dtype)),
-          _i(taps), _ptr(a_log), _ptr(dt_bias), _i(_same_dtype(a_log, dt_bias)), _ptr(ctx.tok_seq), _ptr(ctx.seq_start),
-          _ptr(ctx.seq_slot), sp, ss, _ptr(q), _ptr(k), _ptr(v), _ptr(lg), _ptr(beta), _i(ctx.n_tokens), _i(ctx.n_seqs),
-          _i(heads), _i(kv_heads), _i(dim), _i(vdim), _f(unit_eps), _f(q_scale), _stream(), launches=2 if taps > 1 else 1)
+    sp, ss = _kept(conv_state, taps, 2 * kv_heads * dim + heads * vdim)
+    _call("core", "mdma_delta_prepare", *_delta_inputs(proj, raw, conv_w, taps, a_log, dt_bias, heads, kv_heads, dim, vdim),
+          _ptr(ctx.tok_seq), _ptr(ctx.seq_start), _ptr(ctx.seq_slot), sp, ss, _ptr(q), _ptr(k), _ptr(v), _ptr(lg), _ptr(beta),
+          _i(ctx.n_tokens), _i(heads), _i(kv_heads), _i(dim), _i(vdim), _f(unit_eps), _f(q_scale), _stream())
+
+
+def delta_conv_keep(proj, taps: int, channels: int, ctx, conv_state) -> None:
+    """conv_state[slot] = the last taps - 1 rows of columns [0, channels) each sequence has brought so far."""
+    if taps == 1:
+        return
+    _need_cuda(proj, conv_state)
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= channels
+    sp, ss = _kept(conv_state, taps, channels)
+    _call("core", "mdma_delta_conv_keep", _ptr(proj), _i(proj.stride(0)), _i(taps), _i(channels), _ptr(ctx.seq_start),
+          _ptr(ctx.seq_slot), sp, ss, _i(ctx.n_seqs), _stream())
+
+
+def delta_inner(proj, col: int, decay_rank: int, gate_rank: int, a, g, n_rows: int) -> None:
+    """a, g (bfloat16) = columns [col, col + decay_rank) and the gate_rank after them of float rows."""
+    _need_cuda(proj, a, g)
+    assert proj.dtype == torch.float32 and a.dtype == g.dtype == torch.bfloat16 and a.stride(1) == g.stride(1) == 1
+    assert a.shape[1] >= decay_rank and g.shape[1] >= gate_rank and proj.shape[1] >= col + decay_rank + gate_rank
+    _call("core", "mdma_delta_inner", _ptr(proj), _i(proj.stride(0)), _i(col), _i(decay_rank), _i(gate_rank), _ptr(a),
+          _i(a.stride(0)), _ptr(g), _i(g.stride(0)), _i(n_rows), _stream())
+
+
+def delta_token_fits(heads: int, kv_heads: int, dim: int, vdim: int, decay_rank: int, gate_rank: int, taps: int) -> bool:
+    lib = _build._loaded.get("core") or _build.load("core")
+    return bool(lib.mdma_delta_token_fits(_i(heads), _i(kv_heads), _i(dim), _i(vdim), _i(decay_rank), _i(gate_rank), _i(taps)))
+
+
+def delta_token(proj, a2, g2, conv_w, taps: int, a_log, dt_bias, norm_w, ctx, state, conv_at: int, out, heads: int, dim: int,
+                vdim: int, unit_eps: float, q_scale: float, eps: float, partial=None, splits: int = 0, split_stride: int = 0) -> None:
+    """Single tokens of the serving engine, from the projection rows [q | k | v | b | a | g] (or with `partial` the sums of a
+    K-split product's partial rows) to the gated, normed heads `out` (bfloat16), state and kept inputs brought up to date."""
+    _need_cuda(proj, a2, g2, conv_w, a_log, dt_bias, norm_w, state, out, partial)
+    channels, decay_rank, gate_rank = heads * (2 * dim + vdim), a2.shape[1], g2.shape[1]
+    row_width = channels + heads + decay_rank + gate_rank
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] == row_width
+    for t in (a2, g2, conv_w, out):
+        assert t.dtype == torch.bfloat16 and t.is_contiguous()
+    assert a2.shape[0] == heads * dim and g2.shape[0] == heads * vdim and tuple(conv_w.shape) == (channels, taps)
+    assert out.shape[1] == heads * vdim and norm_w.numel() == vdim and a_log.numel() == heads and dt_bias.numel() == heads * dim
+    sp, ss = _state(state)
+    assert state.shape[1] >= conv_at + (taps - 1) * channels and conv_at >= heads * dim * vdim and ctx.max_new == 1
+    _call("core", "mdma_delta_token", _ptr(proj), _i(proj.stride(0)), _ptr(partial), _i(splits if partial is not None else 0),
+          ctypes.c_long(split_stride), _i(row_width), _ptr(a2), _ptr(g2), _i(decay_rank), _i(gate_rank), _ptr(conv_w), _i(taps),
+          _ptr(a_log), _ptr(dt_bias), _ptr(norm_w), _i(_same_dtype(a_log, dt_bias, norm_w)), _ptr(ctx.seq_slot), sp, ss,
+          _i(conv_at), _ptr(out), _i(ctx.n_seqs), _i(heads), _i(dim), _i(vdim), _f(unit_eps), _f(q_scale), _f(eps), _stream())
 
 
 def delta_scan(q, k, v, lg, beta, ctx, state, out, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
@@ -888,18 +943,20 @@ def delta_chunk_floats(heads: int, dim: int, vdim: int) -> int:
     return heads * (16 * (3 * padded + 44) + padded + -(-vdim // 16) * 320)
 
 
-def delta_chunks(q, k, v, lg, beta, scratch, ctx, state, out, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
-    """`delta_scan` a chunk of sixteen rows at a time (equal up to rounding; dim and vdim multiples of four).  `scratch`:
-    (T // 16 + sequences + 1) * `delta_chunk_floats` floats."""
-    _need_cuda(q, k, v, lg, beta, scratch, state, out)
-    for t, c in ((q, kv_heads * dim), (k, kv_heads * dim), (v, heads * vdim), (lg, heads * dim), (beta, heads), (out, heads * vdim)):
-        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape[1] == c and t.shape[0] >= ctx.n_tokens
+def delta_chunks(proj, raw, conv_w, taps: int, a_log, dt_bias, conv_state, scratch, ctx, state, out, heads: int, kv_heads: int,
+                 dim: int, vdim: int, unit_eps: float, q_scale: float) -> None:
+    """`delta_prepare` and `delta_scan` a chunk of sixteen rows at a time (equal up to rounding; dim and vdim multiples of
+    four).  `scratch`: (T // 16 + sequences + 1) * `delta_chunk_floats` floats."""
+    _need_cuda(proj, raw, conv_w, a_log, dt_bias, conv_state, scratch, state, out)
+    assert out.dtype == torch.float32 and out.is_contiguous() and out.shape[1] == heads * vdim and out.shape[0] >= ctx.n_tokens
     assert scratch.dtype == torch.float32 and scratch.is_contiguous()
+    kept, stride = _kept(conv_state, taps, 2 * kv_heads * dim + heads * vdim)
     sp, ss = _state(state)
-    assert state.shape[1] >= heads * dim * vdim
-    _call("core", "mdma_delta_chunks", _ptr(q), _ptr(k), _ptr(v), _ptr(lg), _ptr(beta), _ptr(scratch), ctypes.c_long(scratch.numel()),
-          _ptr(ctx.seq_start), _ptr(ctx.seq_slot), sp, ss, _ptr(out), _i(ctx.n_tokens), _i(ctx.n_seqs), _i(ctx.max_new),
-          _i(heads), _i(kv_heads), _i(dim), _i(vdim), _stream(), launches=2)
+    assert state.shape[1] >= heads * dim * vdim and (taps == 1 or stride.value == ss.value)
+    _call("core", "mdma_delta_chunks", *_delta_inputs(proj, raw, conv_w, taps, a_log, dt_bias, heads, kv_heads, dim, vdim), kept,
+          _ptr(scratch), ctypes.c_long(scratch.numel()), _ptr(ctx.seq_start), _ptr(ctx.seq_slot), sp, ss, _ptr(out),
+          _i(ctx.n_tokens), _i(ctx.n_seqs), _i(ctx.max_new), _i(heads), _i(kv_heads), _i(dim), _i(vdim), _f(unit_eps),
+          _f(q_scale), _stream(), launches=2)
 
 
 def gated_head_rmsnorm(o: torch.Tensor, gate: torch.Tensor, w: Optional[torch.Tensor], out: torch.Tensor, n_rows: int,

@@ -157,15 +157,16 @@ def flush_pending(device: torch.device, st: Optional[TensorState] = None) -> Non
           _i(pend.cols), _ptr(out), _i(out.stride(0)), _i(int(out.dtype == torch.float32)), _stream())
 
 
-def take_pending(target: torch.Tensor, mode: int, rows: int, st: Optional[TensorState] = None):
+def take_pending(target: torch.Tensor, mode: int, rows: int, st: Optional[TensorState] = None, any_pitch: bool = False):
     """If partial sums for exactly this target wait in the scratch, hand them to the caller, who
-    will add them up itself: returns (scratch, splits, floats per split) or None."""
+    will add them up itself: returns (scratch, splits, floats per split) or None.  `any_pitch`: the caller
+    reads the partial rows by their own width, whatever the pitch of the target's rows."""
     st = st or _default.get(target.device.index)
     if st is None or st.pending is None:
         return None
     pend = st.pending
     if (pend.target_ptr != target.data_ptr() or pend.mode != mode or pend.rows != rows
-            or pend.cols != target.shape[1] or target.stride(0) != pend.cols):
+            or pend.cols != target.shape[1] or (target.stride(0) != pend.cols and not any_pitch)):
         return None
     st.pending = None
     return st.scratch, pend.splits, pend.rows * pend.cols

@@ -12,9 +12,10 @@ Each head's o is divided by its root mean square, multiplied by the weight `norm
 sigmoid(g2 g1 h), and the heads side by side go through Wo.
 
 State per sequence: S (floats) and the convolutions' last taps-1 inputs.  Everything that enters the recurrence is float
-in both engines (the projections write float rows); the inner rows of the two low-rank projections are in the compute
-dtype.  The 32-bit engine and short portions walk row by row in one fixed order; the serving engine walks portions of
-`CHUNKS_FROM` rows or more a chunk of rows at a time (csrc/delta_chunk.cu).
+in both engines (the projections write float rows); the inner rows of the two low-rank projections go into their second products in
+the compute dtype.  The 32-bit engine and short portions walk row by row in one fixed order; the serving engine walks portions of
+`CHUNKS_FROM` rows or more a chunk of rows at a time (csrc/delta_chunk.cu), and its single tokens take one kernel from
+the projection to the gated norm where its sizes fit (one q/k head per head).
 """
 from __future__ import annotations
 
@@ -48,11 +49,10 @@ class ChannelDelta(Part):
             raise ValueError(f"{self.heads} heads do not divide over {self.kv_heads} kv heads")
         self.qk_width, self.k_width, self.v_width = self.kv_heads * self.dim, self.heads * self.dim, self.heads * self.v_dim
         self.channels = 2 * self.qk_width + self.v_width            # what the convolutions see
-        self.row_width = self.channels + self.heads
+        # a projection row: q, k, v, the step sizes' logits, the inner rows of the decays and of the gate
+        self.inner_col = self.channels + self.heads
+        self.row_width = self.inner_col + self.decay_rank + self.gate_rank
         self.row_pitch = -(-self.row_width // 8) * 8
-        # the two inner rows lie side by side when the second then starts on a 16-byte boundary
-        self.inner_fused = self.decay_rank % 8 == 0
-        self.inner_width = self.decay_rank + self.gate_rank
         self.state_floats = self.heads * self.dim * self.v_dim
         self.conv_at = -(-self.state_floats // 4) * 4
         self.chunks_fit = self.dim % 4 == 0 and self.v_dim % 4 == 0 and self.v_dim <= 512
@@ -77,10 +77,7 @@ class ChannelDelta(Part):
                 "o": TensorSpec((W, self.v_width))}
 
     def fused_tensors(self):
-        fused = {"qkvb": ("q", "k", "v", "b"), "conv": ("q.conv", "k.conv", "v.conv")}
-        if self.inner_fused:
-            fused["a1g1"] = ("a1", "g1")
-        return fused
+        return {"qkvbag": ("q", "k", "v", "b", "a1", "g1"), "conv": ("q.conv", "k.conv", "v.conv")}
 
     def kv_need(self):
         return None
@@ -100,11 +97,8 @@ class ChannelDelta(Part):
               n["out"]: (self.v_width, "act")}
         if self.chunks_fit:
             ws[n["chunks"]] = (self._chunk_columns(), "f32")
-        if self.inner_fused:
-            ws[f"delta_inner_{self.inner_width}"] = (-(-self.inner_width // 8) * 8, "act")
-        else:
-            ws[f"delta_a1_{self.decay_rank}"] = (-(-self.decay_rank // 8) * 8, "act")
-            ws[f"delta_g1_{self.gate_rank}"] = (-(-self.gate_rank // 8) * 8, "act")
+        ws[f"delta_a1_{self.decay_rank}"] = (-(-self.decay_rank // 8) * 8, "act")
+        ws[f"delta_g1_{self.gate_rank}"] = (-(-self.gate_rank // 8) * 8, "act")
         return ws
 
     def _chunk_columns(self) -> int:
@@ -117,27 +111,23 @@ class ChannelDelta(Part):
         def whole(name, pieces):
             t = tensors.get(name)
             return t if t is not None else torch.cat([tensors[n] for n in pieces], dim=0).contiguous()
-        self.proj = Linear(whole("qkvb", ("q", "k", "v", "b")), rt)
+        self.proj = Linear(whole("qkvbag", ("q", "k", "v", "b", "a1", "g1")), rt)
         self.conv = whole("conv", ("q.conv", "k.conv", "v.conv"))
-        if self.inner_fused:
-            self.inner = Linear(whole("a1g1", ("a1", "g1")), rt)
-        else:
-            self.a1, self.g1 = Linear(tensors["a1"], rt), Linear(tensors["g1"], rt)
         self.a2, self.g2, self.o = Linear(tensors["a2"], rt), Linear(tensors["g2"], rt), Linear(tensors["o"], rt)
         self.a_log, self.dt_bias, self.norm = tensors["A_log"], tensors["dt_bias"], tensors["norm"]
+        self._token_ok = (rt.dtype != torch.float32 and self.conv.dtype == torch.bfloat16
+                          and self.a_log.dtype == self.dt_bias.dtype == self.norm.dtype
+                          and ops.delta_token_fits(self.heads, self.kv_heads, self.dim, self.v_dim, self.decay_rank, self.gate_rank, self.taps))
 
-    def _low_rank(self, ctx, h, raw, gate):
+    def _low_rank(self, ctx, proj, raw, gate):
         """raw = a2 a1 h (float rows), gate = g2 g1 h."""
-        n = ctx.n_tokens
-        if self.inner_fused:
-            inner = ctx.buf(f"delta_inner_{self.inner_width}", -(-self.inner_width // 8) * 8)
-            self.inner.store(h, inner[:, :self.inner_width], n)
-            a, g = inner[:, :self.decay_rank], inner[:, self.decay_rank:self.inner_width]
+        n, c = ctx.n_tokens, self.inner_col
+        if proj.dtype == gate.dtype:
+            a, g = proj[:, c:c + self.decay_rank], proj[:, c + self.decay_rank:self.row_width]
         else:
             a = ctx.buf(f"delta_a1_{self.decay_rank}", -(-self.decay_rank // 8) * 8)[:, :self.decay_rank]
             g = ctx.buf(f"delta_g1_{self.gate_rank}", -(-self.gate_rank // 8) * 8)[:, :self.gate_rank]
-            self.a1.store(h, a, n)
-            self.g1.store(h, g, n)
+            ops.delta_inner(proj, c, self.decay_rank, self.gate_rank, a, g, n)
         self.a2.store(a, raw, n)
         self.g2.store(g, gate, n)
 
@@ -145,18 +135,32 @@ class ChannelDelta(Part):
         n = ctx.n_tokens
         names = self._names()
         f32 = torch.float32
-        proj = ctx.buf(names["proj"], self.row_pitch, f32)
-        raw, gate = ctx.buf(names["raw"], self.k_width, f32), ctx.buf(names["gate"], self.v_width)
-        q, k = ctx.buf(names["q"], self.qk_width, f32), ctx.buf(names["k"], self.qk_width, f32)
-        v, lg = ctx.buf(names["v"], self.v_width, f32), ctx.buf(names["lg"], self.k_width, f32)
-        beta, sums = ctx.buf(names["beta"], self.heads, f32), ctx.buf(names["sum"], self.v_width, f32)
+        proj = ctx.buf(names["proj"], self.row_pitch, f32)[:, :self.row_width]
         out = ctx.buf(names["out"], self.v_width)
         state = view.state[:, :self.state_floats]
         conv_state = view.state[:, self.conv_at:self.conv_at + self.conv_floats] if self.taps > 1 else None
-        self.proj.store(h, proj[:, :self.row_width], n)
-        self._low_rank(ctx, h, raw, gate)
-        ops.delta_prepare(proj, raw, self.conv, self.taps, self.a_log, self.dt_bias, ctx, conv_state, q, k, v, lg, beta,
-                          self.heads, self.kv_heads, self.dim, self.v_dim, self.unit_eps, self.dim ** -0.5)
+        q_scale = self.dim ** -0.5
+        single = ctx.max_new == 1 and self._token_ok
+        self.proj.store(h, proj, n, defer=single)
+        if single:
+            partial, splits, stride = None, 0, 0
+            if self.rt.gemm == "tensor":
+                from .. import ops_tensor
+                pend = ops_tensor.take_pending(proj, ops.GEMM_STORE, n, self.rt.tc, any_pitch=True)
+                if pend is not None:
+                    partial, splits, stride = pend
+                else:
+                    ops_tensor.flush_pending(proj.device, self.rt.tc)
+            ops.delta_token(proj, self.a2.w, self.g2.w, self.conv, self.taps, self.a_log, self.dt_bias, self.norm, ctx, view.state,
+                            self.conv_at, out, self.heads, self.dim, self.v_dim, self.unit_eps, q_scale, self.eps, partial, splits,
+                            stride)
+            return out
+        raw, gate = ctx.buf(names["raw"], self.k_width, f32), ctx.buf(names["gate"], self.v_width)
+        sums = ctx.buf(names["sum"], self.v_width, f32)
+        self._low_rank(ctx, proj, raw, gate)
+        if self.rt.gemm == "tensor":
+            from .. import ops_tensor
+            ops_tensor.flush_pending(proj.device, self.rt.tc)
         chunks = None
         if self.chunks_fit and self.rt.dtype != f32 and ctx.max_new >= self.CHUNKS_FROM:
             # (room for them all, unless very many short sequences come with a long one)
@@ -164,9 +168,16 @@ class ChannelDelta(Part):
             if (n // 16 + ctx.n_seqs + 1) * ops.delta_chunk_floats(self.heads, self.dim, self.v_dim) > chunks.numel():
                 chunks = None
         if chunks is not None:
-            ops.delta_chunks(q, k, v, lg, beta, chunks, ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
+            ops.delta_chunks(proj, raw, self.conv, self.taps, self.a_log, self.dt_bias, conv_state, chunks, ctx, state, sums,
+                             self.heads, self.kv_heads, self.dim, self.v_dim, self.unit_eps, q_scale)
         else:
+            q, k = ctx.buf(names["q"], self.qk_width, f32), ctx.buf(names["k"], self.qk_width, f32)
+            v, lg = ctx.buf(names["v"], self.v_width, f32), ctx.buf(names["lg"], self.k_width, f32)
+            beta = ctx.buf(names["beta"], self.heads, f32)
+            ops.delta_prepare(proj, raw, self.conv, self.taps, self.a_log, self.dt_bias, ctx, conv_state, q, k, v, lg, beta,
+                              self.heads, self.kv_heads, self.dim, self.v_dim, self.unit_eps, q_scale)
             ops.delta_scan(q, k, v, lg, beta, ctx, state, sums, self.heads, self.kv_heads, self.dim, self.v_dim)
+        ops.delta_conv_keep(proj, self.taps, self.channels, ctx, conv_state)
         ops.gated_head_rmsnorm(sums, gate, self.norm, out, n, self.heads, self.v_dim, self.eps)
         return out
 
@@ -177,5 +188,4 @@ class ChannelDelta(Part):
         self.o.store(self._run(ctx, h, view), out, ctx.n_tokens, defer=defer)
 
     def resident_tensors(self):
-        ts = [self.proj.w, self.conv, self.a2.w, self.g2.w, self.o.w, self.a_log, self.dt_bias, self.norm]
-        return ts + ([self.inner.w] if self.inner_fused else [self.a1.w, self.g1.w])
+        return [self.proj.w, self.conv, self.a2.w, self.g2.w, self.o.w, self.a_log, self.dt_bias, self.norm]
