@@ -48,9 +48,14 @@ __device__ __forceinline__ uint32_t mw_pack(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<uint32_t*>(&v);
 }
+__device__ __forceinline__ float mw_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 // a raw dot product as a score in powers of two: `a` = cap log2(e) and `b` = 2 log2(e) factor / cap, or b = log2(e) factor
 __device__ __forceinline__ float mw_score(float x, bool capped, float a, float b) {
-    return capped ? a - __fdividef(2.0f * a, 1.0f + exp2f(x * b)) : x * b;
+    return capped ? fmaf(-2.0f * a, __fdividef(1.0f, 1.0f + mw_exp2(x * b)), a) : x * b;
 }
 
 struct MwCache {
@@ -61,19 +66,21 @@ struct MwCache {
     __device__ __forceinline__ size_t row(int p) const { return (size_t)pages[p / page_size] * page_size + (size_t)(p % page_size); }
 };
 
-static size_t mw_rows_smem(int dim, int cols) {
-    return ((size_t)kMwWarps * kMwTile * (dim + 8) + 2 * (size_t)kMwChunk * ((dim + 8) + (cols + 8))) * 2;
+static size_t mw_rows_smem(int dim, int vt) {
+    return ((size_t)kMwWarps * kMwTile * (dim + 8) + 2 * (size_t)kMwChunk * ((dim + 8) + (8 * vt + 8))) * 2;
 }
 
 // VT: value n-tiles of eight columns a warp accumulates.
-template <int VT>
+// KD: the head size over sixteen where it is known at compile time, else 0.
+template <int VT, int KD>
 __global__ void __launch_bounds__(kMwWarps * 32, 2)
 mixed_rows_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const __nv_bfloat16* __restrict__ k_cache,
                   const __nv_bfloat16* __restrict__ v_cache, const float* __restrict__ factor, float softcap,
                   const int* __restrict__ seq_start, const int* __restrict__ seq_pos0, const int* __restrict__ seq_slot,
                   const int* __restrict__ page_table, int max_pages, int page_size, float* __restrict__ sums, int n_heads,
-                  int n_kv_heads, int dim, int v_dim, int window, int keep_first, int heads_per_block, int cols,
+                  int n_kv_heads, int dim_, int v_dim, int window, int keep_first, int heads_per_block, int cols,
                   int slab0, int slab1) {
+    const int dim = KD > 0 ? 16 * KD : dim_;
     chain_release();
     chain_wait();
     extern __shared__ __align__(16) unsigned char mw_smem[];
@@ -97,10 +104,11 @@ mixed_rows_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const _
     const int first = window > 0 ? max(0, pos_b + 1 - window) : 0;
     const int kept = min(keep_first, first), gap = first - kept, n_keys = last + 1 - gap;
     const MwCache cache = {k_cache, v_cache, page_table + (size_t)seq_slot[s] * max_pages, page_size, n_kv_heads, dim, v_dim};
-    const int qp = dim + 8, vp = cols + 8;
+    constexpr int vp = VT * 8 + 8;
+    const int qp = dim + 8;
     __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(mw_smem) + (size_t)warp * kMwTile * qp;
     __nv_bfloat16* sk = reinterpret_cast<__nv_bfloat16*>(mw_smem) + (size_t)kMwWarps * kMwTile * qp;      // [2][32][dim + 8]
-    __nv_bfloat16* sv = sk + 2 * (size_t)kMwChunk * qp;                                                    // [2][32][cols + 8]
+    __nv_bfloat16* sv = sk + 2 * (size_t)kMwChunk * qp;                                                    // [2][32][8 VT + 8]
     const uint4 zero4 = make_uint4(0, 0, 0, 0);
     for (int e = lane; e < kMwTile * (dim / 8); e += 32) {
         const int r = e / (dim / 8), d8 = e % (dim / 8);
@@ -126,6 +134,9 @@ mixed_rows_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const _
         }
         mw_commit();
     };
+    // columns beyond the block's: zero, and computed along with the others
+    for (int e = threadIdx.x; e < 2 * kMwChunk * (VT - cw / 8); e += kMwWarps * 32)
+        *reinterpret_cast<uint4*>(sv + (size_t)(e / (VT - cw / 8)) * vp + cw + (e % (VT - cw / 8)) * 8) = zero4;
     float o[VT][4];
 #pragma unroll
     for (int n = 0; n < VT; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
@@ -150,7 +161,7 @@ mixed_rows_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const _
             float sc[4][4];
 #pragma unroll
             for (int n = 0; n < 4; ++n) { sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f; }
-#pragma unroll 4
+#pragma unroll(KD > 0 ? KD : 4)
             for (int k0 = 0; k0 < dim; k0 += 16) {
                 uint32_t a0, a1, a2, a3;
                 mw_ldmatrix_x4(sq_addr + (uint32_t)(((lane & 15) * qp + k0 + (lane >> 4) * 8) * 2), a0, a1, a2, a3);
@@ -189,14 +200,14 @@ mixed_rows_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const _
             const float n_lo = fmaxf(m_lo, c_lo), n_hi = fmaxf(m_hi, c_hi);
             // a row that has seen no key yet keeps its zero sums (2^(-inf - -inf) is avoided)
             const float z_lo = n_lo == -INFINITY ? 0.f : n_lo, z_hi = n_hi == -INFINITY ? 0.f : n_hi;
-            const float f_lo = exp2f(m_lo - z_lo), f_hi = exp2f(m_hi - z_hi);
+            const float f_lo = mw_exp2(m_lo - z_lo), f_hi = mw_exp2(m_hi - z_hi);
             float s_lo = 0.f, s_hi = 0.f;
 #pragma unroll
             for (int n = 0; n < 4; ++n) {
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
-                    sc[n][i] = exp2f(sc[n][i] - z_lo);
-                    sc[n][2 + i] = exp2f(sc[n][2 + i] - z_hi);
+                    sc[n][i] = mw_exp2(sc[n][i] - z_lo);
+                    sc[n][2 + i] = mw_exp2(sc[n][2 + i] - z_hi);
                     s_lo += sc[n][i];
                     s_hi += sc[n][2 + i];
                 }
@@ -217,12 +228,10 @@ mixed_rows_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const _
                 const uint32_t v_addr = sv_addr + (uint32_t)((vrow * vp + (lane >> 4) * 8) * 2);
 #pragma unroll
                 for (int n2 = 0; n2 < VT / 2; ++n2) {
-                    if (n2 * 16 < cw) {
-                        uint32_t b0_, b1_, b2_, b3_;
-                        mw_ldmatrix_x4_trans(v_addr + n2 * 32, b0_, b1_, b2_, b3_);
-                        mw_mma(o[n2 * 2], a0, a1, a2, a3, b0_, b1_);
-                        mw_mma(o[n2 * 2 + 1], a0, a1, a2, a3, b2_, b3_);
-                    }
+                    uint32_t b0_, b1_, b2_, b3_;
+                    mw_ldmatrix_x4_trans(v_addr + n2 * 32, b0_, b1_, b2_, b3_);
+                    mw_mma(o[n2 * 2], a0, a1, a2, a3, b0_, b1_);
+                    mw_mma(o[n2 * 2 + 1], a0, a1, a2, a3, b2_, b3_);
                 }
             }
         }
@@ -383,7 +392,7 @@ mixed_step_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const _
         for (int h = warp; h < n_heads; h += kMwStepWarps) {
             const float x = ss[h * (kMwChunk + 1) + lane];                   // a chunk has at least one key
             const float m_old = sm[h], m_new = fmaxf(m_old, warp_max(x));
-            const float p = exp2f(x - m_new), corr = exp2f(m_old - m_new), sum = warp_sum(p);
+            const float p = mw_exp2(x - m_new), corr = mw_exp2(m_old - m_new), sum = warp_sum(p);
             sp[h * pp + lane] = __float2bfloat16_rn(p);
             if (lane == 0) { sm[h] = m_new; sl[h] = sl[h] * corr + sum; scorr[h] = corr; }
         }
@@ -403,16 +412,14 @@ mixed_step_kernel(const __nv_bfloat16* __restrict__ q, int q_row_stride, const _
             for (int m = 0; m < MT; ++m)
                 mw_ldmatrix_x4(sp_addr + (uint32_t)(((m * 16 + (lane & 15)) * pp + j * 16 + (lane >> 4) * 8) * 2), a[m][0], a[m][1], a[m][2], a[m][3]);
 #pragma unroll
-            for (int n2 = 0; n2 < NT / 2; ++n2) {
-                if (n2 < n_pairs) {
-                    uint32_t b0, b1, b2, b3;
-                    const int vrow = j * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
-                    mw_ldmatrix_x4_trans(sv_addr + (uint32_t)((vrow * vp + (pair0 + n2) * 16 + (lane >> 4) * 8) * 2), b0, b1, b2, b3);
+            for (int n2 = 0; n2 < NT / 2; ++n2) {      // (a pair beyond the warp's computes the last one again, for nothing)
+                uint32_t b0, b1, b2, b3;
+                const int vrow = j * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
+                mw_ldmatrix_x4_trans(sv_addr + (uint32_t)((vrow * vp + min(pair0 + n2, pairs - 1) * 16 + (lane >> 4) * 8) * 2), b0, b1, b2, b3);
 #pragma unroll
-                    for (int m = 0; m < MT; ++m) {
-                        mw_mma(o[m][n2 * 2], a[m][0], a[m][1], a[m][2], a[m][3], b0, b1);
-                        mw_mma(o[m][n2 * 2 + 1], a[m][0], a[m][1], a[m][2], a[m][3], b2, b3);
-                    }
+                for (int m = 0; m < MT; ++m) {
+                    mw_mma(o[m][n2 * 2], a[m][0], a[m][1], a[m][2], a[m][3], b0, b1);
+                    mw_mma(o[m][n2 * 2 + 1], a[m][0], a[m][1], a[m][2], a[m][3], b2, b3);
                 }
             }
         }
@@ -458,7 +465,7 @@ mixed_merge_kernel(const float* __restrict__ partial, const float* __restrict__ 
         const float* stat = src + (size_t)n_heads * total + h;
         const float m0 = k0 < splits ? stat[k0 * pitch] : -INFINITY, m1 = k1 < splits ? stat[k1 * pitch] : -INFINITY;
         const float l0 = k0 < splits ? stat[k0 * pitch + n_heads] : 0.f, l1 = k1 < splits ? stat[k1 * pitch + n_heads] : 0.f;
-        const float M = warp_max(fmaxf(m0, m1)), e0 = exp2f(m0 - M), e1 = exp2f(m1 - M);          // 0 for a run without keys
+        const float M = warp_max(fmaxf(m0, m1)), e0 = mw_exp2(m0 - M), e1 = mw_exp2(m1 - M);          // 0 for a run without keys
         const float inv = 1.0f / warp_sum(fmaf(l0, e0, l1 * e1));
         if (k0 < splits) fac[k0 * n_heads + h] = e0 * inv;
         if (k1 < splits) fac[k1 * n_heads + h] = e1 * inv;
@@ -473,9 +480,10 @@ mixed_merge_kernel(const float* __restrict__ partial, const float* __restrict__ 
 #pragma unroll
         for (int j = 0; j < GROUP; ++j) acc[j] = 0.f;
         if (live)
+#pragma unroll 2
             for (int g = part; g < n_heads; g += kMergeParts) {
                 float x = 0.f;
-#pragma unroll 8
+#pragma unroll 16
                 for (int k = 0; k < splits; ++k) x = fmaf(src[k * pitch + (size_t)g * total + col], fac[k * n_heads + g], x);
 #pragma unroll
                 for (int j = 0; j < GROUP; ++j) acc[j] = fmaf(mix[(size_t)(c * group + g0 + j) * n_heads + g], x, acc[j]);
@@ -523,24 +531,24 @@ int mdma_mixed_weights_rows(const void* q, int q_row_stride, const void* k_cache
     const int block_rows = kMwWarps / heads_per_block * kMwTile;
     const int parts = (total + 255) / 256;
     const int cols = ((total + parts - 1) / parts + 15) / 16 * 16;
-    const size_t smem = mw_rows_smem(dim, cols);
     const int gp = mw_group_part(group);
     for (int slab0 = 0; slab0 < n_tokens; slab0 += slab_tokens) {
         const int slab1 = slab0 + slab_tokens < n_tokens ? slab0 + slab_tokens : n_tokens;
         const int most = max_new < slab1 - slab0 ? max_new : slab1 - slab0;
         dim3 grid((most + block_rows - 1) / block_rows, (n_heads / heads_per_block) * parts, n_seqs);
-#define MDMA_MW_ROWS(VT)                                                                                                     \
+#define MDMA_MW_ROWS(VT, KD)                                                                                                 \
     do {                                                                                                                     \
         static bool raised = false;                                                                                          \
-        if (!raised) { cudaFuncSetAttribute(mixed_rows_kernel<VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMwSmemLimit); raised = true; } \
-        launch_chained(mixed_rows_kernel<VT>, grid, dim3(kMwWarps * 32), smem, stream, (const __nv_bfloat16*)q, q_row_stride, \
-                       (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, factor, softcap, seq_start, seq_pos0,   \
-                       seq_slot, page_table, max_pages, page_size, sums, n_heads, n_kv_heads, dim, v_dim, window, keep_first, \
-                       heads_per_block, cols, slab0, slab1);                                                                 \
+        if (!raised) { cudaFuncSetAttribute(mixed_rows_kernel<VT, KD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMwSmemLimit); raised = true; } \
+        launch_chained(mixed_rows_kernel<VT, KD>, grid, dim3(kMwWarps * 32), mw_rows_smem(dim, VT), stream, (const __nv_bfloat16*)q, \
+                       q_row_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, factor, softcap, seq_start, \
+                       seq_pos0, seq_slot, page_table, max_pages, page_size, sums, n_heads, n_kv_heads, dim, v_dim, window,  \
+                       keep_first, heads_per_block, cols, slab0, slab1);                                                     \
     } while (0)
-        if (cols <= 64) MDMA_MW_ROWS(8);
-        else if (cols <= 128) MDMA_MW_ROWS(16);
-        else MDMA_MW_ROWS(32);
+        if (cols <= 64) MDMA_MW_ROWS(8, 0);
+        else if (cols <= 128) MDMA_MW_ROWS(16, 0);
+        else if (dim == 128) MDMA_MW_ROWS(32, 8);
+        else MDMA_MW_ROWS(32, 0);
 #undef MDMA_MW_ROWS
         MDMA_LAUNCH_OK("mixed_weights_rows");
         const long items = (long)(slab1 - slab0) * total;
