@@ -1,0 +1,130 @@
+"""The Degavik architecture against its plain statement (tests/plain_degavik.py): every mechanism alone through its
+kernels, then whole models through the engine's step function, the cache manager, the scheduler and the generation
+loop.  Configurations and weights are made here (tests/degavik_tiny.py)."""
+import json
+import os
+
+import numpy as np
+import pytest
+import torch
+
+import plain_degavik as pd
+from degavik_tiny import CONFIGS, attention, config, delta, dense, make_model, make_tensors, moe, retention, with_ranks
+
+# float32: absolute, against the float64 statement.  bfloat16: the largest error as a share of the deviation of the
+# reference logits, and a row's root-mean-square error as a share of the row's own deviation.
+TOL_F32 = 5e-5
+TOL_BF16, TOL_ROW_BF16 = 0.12, 0.04
+CLOSE_CALL = 0.15        # a bfloat16 row behind a routing choice closer than this may take another expert
+
+
+def ids_of(cfg, n, seed):
+    g = torch.Generator().manual_seed(seed)
+    return torch.randint(0, cfg["vocab"], (n,), generator=g).tolist()
+
+
+def close(got, ref, dtype, what="", calm=None):
+    """Logits [rows, vocab] against the statement's.  `calm` [rows] of bool: rows that no close routing choice precedes;
+    the others are only asked to be finite in bfloat16."""
+    got, ref = np.atleast_2d(np.asarray(got, dtype=np.float64)), np.atleast_2d(np.asarray(ref, dtype=np.float64))
+    assert got.shape == ref.shape, (what, got.shape, ref.shape)
+    assert np.isfinite(got).all(), f"{what}: logits that are not finite"
+    err = np.abs(got - ref)
+    if dtype == "float32":
+        assert err.max() < TOL_F32, f"{what}: {err.max()}"
+        return
+    share = err.max(axis=-1) / max(float(ref.std()), 0.25)
+    rel = np.sqrt((err ** 2).mean(axis=-1)) / np.maximum(ref.std(axis=-1), 1e-3)
+    bad = (share >= TOL_BF16) | (rel >= TOL_ROW_BF16)
+    if calm is not None:
+        bad &= np.asarray(calm, dtype=bool)
+    assert not bad.any(), f"{what}: rows {np.nonzero(bad)[0].tolist()} are off (share {share[bad]}, row error {rel[bad]})"
+
+
+# =====================================================================================================
+# Without a device.
+
+def test_config_is_read_and_checked(capsys):
+    from mdma_b200.config import ConfigError, DegavikConfig
+    cfg, ranks = CONFIGS["A"]
+    c = DegavikConfig.from_dict(with_ranks(cfg, ranks))
+    assert (c.vocab, c.width, len(c.layers)) == (97, 60, 6)
+    a = c.layers[1].mixer
+    assert (a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.keep_first, a.softcap, a.rot_dims) == (6, 2, 24, 16, 19, 3, 6.0, 8)
+    d = c.layers[0].mixer
+    assert (d.kv_heads, d.conv, d.decay_rank, d.gate_rank) == (2, 3, 11, 7)
+    assert [l.weights_of for l in c.layers] == [None, None, None, 0, 2, 1]
+    assert c.layers[2].mlp is None and c.layers[1].mlp.shared_ff == 36
+    b = DegavikConfig.from_dict(CONFIGS["B"][0])
+    assert b.layers[1].mixer.window == 0 and b.layers[1].mixer.rot_dims == 0 and b.layers[1].mixer.softcap == 0.0
+    assert "leaves alone" not in capsys.readouterr().err
+    chain = json.loads(json.dumps(cfg))
+    chain["layers"][5] = dict(chain["layers"][3], weights_of=3)                # a layer whose source has a source
+    assert DegavikConfig.from_dict(chain).layers[5].weights_of == 0
+
+    def refuse(change):
+        bad = json.loads(json.dumps(cfg))
+        change(bad)
+        with pytest.raises(ConfigError):
+            DegavikConfig.from_dict(bad)
+    refuse(lambda r: r.pop("norm"))
+    refuse(lambda r: r["layers"][0].update(type="mamba"))
+    refuse(lambda r: r["layers"][0]["mixer"].update(kv_heads=3))
+    refuse(lambda r: r["layers"][1]["mixer"]["rot"].update(dims=26))
+    refuse(lambda r: r["layers"][1]["mlp"]["router"].update(top=6))
+    refuse(lambda r: r["layers"][2]["mixer"].update(decay=[0.5]))
+    refuse(lambda r: r["layers"][3].update(weights_of=3))
+    refuse(lambda r: r["layers"][3].update(weights_of=9))
+    refuse(lambda r: r["layers"][3]["mixer"].update(dim=8))                    # not what the tensors' layer says
+    refuse(lambda r: r["layers"][0].update(mlp={"kind": "sparse"}))
+
+
+def test_sizes_come_from_the_tensors_shapes(tmp_path):
+    """The low-rank sizes stand in no config.json: a folder's headers give them, for layers with other layers' tensors too."""
+    from mdma_b200.config import load_config
+    from mdma_b200.engine.model import expected_tensors
+    from mdma_b200.weights import check_entries, open_model_files
+    cfg, ranks = CONFIGS["C"]
+    d, _ = make_model(cfg, ranks, 1, root=str(tmp_path))
+    arch, typed = load_config(d)
+    assert [(l.mixer.decay_rank, l.mixer.gate_rank) for l in typed.layers if l.type == "channel_delta"] == [(16, 24), (24, 8), (16, 24)]
+    entries = {}
+    for f in open_model_files(d):
+        entries.update(f.entries)
+    check_entries(entries, expected_tensors(arch.describe(typed)))
+    os.remove(os.path.join(d, "model.safetensors"))
+    _, typed = load_config(d)                                                   # no tensors: a head's size
+    assert typed.layers[1].mixer.decay_rank == 64
+
+
+def test_layers_with_other_layers_tensors_are_runs_of_those_layers():
+    from mdma_b200.config import load_config
+    from mdma_b200.engine.model import DecoderModel
+    arch, typed = load_config(with_ranks(*CONFIGS["A"]))
+    spec = arch.describe(typed)
+    assert [e.layer for e in spec.schedule] == [0, 1, 2, 0, 2, 1] and all(e.cache is None for e in spec.schedule)
+    model = DecoderModel(spec)
+    names = set(model.expected_tensors())
+    assert "l1.mix.talk" in names and "l0.mix.q.conv" in names and not any(n.startswith(("l3.", "l4.", "l5.")) for n in names)
+    assert [n is not None for n in model.kv_needs()] == [False, True, False, False, False, True]
+    assert [n is not None for n in model.state_needs()] == [True, False, True, True, True, False]
+
+
+def test_plan_without_a_device(tmp_path):
+    from mdma_b200.engine.step import plan_only
+    for key in CONFIGS:
+        d, _ = make_model(*CONFIGS[key], 2, root=str(tmp_path))
+        for dtype in ("float32", "bfloat16"):
+            p = plan_only(d, dtype=dtype, max_batch=3, max_context=128)
+            assert p["total_bytes"] > p["weights_bytes"] > 0 and p["slots"] == 3
+
+
+def test_the_benchmark_configuration_is_a_valid_model():
+    import bench
+    from mdma_b200.config import load_config
+    from mdma_b200.engine.model import DecoderModel
+    from mdma_b200.ops_tensor import mixed_weights_supported
+    arch, typed = load_config(bench.degavik_config(2048, 4, 32000))
+    model = DecoderModel(arch.describe(typed))
+    assert {l.type for l in typed.layers} == {"channel_delta", "attention", "retention"}
+    assert mixed_weights_supported(16, 4, 128, 128) and len(model.expected_tensors()) > 100
