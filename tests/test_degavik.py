@@ -128,3 +128,60 @@ def test_the_benchmark_configuration_is_a_valid_model():
     model = DecoderModel(arch.describe(typed))
     assert {l.type for l in typed.layers} == {"channel_delta", "attention", "retention"}
     assert mixed_weights_supported(16, 4, 128, 128) and len(model.expected_tensors()) > 100
+
+
+def test_the_plain_statement_notices_each_mechanism():
+    """With one mechanism of the statement changed, some logit moves by many times the tolerance: a test that passes with
+    the engine doing the same wrong thing is not possible without being noticed here."""
+    cfg, ranks = CONFIGS["A"]
+    W = {n: t.double() for n, t in make_tensors(cfg, ranks, 23).items()}
+    ids = ids_of(cfg, 40, 3)
+    ref = pd.forward(cfg, W, ids)
+
+    def moved(cfg2=cfg, W2=W):
+        return float((pd.forward(cfg2, W2, ids) - ref).abs().max())
+
+    def change(layer, **mixer):
+        out = json.loads(json.dumps(cfg))
+        for key, v in mixer.items():
+            out["layers"][layer]["mixer"][key] = v
+        return out
+    floor = 200 * TOL_F32
+    assert moved(change(1, mask={"size": 20, "keep_first": 3})) > floor        # the window's edge
+    assert moved(change(1, mask={"size": 19, "keep_first": 2})) > floor        # the kept tokens' edge
+    assert moved(change(1, softcap=None)) > floor
+    assert moved(change(1, rot={"dims": 8, "base": 110.0})) > floor
+    assert moved(change(2, decay=[0.6, 0.93, 0.99])) > floor
+    assert moved(change(2, rot=None)) > floor
+    for name in W:
+        if not name.startswith(("l0.", "l1.", "l2.")) or ".mlp.e" in name:
+            continue
+        assert moved(cfg, {**W, name: W[name].roll(1, 0)}) > floor, name        # its rows in another order
+    layers = json.loads(json.dumps(cfg))["layers"]
+    layers[3]["weights_of"] = 3
+    own = {n.replace("l0.", "l3."): t * 1.1 for n, t in W.items() if n.startswith("l0.")}
+    assert moved(dict(cfg, layers=layers), {**W, **own}) > floor                # a layer with tensors of its own
+
+
+def test_kept_first_tokens_keep_their_pages():
+    """A windowed group with kept tokens gives pages back in the middle of a sequence, never those of the first tokens."""
+    from mdma_b200.cache import KVNeed, SequenceCache
+    for keep, pages in ((0, 0), (1, 1), (4, 1), (5, 2)):
+        c = SequenceCache([KVNeed(1, 8, window=6, keep_first=keep)], [None], max_tokens=64, max_slots=2, max_context=64,
+                          dtype=torch.float32, device="cpu", page_size=4)
+        s, t = c.acquire(), c.acquire()
+        for slot, n in ((s, 21), (t, 3)):
+            c.extend({slot: n})
+            c.commit({slot: n})
+        g = c.groups[0]
+        for length in range(21, 40):
+            held = set(g.seq_pages[s])
+            live = set(range(max(0, length + 1 - 6) // 4, (length - 1) // 4 + 1))
+            assert held == live | set(range(pages)), (keep, length, held)
+            c.check()
+            c.extend({s: 1})
+            c.commit({s: 1})
+        c.release(s)
+        c.release(t)
+        c.check()
+        assert g.pages.free_count == g.n_pages
