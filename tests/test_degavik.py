@@ -185,3 +185,115 @@ def test_kept_first_tokens_keep_their_pages():
         c.release(t)
         c.check()
         assert g.pages.free_count == g.n_pages
+
+
+# =====================================================================================================
+# Kernels alone (GPU).
+
+def _dev(t, dtype=torch.float32):
+    return t.to(device="cuda", dtype=dtype).contiguous()
+
+
+def _i32(a):
+    return torch.as_tensor(np.asarray(a, dtype=np.int32), device="cuda")
+
+
+class _Step:
+    """The step metadata the kernels' entry points read, for a call outside an engine."""
+
+    def __init__(self, lengths, pos0, slots):
+        self.n_seqs, self.n_tokens = len(lengths), sum(lengths)
+        self.max_new, self.max_len = max(lengths), max(p + n for p, n in zip(pos0, lengths))
+        self.seq_start = _i32(np.concatenate([[0], np.cumsum(lengths)]))
+        self.seq_pos0, self.seq_slot = _i32(pos0), _i32(slots)
+        self.tok_seq = _i32(np.concatenate([np.full(n, s) for s, n in enumerate(lengths)]))
+        self.tok_pos = _i32(np.concatenate([np.arange(p, p + n) for p, n in zip(pos0, lengths)]))
+        self.most_seqs = None
+
+
+DELTA_SIZES = [(3, 3, 32, 32, 4, 24, 24, 0.0), (4, 2, 12, 20, 3, 11, 7, 0.0), (2, 2, 9, 13, 1, 5, 13, 0.0), (2, 2, 96, 40, 2, 16, 8, 0.0),
+               (2, 1, 160, 64, 7, 8, 16, 0.0), (3, 3, 48, 96, 5, 20, 12, 0.0), (2, 2, 128, 128, 4, 128, 64, 0.0), (2, 2, 64, 48, 4, 16, 16, 4.0)]
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("H,G,D,V,taps,ra,rg,strong", DELTA_SIZES)
+@pytest.mark.parametrize("walk", ["rows", "chunks", "tokens"])
+def test_delta_rule_walks(walk, H, G, D, V, taps, ra, rg, strong):
+    """Unequal sequences in two steps each (the second starts from kept inputs and state, at no chunk's edge), against the
+    statement's recurrence: row by row, a chunk of rows at a time, and single tokens from the projection to the gated
+    norm.  `strong`: decays that take a channel to nothing within a token.  Slots are taken out of order."""
+    from mdma_b200 import ops
+    if walk == "chunks" and (D % 4 or V % 4):
+        pytest.skip("the chunk kernels take heads of multiples of four")
+    if walk == "tokens" and not ops.delta_token_fits(H, G, D, V, ra, rg, taps):
+        pytest.skip("the single-token kernel does not take these sizes")
+    gen = torch.Generator().manual_seed(5)
+    rn = lambda *s: torch.randn(s, generator=gen, dtype=torch.float64)
+    bf = lambda t: t.bfloat16().double()
+    ch = 2 * G * D + H * V
+    conv_at = -(-H * D * V // 4) * 4
+    conv = bf(0.6 * rn(ch, taps))
+    a_log, dt, norm = bf(1.5 * rn(H) - 1), bf(rn(H * D) - 1.5 + strong), bf(1 + 0.3 * rn(V))
+    a2, g2 = bf(rn(H * D, ra) * ra ** -0.5), bf(rn(H * V, rg) * rg ** -0.5)
+    first, then = ([37, 1, 16], [19, 30, 2]) if walk != "tokens" else ([1, 1, 1], [1, 1, 1])
+    cuts = [first, then] if walk != "tokens" else [[1, 1, 1]] * 7
+    slots, n_slots = [2, 0, 3], 4
+    total = [sum(c[s] for c in cuts) for s in range(3)]
+    rows = [rn(t, ch + H + ra + rg).float().double() for t in total]
+    refs, gated = [], []
+    for x in rows:
+        T = x.shape[0]
+        y = pd.silu(pd.short_conv(x[:, :ch], conv))
+        q = pd.unit_vector(y[:, :G * D].reshape(T, G, D)) * D ** -0.5
+        k = pd.unit_vector(y[:, G * D:2 * G * D].reshape(T, G, D))
+        rep = H // G
+        step = pd.softplus(x[:, ch + H:ch + H + ra] @ a2.T + dt).reshape(T, H, D)
+        g = torch.exp(-torch.exp(a_log)[None, :, None] * step)
+        o = pd.delta_steps(q.repeat_interleave(rep, 1), k.repeat_interleave(rep, 1), y[:, 2 * G * D:].reshape(T, H, V), g,
+                           torch.sigmoid(x[:, ch:ch + H]))
+        refs.append(o.reshape(T, H * V))
+        gated.append((pd.rms_unit(o, 1e-5) * norm).reshape(T, H * V) * torch.sigmoid(x[:, ch + H + ra:] @ g2.T))
+    state = torch.full((n_slots, conv_at + (taps - 1) * ch + 4), float("nan"), device="cuda")[:, :conv_at + (taps - 1) * ch]
+    for s in slots:
+        state[s] = 0.0
+    kept = state[:, conv_at:] if taps > 1 else None
+    c_conv, c_a, c_dt = _dev(conv, torch.bfloat16), _dev(a_log, torch.bfloat16), _dev(dt, torch.bfloat16)
+    at = [0, 0, 0]
+    for cut in cuts:
+        ctx = _Step(cut, at, slots)
+        n = ctx.n_tokens
+        x = torch.cat([rows[s][at[s]:at[s] + cut[s]] for s in range(3)])
+        proj = _dev(x)
+        want = torch.cat([refs[s][at[s]:at[s] + cut[s]] for s in range(3)])
+        if walk == "tokens":
+            out = torch.zeros(n, H * V, dtype=torch.bfloat16, device="cuda")
+            half = 0.25 * proj                                                   # the projection as two partial sums
+            partial = torch.stack([half, proj - half]).contiguous()
+            split = at[0] % 2 == 1
+            src = torch.full_like(proj, float("nan")) if split else proj
+            ops.delta_token(src, _dev(a2, torch.bfloat16), _dev(g2, torch.bfloat16), c_conv, taps, c_a, c_dt, _dev(norm, torch.bfloat16),
+                            ctx, state, conv_at, out, H, D, V, 1e-6, D ** -0.5, 1e-5, partial if split else None, 2, n * proj.shape[1])
+            want = torch.cat([gated[s][at[s]:at[s] + 1] for s in range(3)])
+            torch.testing.assert_close(out.double().cpu(), want, rtol=1e-2, atol=2e-3)
+        else:
+            raw = _dev(x[:, ch + H:ch + H + ra] @ a2.T)
+            out = torch.zeros(n, H * V, device="cuda")
+            if walk == "rows":
+                e = lambda c: torch.empty(n, c, device="cuda")
+                q, k, v, lg, beta = e(G * D), e(G * D), e(H * V), e(H * D), e(H)
+                ops.delta_prepare(proj, raw, c_conv, taps, c_a, c_dt, ctx, kept, q, k, v, lg, beta, H, G, D, V, 1e-6, D ** -0.5)
+                ops.delta_scan(q, k, v, lg, beta, ctx, state[:, :H * D * V], out, H, G, D, V)
+            else:
+                floats = (n // 16 + 4) * ops.delta_chunk_floats(H, D, V)
+                scratch = torch.full((floats + 64,), float("nan"), device="cuda")
+                ops.delta_chunks(proj, raw, c_conv, taps, c_a, c_dt, kept, scratch[:floats], ctx, state[:, :H * D * V], out, H, G, D, V,
+                                 1e-6, D ** -0.5)
+                assert torch.isnan(scratch[floats:]).all()
+            ops.delta_conv_keep(proj, taps, ch, ctx, kept)
+            torch.testing.assert_close(out.double().cpu(), want, rtol=2e-5, atol=4e-6)
+        at = [a + c for a, c in zip(at, cut)]
+    assert torch.isnan(state[1]).all()                                           # a slot of nobody's is left alone
+    if taps > 1:
+        for s in range(3):                                                       # the kept inputs: the last rows, zeros before
+            have = torch.cat([torch.zeros(taps - 1, ch, dtype=torch.float64), rows[s][:, :ch]])[-(taps - 1):]
+            torch.testing.assert_close(kept[slots[s]].reshape(taps - 1, ch).double().cpu(), have, rtol=1e-6, atol=1e-6)
