@@ -297,3 +297,326 @@ def test_delta_rule_walks(walk, H, G, D, V, taps, ra, rg, strong):
         for s in range(3):                                                       # the kept inputs: the last rows, zeros before
             have = torch.cat([torch.zeros(taps - 1, ch, dtype=torch.float64), rows[s][:, :ch]])[-(taps - 1):]
             torch.testing.assert_close(kept[slots[s]].reshape(taps - 1, ch).double().cpu(), have, rtol=1e-6, atol=1e-6)
+
+
+def _plain_mixed(q, k, v, mix, factor, cap, window, keep):
+    """q [T, H, D], k [T, G, D], v [T, G, V] -> [T, H * V]: the statement's softmax, visibility and mixing."""
+    T, H, _ = q.shape
+    rep = H // k.shape[1]
+    s = torch.einsum("ihd,jhd->hij", q, k.repeat_interleave(rep, 1)) * factor[:, None, None]
+    if cap:
+        s = cap * torch.tanh(s / cap)
+    see = pd.visible(T, {"size": window, "keep_first": keep} if window else None)
+    p = torch.einsum("hg,gij->hij", mix, torch.softmax(s.masked_fill(~see, -float("inf")), -1))
+    return torch.einsum("hij,jhd->ihd", p, v.repeat_interleave(rep, 1)).reshape(T, -1)
+
+
+ATTENTION_SIZES = [(6, 2, 24, 16, 19, 3, 6.0), (8, 4, 32, 48, 64, 18, 12.0), (5, 1, 10, 6, 0, 0, 0.0), (8, 2, 16, 8, 2, 1, 3.0),
+                   (16, 4, 64, 128, 48, 0, 30.0), (24, 2, 16, 16, 33, 5, 4.0), (4, 4, 48, 96, 0, 0, 8.0), (12, 12, 128, 128, 70, 2, 0.0),
+                   (3, 3, 256, 16, 40, 70, 5.0), (32, 8, 128, 32, 100, 1, 20.0)]
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("kernel", ["plain32", "plain16", "rows", "step"])
+@pytest.mark.parametrize("H,G,D,V,window,keep,cap", ATTENTION_SIZES)
+def test_attention_with_mixed_weights_edges_pages_and_batches(kernel, H, G, D, V, window, keep, cap):
+    """Unequal sequences with shuffled pages (rows nobody owns hold NaN); prompts from the start and portions on a cached
+    prefix.  At every row one key stands out: the first one inside the window, or the last one before it (whose weight must
+    be nothing), or the last kept token, or the one after it: a window or a kept range one token off moves the row by far
+    more than the tolerance."""
+    from mdma_b200 import ops, ops_tensor
+    half = kernel != "plain32"
+    if kernel in ("rows", "step") and not ops_tensor.mixed_weights_supported(H, G, D, V):
+        pytest.skip("the tensor-core kernels do not take these sizes")
+    if kernel == "step" and not ops_tensor.mixed_weights_step_fits(H, G, D, V):
+        pytest.skip("the single-token kernel does not take these sizes")
+    dtype = torch.bfloat16 if half else torch.float32
+    gen = torch.Generator().manual_seed(11)
+    rn = lambda *s: torch.randn(s, generator=gen, dtype=torch.float64)
+    r = (lambda t: t.bfloat16().double()) if half else (lambda t: t.float().double())
+    mix, factor = r(torch.eye(H, dtype=torch.float64) + 0.5 * rn(H, H)), (0.7 + 0.5 * torch.rand(H, generator=gen, dtype=torch.float64)).float().double() * D ** -0.5
+    page, lengths, pages_per = 16, [150, 33, 1, 97], 10
+    sets = []
+    for T in lengths:
+        q, k, v = 0.3 * rn(T, H, D), rn(T, G, D), rn(T, G, V)
+        k = k / k.norm(dim=-1, keepdim=True)
+        for i in range(T):                              # the key that stands out for row i: by turns
+            edges = ([i - window + 1, i - window, keep - 1, keep] if window else [0, i // 2, i, i - 31])
+            j = edges[i % 4]
+            if 0 <= j <= i:
+                q[i] = q[i] + (14.0 / D ** -0.5 / 8) * k[j].repeat_interleave(H // G, 0)
+        sets.append((r(q), r(k), r(v)))
+    refs = [_plain_mixed(q, k, v, mix, factor, cap, window, keep) for q, k, v in sets]
+    if window:                                          # a token more or less would show
+        for w2, k2 in ((window + 1, keep), (window - 1 or 3, keep), (window, keep + 1)) + (((window, keep - 1),) if keep else ()):
+            moved = float((_plain_mixed(*sets[0], mix, factor, cap, w2, k2) - refs[0]).abs().max())
+            assert moved > 3 * (1e-2 * float(refs[0].abs().max().clamp(min=1.0)) if half else 3e-5), (w2, k2, moved)
+    perm = torch.randperm(4 * pages_per + 3, generator=gen)[:4 * pages_per].reshape(4, pages_per)
+    kc = torch.full((4 * pages_per + 3, page, G, D), float("nan"), dtype=dtype, device="cuda")
+    vc = torch.full((4 * pages_per + 3, page, G, V), float("nan"), dtype=dtype, device="cuda")
+    slots = [3, 1, 0, 2]
+
+    class View:
+        pass
+    view = View()
+    view.k, view.v, view.page_size, view.max_pages = kc, vc, page, pages_per
+    view.page_table = _i32(perm.numpy())
+    for s, (q, k, v) in enumerate(sets):
+        for t in range(lengths[s]):
+            p = int(perm[slots[s], t // page])
+            kc[p, t % page], vc[p, t % page] = k[t].to(dtype).cuda(), v[t].to(dtype).cuda()
+
+    def call(new, pos0, which):
+        ctx = _Step(new, pos0, [slots[s] for s in which])
+        pitch = -(-H * D // 8) * 8 + 8
+        rows = torch.full((ctx.n_tokens, pitch), float("nan"), dtype=dtype, device="cuda")
+        rows[:, :H * D] = torch.cat([sets[s][0][p:p + n].reshape(n, -1) for s, n, p in zip(which, new, pos0)]).to(dtype).cuda()
+        out = torch.full((ctx.n_tokens, H * V), float("nan"), dtype=dtype, device="cuda")
+        m, f = _dev(mix), _dev(factor)
+        if kernel.startswith("plain"):
+            ops.mixed_weights_attention(rows, kc, vc, m, f, cap, ctx, view.page_table, pages_per, page, out, H, G, D, V, window, keep)
+        elif kernel == "rows":
+            scratch = torch.full((41 * H * G * V,), float("nan"), device="cuda")             # slabs of 41 tokens
+            ops_tensor.mixed_weights_attention(ctx, rows, view, m, f, cap, out, scratch, H, G, D, V, window, keep)
+        else:
+            for splits in (1, 3, 40):
+                out.fill_(float("nan"))
+                scratch = torch.full((ctx.n_seqs * splits * H * (G * V + 2),), float("nan"), device="cuda")
+                ops_tensor.mixed_weights_attention(ctx, rows, view, m, f, cap, out, scratch, H, G, D, V, window, keep, step=splits)
+                compare(out, new, pos0, which)
+        return out
+
+    def compare(out, new, pos0, which):
+        want = torch.cat([refs[s][p:p + n] for s, n, p in zip(which, new, pos0)])
+        tol = dict(rtol=3e-5, atol=3e-5) if not half else dict(rtol=1e-2, atol=1e-2 * float(want.abs().max().clamp(min=1.0)))
+        torch.testing.assert_close(out.double().cpu(), want, **tol)
+    if kernel == "step":
+        for back in (1, 2, 3, 4, 60):
+            which = [s for s in range(4) if lengths[s] >= back]
+            call([1] * len(which), [lengths[s] - back for s in which], which)
+        return
+    for new, pos0, which in (([150, 33, 1, 97], [0, 0, 0, 0], [0, 1, 2, 3]), ([50, 2, 47], [100, 31, 50], [0, 1, 3]), ([3], [147], [0])):
+        compare(call(new, pos0, which), new, pos0, which)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,D,V,dims,layout,decay", [(3, 20, 28, 20, "split_half", (0.6, 0.93, 0.995)), (2, 10, 6, 4, "split_half", (1.0, 0.8)),
+                                                     (2, 64, 64, 0, "split_half", (0.9, 0.99)), (2, 64, 32, 64, "split_half", (0.97, 0.9995)),
+                                                     (1, 128, 48, 96, "interleaved", (0.99,)), (4, 16, 16, 16, "interleaved", (0.5, 0.9, 0.99, 1.0))])
+@pytest.mark.parametrize("walk", ["rows", "chunks", "runs", "single"])
+def test_retention_walks(walk, dtype, H, D, V, dims, layout, decay):
+    """Linear attention without SiLU on turned q and k: two steps of unequal sequences from positions that go on, against
+    the statement's recurrence, for every walk of the kernel."""
+    from mdma_b200 import ops
+    from mdma_b200.parts.rotary import inverse_frequencies
+    gen = torch.Generator().manual_seed(13)
+    rn = lambda *s: torch.randn(s, generator=gen, dtype=torch.float64)
+    cuts = {"single": [[1, 1]] * 6, "runs": [[300, 70], [280, 259]]}.get(walk, [[45, 3], [20, 33]])
+    total = [sum(c[s] for c in cuts) for s in range(2)]
+    width = H * (2 * D + V)
+    rows = [rn(t, width).to(dtype).double() for t in total]
+    k_scale, base = D ** -0.5, 50.0
+    refs = []
+    for x in rows:
+        T, pos = x.shape[0], torch.arange(x.shape[0])
+        rot = {"dims": dims, "base": base}
+        q = pd.rotate(x[:, :H * D].reshape(T, H, D), pos, rot, layout)
+        k = pd.rotate(x[:, H * D:2 * H * D].reshape(T, H, D), pos, rot, layout) * k_scale
+        v = x[:, 2 * H * D:].reshape(T, H, V)
+        S, o = torch.zeros(H, D, V, dtype=torch.float64), torch.empty(T, H, V, dtype=torch.float64)
+        dk = torch.tensor(decay, dtype=torch.float64)[:, None, None]
+        for t in range(T):
+            S = dk * S + k[t][:, :, None] * v[t][:, None, :]
+            o[t] = torch.einsum("hdc,hd->hc", S, q[t])
+        refs.append(o.reshape(T, H * V))
+    table = _dev(inverse_frequencies(dims, base)) if dims else None
+    state = torch.zeros(4, H * D * V, device="cuda")
+    at, slots = [0, 0], [3, 1]
+    for cut in cuts:
+        ctx = _Step(cut, at, slots)
+        proj = _dev(torch.cat([rows[s][at[s]:at[s] + cut[s]] for s in range(2)]), dtype)
+        out = torch.full((ctx.n_tokens, H * V), float("nan"), device="cuda")
+        run_rows, most = (128, -(-max(cut) // 128)) if walk == "runs" else (0, 1)
+        scratch = torch.full((2 * most * H * D * V,), float("nan"), device="cuda") if run_rows else None
+        ops.linear_attention(proj, 0, H * D, 2 * H * D, _dev(torch.tensor(decay)), ctx.seq_start, ctx.seq_slot, state, out, 2, H, D, V,
+                             walk in ("chunks", "runs"), run_rows, most, scratch, single=walk == "single", silu=False, k_scale=k_scale,
+                             inv_freq=table, rotary_dim=dims, interleaved=layout == "interleaved", tok_pos=ctx.tok_pos)
+        want = torch.cat([refs[s][at[s]:at[s] + cut[s]] for s in range(2)])
+        torch.testing.assert_close(out.double().cpu(), want, rtol=5e-5, atol=5e-5 * float(want.abs().max()))
+        at = [a + c for a, c in zip(at, cut)]
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("gate_act", ["sigmoid", "silu"])
+@pytest.mark.parametrize("gdtype,odtype", [(torch.float32, torch.float32), (torch.bfloat16, torch.bfloat16)])
+@pytest.mark.parametrize("H,V,weighted", [(3, 28, True), (1, 5, False), (16, 128, True), (7, 40, False)])
+def test_gated_norm_per_head(H, V, weighted, gdtype, odtype, gate_act):
+    from mdma_b200 import ops
+    gen = torch.Generator().manual_seed(3)
+    n = 19
+    o, w = torch.randn(n, H * V, generator=gen), torch.randn(V, generator=gen)
+    gate = torch.randn(n, H * V + 3, generator=gen).to(gdtype)
+    out = torch.full((n, H * V), float("nan"), dtype=odtype, device="cuda")
+    ops.gated_head_rmsnorm(_dev(o), gate.cuda()[:, 3:], _dev(w) if weighted else None, out, n, H, V, 1e-5, gate_act)
+    g = gate[:, 3:].double()
+    want = pd.rms_unit(o.double().reshape(n, H, V), 1e-5) * (w.double() if weighted else 1.0)
+    want = want.reshape(n, H * V) * (pd.silu(g) if gate_act == "silu" else torch.sigmoid(g))
+    tol = 1e-5 if odtype == torch.float32 else 1e-2
+    torch.testing.assert_close(out.double().cpu(), want, rtol=tol, atol=tol)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("width", [35, 60, 128, 2048, 5120, 9000])
+@pytest.mark.parametrize("splits,stored", [(0, True), (3, True), (5, False)])
+@pytest.mark.parametrize("copy", [None, torch.bfloat16, torch.float32])
+def test_norm_on_a_result_added_with_a_copy_of_the_stream(width, splits, stored, copy):
+    """x += norm(y) * w, y whole or as partial sums (alone, or on top of what y holds), and the new x in another dtype."""
+    from mdma_b200 import ops
+    gen = torch.Generator().manual_seed(7)
+    n = 6
+    x, y, w = (torch.randn(*s, generator=gen) for s in ((n, width), (n, width), (width,)))
+    part = torch.randn(max(splits, 1), n, width, generator=gen)
+    only = stored and splits > 0
+    full = (torch.zeros_like(y) if only else y).double() + (part.double().sum(0) if splits else 0.0)
+    want = x.double() + pd.rms_unit(full, 1e-5) * w.double()
+    xd, yd = _dev(x), _dev(torch.full_like(y, float("nan")) if only else y)
+    out = None if copy is None else torch.full((n, width), float("nan"), dtype=copy, device="cuda")
+    pt = _dev(part) if splits else None
+    ops.rmsnorm_add(xd, yd, _dev(w), 1e-5, n, pt, splits, n * width, only, out)
+    torch.testing.assert_close(xd.double().cpu(), want, rtol=1e-5, atol=1e-5)
+    if out is not None:
+        assert torch.equal(out, xd.to(copy))
+    rounded = torch.empty(n, width, dtype=torch.bfloat16, device="cuda")
+    ops.copy_rows(xd, rounded, n)
+    assert torch.equal(rounded, xd.bfloat16())
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("experts,top,W", [(5, 2, 60), (3, 1, 35), (4, 4, 35), (64, 6, 128)])
+def test_router_with_a_bias_on_its_logits(dtype, experts, top, W):
+    """Choice and weights both follow the biased logits."""
+    from mdma_b200 import ops
+    gen = torch.Generator().manual_seed(19)
+    h, router = torch.randn(33, W, generator=gen).to(dtype), (torch.randn(experts, W, generator=gen) * W ** -0.5).to(dtype)
+    bias = (torch.randn(experts, generator=gen) * 4).to(dtype)
+    chosen, weights = torch.zeros(33, top, dtype=torch.int32, device="cuda"), torch.zeros(33, top, device="cuda")
+    ops.route(_dev(h, dtype), _dev(router, dtype), None, None, 33, top, 1, 1, chosen, weights, None, logit_bias=_dev(bias, dtype))
+    z = h.double() @ router.double().T + bias.double()
+    best = torch.sort(z, -1, descending=True)
+    want = torch.zeros(33, experts, dtype=torch.float64).scatter(1, best.indices[:, :top], torch.softmax(best.values[:, :top], -1))
+    got = torch.zeros(33, experts, dtype=torch.float64).scatter(1, chosen.long().cpu(), weights.double().cpu())
+    torch.testing.assert_close(got, want, rtol=1e-4, atol=1e-5)
+
+
+# =====================================================================================================
+# Whole models through the engine (GPU).
+
+_models: dict = {}
+
+
+def model_of(key, dtype, drawn=None, seed=None):
+    """(folder, config, float64 tensors as the engine holds them) of configuration `key`."""
+    k = (key, dtype)
+    if k not in _models:
+        store = torch.float32 if dtype == "float32" else torch.bfloat16
+        cfg, ranks = drawn or CONFIGS[key]
+        d, W = make_model(cfg, ranks, seed if seed is not None else 23 + ord(key[0]), store)
+        _models[k] = (d, cfg, W)
+    return _models[k]
+
+
+_refs: dict = {}
+
+
+def ref_of(key, dtype, ids):
+    """(the statement's logits, whether no close routing choice lies at or before a row)."""
+    k = (key, dtype, tuple(ids))
+    if k not in _refs:
+        _, cfg, W = model_of(key, dtype)
+        calls = []
+        logits = pd.forward(cfg, W, ids, closeness=calls).numpy()
+        gap = torch.stack(calls).min(0).values.numpy() if calls else np.full(len(ids), 9.0)
+        _refs[k] = (logits, np.minimum.accumulate(gap) > CLOSE_CALL)
+    return _refs[k]
+
+
+def check(got, pairs, dtype, what):
+    """`pairs`: per row (reference of `ref_of`, position)."""
+    close(got, np.stack([r[0][p] for r, p in pairs]), dtype, what, [r[1][p] for r, p in pairs])
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("key", ["A", "B", "C", "D"])
+def test_every_layer_against_the_plain_statement(key, dtype):
+    """The residual stream after every layer run, then the logits; one short prompt, the first tokens among the rows."""
+    from mdma_b200.engine import Engine, StepEntry
+    d, cfg, W = model_of(key, dtype)
+    ids = ids_of(cfg, 29, 4)
+    _, trace = pd.forward(cfg, W, ids, return_layers=True)
+    ref = ref_of(key, dtype, ids)
+    rows = np.nonzero(ref[1])[0] if dtype == "bfloat16" else np.arange(len(ids))
+    eng = Engine(d, dtype=dtype, max_batch=2, max_context=64, logit_rows=64, page_size=16)
+    got = []
+    eng.model.on_layer = lambda n, x: got.append(x.detach().double().cpu())
+    s = eng.acquire()
+    logits = eng.step([StepEntry(s, ids, list(range(len(ids))))]).cpu().numpy()
+    assert len(got) == len(trace) == len(cfg["layers"])
+    tol = 1e-4 if dtype == "float32" else 0.05
+    for n, (a, b) in enumerate(zip(got, trace)):
+        err = float((a - b)[rows].abs().max()) if len(rows) else 0.0
+        assert err < tol * max(1.0, float(b.abs().max())), f"after layer {n}: {err}"
+    check(logits, [(ref, p) for p in range(len(ids))], dtype, "logits")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("key", ["A", "B", "C", "D"])
+def test_batches_portions_decoding_and_reuse(key, dtype):
+    """Unequal prompts in one step; the same prompts cut in portions down to one and two tokens on a cached prefix;
+    token-by-token decoding; sequences that end early while others go on; slots and pages freed and taken again (rows
+    nobody owns hold NaN throughout).  In float32 every way of cutting gives the same logits to within a few units of
+    the last place."""
+    from mdma_b200.engine import Engine, StepEntry
+    d, cfg, W = model_of(key, dtype)
+    lengths = [90, 1, 33, 2, 17]
+    seqs = [ids_of(cfg, n, 20 + i) for i, n in enumerate(lengths)]
+    refs = [ref_of(key, dtype, s) for s in seqs]
+    eng = Engine(d, dtype=dtype, max_batch=5, max_context=96, logit_rows=160, page_size=16)
+
+    def run(plan):
+        """plan: per sequence, the sizes of its portions.  All sequences advance together, one portion a step."""
+        slots = [eng.acquire() for _ in seqs]
+        rows = [[] for _ in seqs]
+        at = [0] * len(seqs)
+        for step in range(max(len(p) for p in plan)):
+            live = [i for i in range(len(seqs)) if step < len(plan[i])]
+            eng.cache.poison_unused()
+            out = eng.step([StepEntry(slots[i], seqs[i][at[i]:at[i] + plan[i][step]], list(range(plan[i][step])))
+                            for i in live]).cpu().numpy()
+            o = 0
+            for i in live:
+                n = plan[i][step]
+                rows[i].append(out[o:o + n].copy())
+                o += n
+                at[i] += n
+                if at[i] == len(seqs[i]):
+                    eng.release(slots[i])           # ends early; its slot and its pages go back
+        eng.cache.check()
+        return [np.concatenate(r) for r in rows]
+
+    whole = run([[n] for n in lengths])
+    alone = []
+    for i, s in enumerate(seqs):                    # each alone, in a slot that the batch used
+        slot = eng.acquire()
+        alone.append(eng.step([StepEntry(slot, s, list(range(len(s))))]).cpu().numpy().copy())
+        eng.release(slot)
+    pieces = run([[2, 1, 30, 37, 1, 2, 16, 1], [1], [16, 1, 15, 1], [1, 1], [3, 14]])
+    decoded = run([[25] + [1] * 65, [1], [1] * 33, [2], [16, 1]])
+    for name, other in (("whole prompts", whole), ("alone", alone), ("portions", pieces), ("decoded", decoded)):
+        for i, (got, ref) in enumerate(zip(other, refs)):
+            check(got, [(ref, p) for p in range(lengths[i])], dtype, f"{name}, sequence {i}")
+            if dtype == "float32":
+                assert np.abs(got - whole[i]).max() <= 6e-6, f"{name}, sequence {i}: differs from the whole prompt"
