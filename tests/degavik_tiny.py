@@ -145,9 +145,9 @@ def make_tensors(cfg, ranks, seed):
         elif last == "temp":
             t = 1.0 + 0.4 * rn(*shape).abs()
         elif name.endswith("router.b"):
-            t = torch.randperm(shape[0], generator=g).float() * 1.5 + 0.2 * rn(*shape)     # logits lie apart
+            t = torch.randperm(shape[0], generator=g).float() * 2.5 + 0.2 * rn(*shape)     # logits lie apart
         elif last == "router":
-            t = rn(*shape) * (0.4 / shape[1] ** 0.5)
+            t = rn(*shape) * (0.25 / shape[1] ** 0.5)
         elif last == "b":
             t = rn(*shape) * (1.0 / shape[1] ** 0.5)
         elif last == "g" or last in ("a2", "g2"):
