@@ -120,7 +120,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 }
 template <typename TW, typename TC, int NV>
 __global__ void __launch_bounds__(512)
-rmsnorm_add_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ partial, int splits,
+rmsnorm_add_vec_kernel(float* __restrict__ x, float* __restrict__ y, const float* __restrict__ partial, int splits,
                        size_t split_stride, int only_partial, const TW* __restrict__ w, int width, float eps, TC* __restrict__ copy) {
     chain_release();
     const int n4 = width >> 2;
@@ -147,6 +147,7 @@ rmsnorm_add_vec_kernel(float* __restrict__ x, const float* __restrict__ y, const
                 const float4 t = *reinterpret_cast<const float4*>(p + (size_t)s * split_stride);
                 v[k].x += t.x; v[k].y += t.y; v[k].z += t.z; v[k].w += t.w;
             }
+            if (splits > 0 && !only_partial) *reinterpret_cast<float4*>(y + row + 4 * e) = v[k];
             sq = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, sq))));
         }
     }
@@ -226,7 +227,7 @@ int mdma_rmsnorm_add(float* x, float* y, const float* partial, int splits, long 
         const int n4 = width / 4, threads = n4 >= 512 ? 512 : (n4 + 31) / 32 * 32, nv = (n4 + threads - 1) / threads;
 #define MDMA_RA(NV)                                                                                                            \
         MDMA_DISPATCH_DTYPE(w_dtype, TW, MDMA_DISPATCH_DTYPE(copy_dtype, TC,                                                    \
-            launch_chained(rmsnorm_add_vec_kernel<TW, TC, NV>, dim3(n_rows), dim3(threads), 0, stream, x, (const float*)y, partial, \
+            launch_chained(rmsnorm_add_vec_kernel<TW, TC, NV>, dim3(n_rows), dim3(threads), 0, stream, x, y, partial, \
                            splits, (size_t)split_stride, only_partial, (const TW*)w, width, eps, (TC*)copy)))
         if (nv == 1) MDMA_RA(1); else if (nv == 2) MDMA_RA(2); else MDMA_RA(4);
 #undef MDMA_RA
