@@ -1,19 +1,17 @@
 """The gated delta rule with a decay per key channel (`channel_delta`).
 
-q, k = h Wq^T, h Wk^T [kv_heads x dim], v = h Wv^T [heads x v_dim]; head h uses q/k head h // (heads / kv_heads).  Each
-passes a short causal convolution over time per channel (`q.conv`, `k.conv`, `v.conv` [channels, taps], the last column
-is the current token's, zeros before the start) and SiLU; q and k become unit vectors per head, x / sqrt(sum(x^2) +
-unit_eps), and q is multiplied by dim^-1/2.  b = sigmoid(h Wb^T), one per head; g = exp(-exp(A_log_h) softplus(a2 a1 h +
-dt_bias)), one per head and key channel.  Per head, S [dim, v_dim]:
+Projections of a row h: q, k = Wq h, Wk h (kv_heads heads of dim numbers, every one serving heads / kv_heads neighbouring
+heads), v = Wv h (heads of v_dim).  y_t[c] = SiLU(sum_j C[c, taps-1-j] x_(t-j)[c]) replaces every channel c of the three,
+C the stacked `q.conv`, `k.conv`, `v.conv` and x_t = 0 for t < 0.  Then, head by head,
 
-    S <- diag(g) S;   u = b (v - S^T k);   S <- S + k u^T;   o = S^T q.
-
-Each head's o is divided by its root mean square, multiplied by the weight `norm` (shared by the heads) and by
-sigmoid(g2 g1 h), and the heads side by side go through Wo.
+    q' = dim^-1/2 q / |q|,   k' = k / |k|   with |x|^2 = unit_eps + sum x^2,
+    b = sigmoid(Wb h),   log g = -e^A_log softplus(A2 A1 h + dt_bias)      (a number a head; a number a head and channel),
+    S <- diag(g) S,   u = b (v - S^T k'),   S <- S + k' u^T,   o = S^T q'          S [dim, v_dim],
+    result = Wo [rms_unit(o) * norm * sigmoid(G2 G1 h)]      (`norm` has v_dim numbers for all heads).
 
 State per sequence: S (floats) and the convolutions' last taps-1 inputs.  Everything that enters the recurrence is float
-in both engines (the projections write float rows); the inner rows of the two low-rank projections go into their second products in
-the compute dtype.  The 32-bit engine and short portions walk row by row in one fixed order; the serving engine walks portions of
+in both engines (the projections write float rows); A1 h and G1 h go into their second products in the compute dtype.
+The 32-bit engine and short portions walk row by row in one fixed order; the serving engine walks portions of
 `CHUNKS_FROM` rows or more a chunk of rows at a time (csrc/delta_chunk.cu), and its single tokens take one kernel from
 the projection to the gated norm where its sizes fit (one q/k head per head).
 """
