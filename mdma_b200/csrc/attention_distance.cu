@@ -8,6 +8,10 @@
 // `out_scale` multiplies the result.  No rotation is applied here.  Scores, the running maximum, the
 // normaliser and the sums are float.
 //
+// The plain kernel takes further options: which keys a query sees (`KeyRule`: kept first tokens, chunks), a soft cap c
+// on the scores, c tanh(score / c) before the penalty; and several maps per head: query heads [head][map], key heads
+// [kv head][map], every map a softmax of its own over its keys and the kv head's values, results [head][map].
+//
 // Keys and values live in pages: row (page_table[slot][p / page_size] * page_size + p % page_size) of
 // a pool [rows, kv_heads, dim] for keys and [rows, kv_heads, v_dim] for values.
 //
@@ -43,29 +47,31 @@ kv_store_kernel(const T* __restrict__ proj, int proj_stride, int k_col, int v_co
 }
 
 // ---------------------------------------------------------------- plain kernel
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(128)
 attention_distance_plain_kernel(const T* __restrict__ q, int q_row_stride, const T* __restrict__ k_cache,
                                 const T* __restrict__ v_cache, const int* __restrict__ tok_seq,
                                 const int* __restrict__ tok_pos, const int* __restrict__ seq_slot,
                                 const int* __restrict__ page_table, int max_pages, int page_size,
                                 const float* __restrict__ slopes, const T* __restrict__ gate, int gate_stride,
-                                T* __restrict__ out, int n_heads, int n_kv_heads, int dim, int v_dim, int window,
-                                float scale, const float* __restrict__ sinks, int gate_heads, float out_scale) {
+                                TO* __restrict__ out, int n_heads, int n_kv_heads, int dim, int v_dim, KeyRule rule,
+                                float scale, const float* __restrict__ sinks, int gate_heads, float out_scale, float softcap,
+                                int maps) {
     chain_release();
     chain_wait();
     const int t = blockIdx.x;
-    const int h = blockIdx.y * 4 + (threadIdx.x >> 5);
+    const int hm = blockIdx.y * 4 + (threadIdx.x >> 5);        // head * maps + map
     const int lane = threadIdx.x & 31;
-    if (h >= n_heads) return;
+    if (hm >= n_heads * maps) return;
+    const int h = hm / maps;
     const int pos = tok_pos[t];
     const int slot = seq_slot[tok_seq[t]];
-    const int kvh = h / (n_heads / n_kv_heads);
-    const int first = window > 0 ? max(0, pos + 1 - window) : 0;
+    const int kvh = h / (n_heads / n_kv_heads), key_head = kvh * maps + hm % maps;
+    const int first = rule_first(rule, pos), kept = min(rule.keep_first, first);
     const float slope = slopes ? slopes[h] : 0.f;
 
     float qv[kMaxDim / 32], acc[kMaxDim / 32];
-    const T* qp = q + (size_t)t * q_row_stride + (size_t)h * dim;
+    const T* qp = q + (size_t)t * q_row_stride + (size_t)hm * dim;
 #pragma unroll
     for (int j = 0; j < kMaxDim / 32; ++j) {
         const int d = lane + 32 * j;
@@ -74,17 +80,19 @@ attention_distance_plain_kernel(const T* __restrict__ q, int q_row_stride, const
     }
     float m = -INFINITY, l = 0.f;
     const int* pages = page_table + (size_t)slot * max_pages;
-    for (int p = first; p <= pos; ++p) {
-        const size_t row = ((size_t)pages[p / page_size] * page_size + (size_t)(p % page_size)) * n_kv_heads + kvh;
-        const T* kp = k_cache + row * dim;
-        const T* vp = v_cache + row * v_dim;
+    for (int p = kept > 0 ? 0 : first; p <= pos; p = p + 1 == kept ? first : p + 1) {
+        const size_t row = (size_t)pages[p / page_size] * page_size + (size_t)(p % page_size);
+        const T* kp = k_cache + (row * n_kv_heads * maps + key_head) * dim;
+        const T* vp = v_cache + (row * n_kv_heads + kvh) * v_dim;
         float part = 0.f;
 #pragma unroll
         for (int j = 0; j < kMaxDim / 32; ++j) {
             const int d = lane + 32 * j;
             if (d < dim) part = fmaf(qv[j], to_float(kp[d]), part);
         }
-        const float s = warp_sum(part) * scale - slope * (float)(pos - p);
+        float s = warp_sum(part) * scale;
+        if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+        s -= slope * (float)(pos - p);
         const float m_new = fmaxf(m, s);
         const float corr = expf(m - m_new);     // exp(-inf) = 0 on the first key
         const float pe = expf(s - m_new);
@@ -104,7 +112,7 @@ attention_distance_plain_kernel(const T* __restrict__ q, int q_row_stride, const
 #pragma unroll
         for (int j = 0; j < kMaxDim / 32; ++j) acc[j] *= corr;
     }
-    T* op = out + ((size_t)t * n_heads + h) * v_dim;
+    TO* op = out + ((size_t)t * n_heads * maps + hm) * v_dim;
     const T* gp = gate ? gate + (size_t)t * gate_stride + (gate_heads ? (size_t)h : (size_t)h * v_dim) : nullptr;
     const float inv = out_scale / l;
 #pragma unroll
@@ -113,7 +121,7 @@ attention_distance_plain_kernel(const T* __restrict__ q, int q_row_stride, const
         if (d < v_dim) {
             float o = acc[j] * inv;
             if (gp) o *= 1.0f / (1.0f + expf(-to_float(gp[gate_heads ? 0 : d])));
-            op[d] = from_float<T>(o);
+            op[d] = from_float<TO>(o);
         }
     }
 }
@@ -354,18 +362,25 @@ int mdma_attention_distance_tiled_fits(int n_heads, int n_kv_heads, int dim, int
     return tiled_smem_bytes(n_heads / n_kv_heads, dim, v_dim) <= 200 * 1024 ? 1 : 0;
 }
 
-// tiled != 0: the tiled kernel (needs seq_start / seq_pos0 and max_new, the most rows a sequence brings).
+// tiled != 0: the tiled kernel (needs seq_start / seq_pos0 and max_new, the most rows a sequence brings; takes none of
+// keep_first, chunk, softcap, maps > 1 and float results of bfloat16 rows, `out_f32`).
 int mdma_attention_distance(const void* q, int dtype, int q_row_stride, const void* k_cache, const void* v_cache,
                             const int* tok_seq, const int* tok_pos, const int* seq_slot, const int* seq_start,
                             const int* seq_pos0, const int* page_table, int max_pages, int page_size,
                             const float* slopes, const void* gate, int gate_stride, void* out, int n_tokens, int n_seqs,
                             int max_new, int n_heads, int n_kv_heads, int dim, int v_dim, int window, float scale,
-                            int tiled, const float* sinks, int gate_heads, float out_scale, cudaStream_t stream) {
+                            int tiled, const float* sinks, int gate_heads, float out_scale, int keep_first, int chunk,
+                            float softcap, int maps, int out_f32, cudaStream_t stream) {
+    const KeyRule rule = {window, keep_first, chunk};
+    MDMA_REQUIRE(rule_ok(rule) && softcap >= 0.f && maps >= 1, "attention: window %d, kept %d, chunk %d, %d maps do not go together", window, keep_first, chunk, maps);
+    MDMA_REQUIRE(!gate || maps == 1, "attention: a gate goes with one map per head");
     MDMA_REQUIRE(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0, "attention: %d heads over %d kv heads", n_heads, n_kv_heads);
     MDMA_REQUIRE(dim > 0 && dim <= kMaxDim && v_dim > 0 && v_dim <= kMaxDim, "attention: head sizes %d / %d are beyond the limit %d", dim, v_dim, kMaxDim);
     MDMA_REQUIRE(page_table && page_size > 0 && max_pages > 0 && window >= 0, "attention: bad cache geometry");
     if (n_tokens == 0) return 0;
     if (tiled) {
+        MDMA_REQUIRE(keep_first == 0 && chunk == 0 && softcap == 0.f && maps == 1 && !(out_f32 && dtype == kBF16),
+                     "attention: the tiled kernel takes a window, a penalty and sinks only");
         const int group = n_heads / n_kv_heads;
         const size_t smem = tiled_smem_bytes(group, dim, v_dim);
         MDMA_REQUIRE(smem <= 200 * 1024, "attention: the tiled kernel's shared memory (%zu bytes) does not fit", smem);
@@ -393,12 +408,17 @@ int mdma_attention_distance(const void* q, int dtype, int q_row_stride, const vo
         MDMA_LAUNCH_OK("attention_distance_tiled");
         return 0;
     }
-    dim3 grid(n_tokens, (n_heads + 3) / 4);
-    MDMA_DISPATCH_DTYPE(dtype, T,
-        launch_chained(attention_distance_plain_kernel<T>, grid, dim3(128), 0, stream, (const T*)q, q_row_stride,
-                       (const T*)k_cache, (const T*)v_cache, tok_seq, tok_pos, seq_slot, page_table, max_pages, page_size,
-                       slopes, (const T*)gate, gate_stride, (T*)out, n_heads, n_kv_heads, dim, v_dim, window, scale,
-                       sinks, gate_heads, out_scale));
+    dim3 grid(n_tokens, (n_heads * maps + 3) / 4);
+#define MDMA_PLAIN_LAUNCH(TO)                                                                                              \
+        launch_chained(attention_distance_plain_kernel<T, TO>, grid, dim3(128), 0, stream, (const T*)q, q_row_stride,      \
+                       (const T*)k_cache, (const T*)v_cache, tok_seq, tok_pos, seq_slot, page_table, max_pages, page_size, \
+                       slopes, (const T*)gate, gate_stride, (TO*)out, n_heads, n_kv_heads, dim, v_dim, rule, scale,        \
+                       sinks, gate_heads, out_scale, softcap, maps)
+    MDMA_DISPATCH_DTYPE(dtype, T, {
+        if (out_f32) MDMA_PLAIN_LAUNCH(float);
+        else MDMA_PLAIN_LAUNCH(T);
+    });
+#undef MDMA_PLAIN_LAUNCH
     MDMA_LAUNCH_OK("attention_distance");
     return 0;
 }

@@ -1,4 +1,5 @@
 // C entry points of the tensor-core attention (kernels in attention_mma.cuh).
+#define MDMA_ATTENTION_GENERAL       // the EXT launcher too
 #include "attention_mma.cuh"
 
 using namespace mdma;
@@ -82,6 +83,20 @@ int mdma_attention_decode_rotary(const void* qkv, int q_stride, const float* pro
     return launch_attention_mma(qkv, q_stride, k_cache, v_cache, seq_start, seq_pos0, seq_slot, page_table, max_pages,
                                 page_size, out, n_seqs, n_seqs, 1, n_heads, n_kv_heads, head_dim, window, scale, splits,
                                 scratch, scratch_floats, stream, n_pages, status, &fz);
+}
+
+// Everything the EXT forms take; see launch_attention_mma_general.
+int mdma_attention_mma_general(const void* q, int q_stride, const void* k_cache, const void* v_cache, int n_pages,
+                               const int* seq_start, const int* seq_pos0, const int* seq_slot, const int* page_table,
+                               int max_pages, int page_size, void* out, float* out_f32, int n_tokens, int n_seqs, int max_new,
+                               int n_heads, int n_kv_heads, int head_dim, int v_dim, int maps, int window, int keep_first,
+                               int chunk, float softcap, float scale, int splits, float* scratch, long scratch_floats,
+                               int* status, const float* sink_log2, const float* slope_log2, cudaStream_t stream) {
+    const KeyRule rule = {window, keep_first, chunk};
+    return launch_attention_mma_general(q, q_stride, k_cache, v_cache, n_pages, seq_start, seq_pos0, seq_slot, page_table,
+                                        max_pages, page_size, out, out_f32, n_tokens, n_seqs, max_new, n_heads, n_kv_heads,
+                                        head_dim, v_dim, maps, rule, softcap, scale, splits, scratch, scratch_floats, status,
+                                        sink_log2, slope_log2, stream);
 }
 
 int mdma_attention_fused_rotary_supported(int n_heads, int n_kv_heads, int head_dim, int page_size, int rotary_dim) {

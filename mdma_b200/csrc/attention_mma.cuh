@@ -13,6 +13,10 @@
 // its maximum and sum, and a second kernel merges them in split order, so the
 // result does not depend on timing.
 // Limits: head_dim a multiple of 16 up to 128; group size up to 64.
+// EXT forms of the kernels take further options (the fields of AttnParams marked so): value heads of a size of their own,
+// a `KeyRule` (key blocks with kept first tokens in front of the window's are walked as one list), a soft cap on the
+// scores, several maps per head (query heads [head][map], key heads [kv head][map], one value head per kv head; the
+// results and partial sums lie [token][head][map]), float results.
 #pragma once
 #include <mutex>
 
@@ -76,7 +80,18 @@ struct AttnParams {
     const float* rot_inv_freq; int rotary_dim; int rot_interleaved;
     const float* proj_partial; int proj_splits; long proj_split_stride; int proj_width;
     __nv_bfloat16* k_cache_w; __nv_bfloat16* v_cache_w;
+    // EXT only
+    int v_dim, maps;
+    KeyRule rule;                                   // in the place of `window`
+    float cap_log2, cap_rate;                       // soft cap c: cap_log2 = c log2(e), cap_rate = 2 scale log2(e) / c on the raw score; 0: none
+    float* out_f32;                                 // results as float rows instead of `out`
 };
+// A raw dot product as a score in powers of two: capped, cap_log2 tanh(x) with tanh as 1 - 2 / (1 + e^(2 x)).
+template <bool EXT>
+__device__ __forceinline__ float score_log2(float raw, const AttnParams& p) {
+    if (EXT && p.cap_log2 > 0.f) return fmaf(-2.0f * p.cap_log2, __fdividef(1.0f, 1.0f + exp2f(raw * p.cap_rate)), p.cap_log2);
+    return raw * p.scale_log2;
+}
 
 // Tile shared-memory rows are DMAX elements wide; 16-byte chunk c of row r sits at chunk c ^ (r & 7).
 template <int DMAX>
@@ -84,7 +99,7 @@ __device__ __forceinline__ uint32_t tile_offset(int row, int chunk) {
     return (uint32_t)(row * DMAX * 2 + ((chunk ^ (row & 7)) << 4));
 }
 
-template <int DMAX>
+template <int DMAX, bool EXT = false>
 __global__ void __launch_bounds__(kAttnThreads)
 attention_mma_kernel(const AttnParams p) {
     constexpr int kChunks = DMAX / 8;              // 16-byte chunks per row
@@ -96,7 +111,8 @@ attention_mma_kernel(const AttnParams p) {
     chain_release();
     chain_wait();
     const int seq = blockIdx.y;
-    const int kvh = blockIdx.z / p.splits, split = blockIdx.z % p.splits;
+    const int key_head = blockIdx.z / p.splits, split = blockIdx.z % p.splits;
+    const int maps = EXT ? p.maps : 1, kvh = EXT ? key_head / maps : key_head, map = EXT ? key_head % maps : 0;
     const int row0_seq = p.seq_start[seq];
     const int n_new = p.seq_start[seq + 1] - row0_seq;
     const int tok0 = blockIdx.x * p.tile_tokens;            // first token of this tile within the sequence's new tokens
@@ -106,14 +122,18 @@ attention_mma_kernel(const AttnParams p) {
     const int last_pos = pos0 + n_tok - 1;
     const int* pages = p.page_table + (size_t)p.seq_slot[seq] * p.max_pages;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int D = p.head_dim, G = p.group;
-    const int d_chunks = D / 8;
+    const int D = p.head_dim, G = p.group, DV = EXT ? p.v_dim : D;
+    const int d_chunks = D / 8, dv_chunks = DV / 8;
 
     // key range of the tile, then of this split
-    const int first_key = p.window > 0 ? max(0, pos0 + 1 - p.window) : 0;
+    const int first_key = EXT ? rule_first(p.rule, pos0) : p.window > 0 ? max(0, pos0 + 1 - p.window) : 0;
     const int blk_lo = first_key / kKeys, blk_hi = last_pos / kKeys + 1;
-    const int per = (blk_hi - blk_lo + p.splits - 1) / p.splits;
-    const int b0 = blk_lo + split * per, b1 = min(blk_hi, b0 + per);
+    // block i of the walk: the blocks with kept first tokens in front of the window's first, then those up to the last
+    const int keep = EXT ? p.rule.keep_first : 0, kb = EXT ? min((keep + kKeys - 1) / kKeys, blk_lo) : 0;
+    auto block_of = [&](int i) { return EXT && i < blk_lo ? i - (blk_lo - kb) : i; };
+    const int list_lo = blk_lo - kb;
+    const int per = (blk_hi - list_lo + p.splits - 1) / p.splits;
+    const int b0 = list_lo + split * per, b1 = min(blk_hi, b0 + per);
 
     // ---- Q tile -> shared -------------------------------------------------
     for (int i = threadIdx.x; i < kRows * kChunks; i += kAttnThreads) {
@@ -121,23 +141,26 @@ attention_mma_kernel(const AttnParams p) {
         const int t = r / G, g = r % G;
         const bool valid = t < n_tok && c < d_chunks;
         const __nv_bfloat16* src = p.q + (size_t)(row0_seq + tok0 + (valid ? t : 0)) * p.q_stride +
-                                   (size_t)(kvh * G + g) * D + (valid ? c : 0) * 8;
+                                   (size_t)((kvh * G + g) * maps + map) * D + (valid ? c : 0) * 8;
         cp_async_16(sQ + tile_offset<DMAX>(r, c), src, valid);
     }
-    auto load_kv = [&](int blk, int stage) {
+    auto load_kv = [&](int at, int stage) {
+        const int blk = block_of(at);
         for (int i = threadIdx.x; i < kKeys * kChunks; i += kAttnThreads) {
             const int r = i / kChunks, c = i % kChunks;
             const int key = blk * kKeys + r;
             // keys outside [first_key, last_pos] are zero-filled, never read: their cache rows may be stale
             // (another sequence's, or not finite) and 0 * NaN would reach the output through P V
-            const bool valid = key <= last_pos && key >= first_key && c < d_chunks;
-            size_t off = 0;
-            if (valid) {
-                const int page = pages[key / p.page_size];
-                off = (((size_t)page * p.page_size + key % p.page_size) * p.n_kv_heads + kvh) * D + c * 8;
+            const bool owned = key <= last_pos && (key >= first_key || (EXT && key < keep));
+            const bool valid = owned && c < d_chunks, v_valid = EXT ? owned && c < dv_chunks : valid;
+            size_t off = 0, v_off = 0;
+            if (valid || v_valid) {
+                const size_t row = (size_t)pages[key / p.page_size] * p.page_size + key % p.page_size;
+                if (valid) off = (row * p.n_kv_heads * maps + key_head) * D + c * 8;
+                if (v_valid) v_off = (row * p.n_kv_heads + kvh) * DV + c * 8;
             }
             cp_async_16(sK + stage * kTile + tile_offset<DMAX>(r, c), p.k_cache + off, valid);
-            cp_async_16(sV + stage * kTile + tile_offset<DMAX>(r, c), p.v_cache + off, valid);
+            cp_async_16(sV + stage * kTile + tile_offset<DMAX>(r, c), p.v_cache + v_off, v_valid);
         }
     };
     if (b0 < b1) load_kv(b0, 0);
@@ -146,7 +169,8 @@ attention_mma_kernel(const AttnParams p) {
     // per-thread rows: r_lo = warp*16 + lane/4, r_hi = r_lo + 8
     const int r_lo = warp * 16 + (lane >> 2), r_hi = r_lo + 8;
     const int pos_lo = pos0 + min(r_lo / G, n_tok - 1), pos_hi = pos0 + min(r_hi / G, n_tok - 1);
-    const int win_lo = p.window > 0 ? pos_lo + 1 - p.window : 0, win_hi = p.window > 0 ? pos_hi + 1 - p.window : 0;
+    const int win_lo = EXT ? rule_first(p.rule, pos_lo) : p.window > 0 ? pos_lo + 1 - p.window : 0;
+    const int win_hi = EXT ? rule_first(p.rule, pos_hi) : p.window > 0 ? pos_hi + 1 - p.window : 0;
     const float sl_lo = p.slope_log2 ? p.slope_log2[kvh * G + r_lo % G] : 0.f, sl_hi = p.slope_log2 ? p.slope_log2[kvh * G + r_hi % G] : 0.f;
 
     float o[DMAX / 8][4];
@@ -182,15 +206,16 @@ attention_mma_kernel(const AttnParams p) {
             }
         }
         // ---- mask, online softmax ---------------------------------------------
-        const int key_base = blk * kKeys + (lane & 3) * 2;
+        const int key_base = block_of(blk) * kKeys + (lane & 3) * 2;
         float mx_lo = m_lo, mx_hi = m_hi;
 #pragma unroll
         for (int n = 0; n < kKeys / 8; ++n) {
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = key_base + n * 8 + e;
-                const float v_lo = (key <= pos_lo && key >= win_lo) ? s[n][e] * p.scale_log2 - sl_lo * (float)(pos_lo - key) : -INFINITY;
-                const float v_hi = (key <= pos_hi && key >= win_hi) ? s[n][2 + e] * p.scale_log2 - sl_hi * (float)(pos_hi - key) : -INFINITY;
+                const bool kept = EXT && key < keep;
+                const float v_lo = (key <= pos_lo && (key >= win_lo || kept)) ? score_log2<EXT>(s[n][e], p) - sl_lo * (float)(pos_lo - key) : -INFINITY;
+                const float v_hi = (key <= pos_hi && (key >= win_hi || kept)) ? score_log2<EXT>(s[n][2 + e], p) - sl_hi * (float)(pos_hi - key) : -INFINITY;
                 s[n][e] = v_lo; s[n][2 + e] = v_hi;
                 mx_lo = fmaxf(mx_lo, v_lo); mx_hi = fmaxf(mx_hi, v_hi);
             }
@@ -223,7 +248,7 @@ attention_mma_kernel(const AttnParams p) {
         for (int kk = 0; kk < kKeys / 16; ++kk) {
 #pragma unroll
             for (int n2 = 0; n2 < DMAX / 16; ++n2) {
-                if (n2 * 16 < D) {
+                if (n2 * 16 < DV) {
                     uint32_t v0, v1, v2, v3;
                     // transposed loads: (keys lo, d lo), (keys hi, d lo), (keys lo, d hi), (keys hi, d hi)
                     const int vrow = kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
@@ -248,23 +273,27 @@ attention_mma_kernel(const AttnParams p) {
         const float l = half ? l_hi : l_lo, m = half ? m_hi : m_lo;
         const size_t token = (size_t)(row0_seq + tok0 + t);
         const int head = kvh * G + g;
+        const size_t out_row = EXT ? (token * p.n_heads + head) * maps + map : token * p.n_heads + head;
         if (p.splits == 1) {
             const float inv = 1.0f / (p.sink_log2 ? l + exp2f(p.sink_log2[head] - m) : l);
-            __nv_bfloat16* dst = p.out + (token * p.n_heads + head) * D;
+            __nv_bfloat16* dst = p.out + out_row * DV;
+            float* fdst = EXT && p.out_f32 ? p.out_f32 + out_row * DV : nullptr;
 #pragma unroll
             for (int n = 0; n < DMAX / 8; ++n) {
                 const int d = n * 8 + (lane & 3) * 2;
-                if (d < D)
-                    *reinterpret_cast<__nv_bfloat162*>(dst + d) =
+                if (d < DV) {
+                    if (EXT && fdst) *reinterpret_cast<float2*>(fdst + d) = make_float2(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
+                    else *reinterpret_cast<__nv_bfloat162*>(dst + d) =
                         __floats2bfloat162_rn(o[n][half * 2] * inv, o[n][half * 2 + 1] * inv);
+                }
             }
         } else {
-            const size_t slot = (token * p.n_heads + head) * p.splits + split;
-            float* dst = p.part_o + slot * D;
+            const size_t slot = out_row * p.splits + split;
+            float* dst = p.part_o + slot * DV;
 #pragma unroll
             for (int n = 0; n < DMAX / 8; ++n) {
                 const int d = n * 8 + (lane & 3) * 2;
-                if (d < D) { dst[d] = o[n][half * 2]; dst[d + 1] = o[n][half * 2 + 1]; }
+                if (d < DV) { dst[d] = o[n][half * 2]; dst[d + 1] = o[n][half * 2 + 1]; }
             }
             if ((lane & 3) == 0) { p.part_ml[slot * 2] = m; p.part_ml[slot * 2 + 1] = l; }
         }
@@ -492,7 +521,7 @@ attention_decode_kernel(const AttnParams p) {
 // NW warps per block.  All blocks should run at once (a second, short round of blocks costs as
 // much as the first): eight warps and one block per SM while the blocks are no more than the SMs, else
 // four, three or two warps with three, four or five blocks per SM, or one warp with ten.
-template <int DMAX, int KB, int NW>
+template <int DMAX, int KB, int NW, bool EXT = false>
 __global__ void __launch_bounds__(NW * 32, NW == 8 ? 1 : NW == 4 ? 3 : NW == 3 ? 4 : NW == 2 ? 5 : 10)
 attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                             const AttnParams p) {
@@ -512,7 +541,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     __nv_bfloat16* fresh_k = reinterpret_cast<__nv_bfloat16*>(smem + kFreshOff);
     __nv_bfloat16* fresh_v = fresh_k + DMAX;
     float* sincos = reinterpret_cast<float*>(smem + kFreshOff + 4 * DMAX);
-    const bool fused = p.rot_inv_freq != nullptr;
+    const bool fused = !EXT && p.rot_inv_freq != nullptr;
     auto kv_offset = [](int row, int chunk) -> uint32_t {      // 16-byte chunk of a key row inside a tile
         return (uint32_t)((chunk >> 3) * kHalf + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
     };
@@ -529,30 +558,35 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     // is not the last one asks for it before waiting for that kernel.
     __syncthreads();                                     // the barriers exist
     const int seq = blockIdx.y;
-    const int kvh = blockIdx.z / p.splits, split = blockIdx.z % p.splits;
+    const int key_head = blockIdx.z / p.splits, split = blockIdx.z % p.splits;
+    const int maps = EXT ? p.maps : 1, kvh = EXT ? key_head / maps : key_head, map = EXT ? key_head % maps : 0;
     const int token = p.seq_start[seq];
     const int pos = p.seq_pos0[seq];
     const int* pages = p.page_table + (size_t)p.seq_slot[seq] * p.max_pages;
-    const int D = p.head_dim, G = p.group, d_chunks = D / 8;
-    const int first_key = p.window > 0 ? max(0, pos + 1 - p.window) : 0;
+    const int D = p.head_dim, G = p.group, d_chunks = D / 8, DV = EXT ? p.v_dim : D;
+    const int first_key = EXT ? rule_first(p.rule, pos) : p.window > 0 ? max(0, pos + 1 - p.window) : 0;
     const int blk_lo = first_key / KB, blk_hi = pos / KB + 1;
-    const int per = (blk_hi - blk_lo + p.splits - 1) / p.splits;
-    const int b0 = blk_lo + split * per, b1 = min(blk_hi, b0 + per);
-    const int halves = (D + 63) / 64;
+    // tile i of the walk: those with kept first tokens in front of the window's first, then those up to the last
+    const int keep = EXT ? p.rule.keep_first : 0, kb = EXT ? min((keep + KB - 1) / KB, blk_lo) : 0;
+    auto tile_of = [&](int i) { return EXT && i < blk_lo ? i - (blk_lo - kb) : i; };
+    const int list_lo = blk_lo - kb;
+    const int per = (blk_hi - list_lo + p.splits - 1) / p.splits;
+    const int b0 = list_lo + split * per, b1 = min(blk_hi, b0 + per);
+    const int k_halves = (D + 63) / 64, v_halves = (DV + 63) / 64;
 
-    auto load_tile = [&](const CUtensorMap* map, uint32_t dst, uint32_t bar, int blk) {      // one lane
-        const int key0 = blk * KB;
+    auto load_tile = [&](const CUtensorMap* tmap, bool is_v, uint32_t dst, uint32_t bar, int at) {      // one lane
+        const int key0 = tile_of(at) * KB, halves = is_v ? v_halves : k_halves, head = is_v ? kvh : key_head;
         const int page = pages[key0 / p.page_size], row = key0 % p.page_size;
         ptx::fence_proxy_async_shared();
         ptx::mbar_expect_tx(bar, halves * kHalf);
-        for (int h = 0; h < halves; ++h) ptx::tma_load_4d(dst + h * kHalf, map, bar, h * 64, kvh, row, page);
+        for (int h = 0; h < halves; ++h) ptx::tma_load_4d(dst + h * kHalf, tmap, bar, h * 64, head, row, page);
     };
     int blk = b0 + warp;
     if (*abort_flag != 0) blk = b1;
     // (with the rotary encoding done here the row of the own token is replaced in shared memory, so
     // the last tile does not depend on the kernel before either)
     const bool early = blk < b1 && (fused || blk != blk_hi - 1);
-    if (early && lane == 0) { load_tile(&map_k, sK, kbar, blk); load_tile(&map_v, sV, vbar, blk); }
+    if (early && lane == 0) { load_tile(&map_k, false, sK, kbar, blk); load_tile(&map_v, true, sV, vbar, blk); }
     if (fused) {
         // sines and cosines of this position (no dependence on the kernel before); the Q tile starts as zeros
         const int half = p.rotary_dim / 2;
@@ -565,7 +599,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(sQ + i * 16), "r"(0u) : "memory");
     }
     chain_wait();
-    if (!early && blk < b1 && lane == 0) { load_tile(&map_k, sK, kbar, blk); load_tile(&map_v, sV, vbar, blk); }
+    if (!early && blk < b1 && lane == 0) { load_tile(&map_k, false, sK, kbar, blk); load_tile(&map_v, true, sV, vbar, blk); }
     if (fused) {
         __syncthreads();                                 // sines, cosines and the zeroed tile are in place
         const int half = p.rotary_dim / 2, tail = D - p.rotary_dim;
@@ -618,7 +652,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         for (int i = threadIdx.x; i < 16 * kChunks; i += NW * 32) {
             const int r = i / kChunks, c = i % kChunks;
             const bool valid = r < G && c < d_chunks;
-            const __nv_bfloat16* src = p.q + (size_t)token * p.q_stride + (size_t)(kvh * G + (valid ? r : 0)) * D + (valid ? c : 0) * 8;
+            const __nv_bfloat16* src = p.q + (size_t)token * p.q_stride + (size_t)((kvh * G + (valid ? r : 0)) * maps + map) * D + (valid ? c : 0) * 8;
             cp_async_16(sQ + tile_offset<DMAX>(r, c), src, valid);
         }
         cp_async_commit();
@@ -632,7 +666,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     for (int kd = 0; kd < DMAX / 16; ++kd)
         ldmatrix_x4(sQ + tile_offset<DMAX>(lane & 15, kd * 2 + (lane >> 4)), qf[kd][0], qf[kd][1], qf[kd][2], qf[kd][3]);
 
-    const int win = p.window > 0 ? pos + 1 - p.window : 0;
+    const int win = EXT ? first_key : p.window > 0 ? pos + 1 - p.window : 0;
     // rows of the tile are the group's query heads: lane / 4 and that + 8
     const float sl_lo = p.slope_log2 ? p.slope_log2[kvh * G + min(lane >> 2, G - 1)] : 0.f;
     const float sl_hi = p.slope_log2 ? p.slope_log2[kvh * G + min((lane >> 2) + 8, G - 1)] : 0.f;
@@ -667,17 +701,17 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         }
         __syncwarp();
         const bool more = blk + NW < b1;
-        if (more && lane == 0) load_tile(&map_k, sK, kbar, blk + NW);     // K buffer is free: fetch the next tile's keys
-        const int key_base = blk * KB + (lane & 3) * 2;
+        if (more && lane == 0) load_tile(&map_k, false, sK, kbar, blk + NW);     // K buffer is free: fetch the next tile's keys
+        const int key_base = tile_of(blk) * KB + (lane & 3) * 2;
         float mx_lo = m_lo, mx_hi = m_hi;
 #pragma unroll
         for (int n = 0; n < KB / 8; ++n) {
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = key_base + n * 8 + e;
-                const bool vis = key <= pos && key >= win;
-                const float v_lo = vis ? s[n][e] * p.scale_log2 - sl_lo * (float)(pos - key) : -INFINITY;
-                const float v_hi = vis ? s[n][2 + e] * p.scale_log2 - sl_hi * (float)(pos - key) : -INFINITY;
+                const bool vis = key <= pos && (key >= win || (EXT && key < keep));
+                const float v_lo = vis ? score_log2<EXT>(s[n][e], p) - sl_lo * (float)(pos - key) : -INFINITY;
+                const float v_hi = vis ? score_log2<EXT>(s[n][2 + e], p) - sl_hi * (float)(pos - key) : -INFINITY;
                 s[n][e] = v_lo; s[n][2 + e] = v_hi;
                 mx_lo = fmaxf(mx_lo, v_lo); mx_hi = fmaxf(mx_hi, v_hi);
             }
@@ -709,11 +743,12 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             // A tile is fetched whole.  Rows of keys outside [first_key, pos] belong to nobody (stale rows of
             // an earlier sequence, possibly not finite): their probabilities are zero, but 0 * NaN is NaN, so
             // their value rows are cleared before the product.  Only the first and the last tile have any.
-            const int r_lo = first_key - blk * KB, r_hi = pos - blk * KB;      // rows [r_lo, r_hi] are real
+            const int tile0 = tile_of(blk) * KB;
+            const int r_lo = first_key - tile0, r_hi = pos - tile0, r_keep = EXT ? keep - tile0 : 0;   // rows [r_lo, r_hi] are real, and those below r_keep
             if (r_lo > 0 || r_hi < KB - 1) {
-                for (int i = lane; i < halves * KB * 8; i += 32) {
+                for (int i = lane; i < v_halves * KB * 8; i += 32) {
                     const int h = i / (KB * 8), r = (i >> 3) % KB, c = i & 7;
-                    if (r < r_lo || r > r_hi)
+                    if ((r < r_lo && !(EXT && r < r_keep)) || r > r_hi)
                         asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(sV + h * kHalf + r * 128 + c * 16), "r"(0u) : "memory");
                 }
                 __syncwarp();
@@ -728,7 +763,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         for (int kk = 0; kk < KB / 16; ++kk) {
 #pragma unroll
             for (int n2 = 0; n2 < DMAX / 16; ++n2) {
-                if (n2 * 16 < D) {
+                if (n2 * 16 < DV) {
                     uint32_t v0, v1, v2, v3;
                     const int vrow = kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
                     ldmatrix_x4_trans(sV + kv_offset(vrow, n2 * 2 + (lane >> 4)), v0, v1, v2, v3);
@@ -738,7 +773,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             }
         }
         __syncwarp();
-        if (more && lane == 0) load_tile(&map_v, sV, vbar, blk + NW);
+        if (more && lane == 0) load_tile(&map_v, true, sV, vbar, blk + NW);
         phase ^= 1u;
     }
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
@@ -764,8 +799,8 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         }
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < G * D; i += NW * 32) {
-        const int r = i / D, d = i % D;
+    for (int i = threadIdx.x; i < G * DV; i += NW * 32) {
+        const int r = i / DV, d = i % DV;
         float m = -INFINITY;
 #pragma unroll
         for (int w = 0; w < NW; ++w) m = fmaxf(m, comb[((size_t)w * 16 + r) * kRowF + DMAX]);
@@ -780,12 +815,14 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             }
         }
         const int head = kvh * G + r;
+        const size_t out_row = EXT ? ((size_t)token * p.n_heads + head) * maps + map : (size_t)token * p.n_heads + head;
         if (p.splits == 1) {
             if (p.sink_log2) l += exp2f(p.sink_log2[head] - m);
-            p.out[((size_t)token * p.n_heads + head) * D + d] = __float2bfloat16_rn(acc / l);
+            if (EXT && p.out_f32) p.out_f32[out_row * DV + d] = acc / l;
+            else p.out[out_row * DV + d] = __float2bfloat16_rn(acc / l);
         } else {
-            const size_t slot = ((size_t)token * p.n_heads + head) * p.splits + split;
-            p.part_o[slot * D + d] = acc;
+            const size_t slot = out_row * p.splits + split;
+            p.part_o[slot * DV + d] = acc;
             if (d == 0) { p.part_ml[slot * 2] = m; p.part_ml[slot * 2 + 1] = l; }
         }
     }
@@ -875,6 +912,7 @@ static int launch_attention_mma(const void* q, int q_stride, const void* k_cache
                        float* scratch, long scratch_floats, cudaStream_t stream, int n_pages = 0,
                        int* status = nullptr, const FusedRotary* fz = nullptr, const float* sink_log2 = nullptr,
                        const float* slope_log2 = nullptr) {
+    // (launch_attention_mma_general below is the launcher of the EXT forms)
     MDMA_REQUIRE(attention_mma_supported(n_heads, n_kv_heads, head_dim),
                  "attention_mma: heads %d / kv heads %d / head_dim %d is outside its limits (head_dim a multiple of 16 up to 128, group up to 64)",
                  n_heads, n_kv_heads, head_dim);
@@ -896,6 +934,7 @@ static int launch_attention_mma(const void* q, int q_stride, const void* k_cache
     p.rot_inv_freq = nullptr; p.rotary_dim = 0; p.rot_interleaved = 0;
     p.proj_partial = nullptr; p.proj_splits = 0; p.proj_split_stride = 0; p.proj_width = 0;
     p.k_cache_w = nullptr; p.v_cache_w = nullptr;
+    p.v_dim = head_dim; p.maps = 1; p.rule = {window, 0, 0}; p.cap_log2 = p.cap_rate = 0.f; p.out_f32 = nullptr;
     if (fz != nullptr) {
         MDMA_REQUIRE(max_new == 1 && n_pages > 0 && attention_fused_rotary_supported(n_heads, n_kv_heads, head_dim, page_size, fz->rotary_dim),
                      "attention: the rotary encoding can be done inside the kernel only for single tokens, page sizes that are multiples of 32 and groups up to 16");
@@ -990,5 +1029,89 @@ static int launch_attention_mma(const void* q, int q_stride, const void* k_cache
     }
     return 0;
 }
+
+#ifdef MDMA_ATTENTION_GENERAL
+// The EXT forms.  With splits > 1 the partial sums stay in `scratch`, [token][head][map][split] rows of v_dim floats and
+// then as many (maximum, sum) pairs; the caller merges them (`attention_finish`).  splits == 1: finished rows in `out`
+// (bfloat16) or `out_f32`, [token][head][map].
+static int launch_attention_mma_general(const void* q, int q_stride, const void* k_cache, const void* v_cache, int n_pages,
+                                        const int* seq_start, const int* seq_pos0, const int* seq_slot, const int* page_table,
+                                        int max_pages, int page_size, void* out, float* out_f32, int n_tokens, int n_seqs,
+                                        int max_new, int n_heads, int n_kv_heads, int head_dim, int v_dim, int maps, KeyRule rule,
+                                        float softcap, float scale, int splits, float* scratch, long scratch_floats, int* status,
+                                        const float* sink_log2, const float* slope_log2, cudaStream_t stream) {
+    MDMA_REQUIRE(attention_mma_supported(n_heads, n_kv_heads, head_dim) && attention_mma_supported(n_heads, n_kv_heads, v_dim),
+                 "attention_mma: heads %d / kv heads %d / sizes %d and %d are outside its limits (multiples of 16 up to 128, group up to 64)",
+                 n_heads, n_kv_heads, head_dim, v_dim);
+    MDMA_REQUIRE(rule_ok(rule) && softcap >= 0.f && maps >= 1, "attention_mma: window %d, kept %d, chunk %d, %d maps do not go together",
+                 rule.window, rule.keep_first, rule.chunk, maps);
+    MDMA_REQUIRE(page_table && page_size > 0 && max_pages > 0, "attention_mma: bad cache geometry");
+    MDMA_REQUIRE(q_stride % 8 == 0 && (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) == 0, "attention_mma: rows must be 16-byte aligned");
+    if (splits < 1) splits = 1;
+    MDMA_REQUIRE(n_seqs <= 65535 && (long)n_kv_heads * maps * splits <= 65535, "attention_mma: grid too large");
+    if (n_tokens == 0 || n_seqs == 0) return 0;
+    AttnParams p = {};
+    p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride;
+    p.k_cache = (const __nv_bfloat16*)k_cache; p.v_cache = (const __nv_bfloat16*)v_cache;
+    p.seq_start = seq_start; p.seq_pos0 = seq_pos0; p.seq_slot = seq_slot;
+    p.page_table = page_table; p.max_pages = max_pages; p.page_size = page_size;
+    p.out = (__nv_bfloat16*)out; p.out_f32 = out_f32;
+    p.n_heads = n_heads; p.n_kv_heads = n_kv_heads; p.head_dim = head_dim;
+    p.group = n_heads / n_kv_heads; p.tile_tokens = kRows / p.group; p.window = rule.window; p.splits = splits;
+    p.scale_log2 = scale * 1.4426950408889634f;
+    p.status = status; p.sink_log2 = splits == 1 ? sink_log2 : nullptr; p.slope_log2 = slope_log2;
+    p.v_dim = v_dim; p.maps = maps; p.rule = rule;
+    if (softcap > 0.f) { p.cap_log2 = softcap * 1.4426950408889634f; p.cap_rate = 2.0f * 1.4426950408889634f * scale / softcap; }
+    if (splits > 1) {
+        const long need = (long)n_tokens * n_heads * maps * splits * (v_dim + 2);
+        MDMA_REQUIRE(scratch && scratch_floats >= need, "attention_mma: %d splits need %ld floats of scratch, %ld given", splits, need, scratch_floats);
+        p.part_o = scratch;
+        p.part_ml = scratch + (long)n_tokens * n_heads * maps * splits * v_dim;
+    }
+    const int widest = head_dim > v_dim ? head_dim : v_dim;
+    dim3 grid((max_new + p.tile_tokens - 1) / p.tile_tokens, n_seqs, n_kv_heads * maps * splits);
+    if (max_new == 1 && p.group <= 16 && n_pages > 0 && page_size % kDecodeKeys == 0) {
+        const int kb = (widest <= 64 && page_size % 64 == 0) ? 64 : kDecodeKeys;
+        CUtensorMap mk, mv;
+        if (int rc = make_cache_map(&mk, k_cache, n_pages, page_size, n_kv_heads * maps, head_dim, kb)) return rc;
+        if (int rc = make_cache_map(&mv, v_cache, n_pages, page_size, n_kv_heads, v_dim, kb)) return rc;
+        auto launch = [&](auto kernel, int nw, int dmax) -> int {
+            const int bytes = nw * 2 * kb * dmax * 2 + 16 * dmax * 2 + nw * 16 + 64 + 8 * dmax;
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+            if (e != cudaSuccess) return fail("attention: cannot reserve %d bytes of shared memory: %s", bytes, cudaGetErrorString(e));
+            e = launch_chained(kernel, grid, dim3(nw * 32), bytes, stream, mk, mv, p);
+            if (e != cudaSuccess) return fail("attention: launch failed: %s", cudaGetErrorString(e));
+            return 0;
+        };
+        int sm_count = 0, dev = 0;
+        cudaGetDevice(&dev);
+        cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev);
+        const long blocks = (long)n_seqs * n_kv_heads * maps * splits;
+        const int nw = blocks <= sm_count ? 8 : blocks <= 3l * sm_count ? 4 : blocks <= 5l * sm_count ? 2 : blocks <= 10l * sm_count ? 1 : 4;
+        int rc;
+        if (kb == 64)
+            rc = nw == 8 ? launch(attention_decode_tma_kernel<64, 64, 8, true>, 8, 64)
+               : nw == 4 ? launch(attention_decode_tma_kernel<64, 64, 4, true>, 4, 64)
+               : nw == 2 ? launch(attention_decode_tma_kernel<64, 64, 2, true>, 2, 64)
+                         : launch(attention_decode_tma_kernel<64, 64, 1, true>, 1, 64);
+        else                     // (narrow heads on pages of 32 use the wide tiles too: the second half is not loaded)
+            rc = nw == 8 ? launch(attention_decode_tma_kernel<128, kDecodeKeys, 8, true>, 8, 128)
+               : nw == 4 ? launch(attention_decode_tma_kernel<128, kDecodeKeys, 4, true>, 4, 128)
+               : nw == 2 ? launch(attention_decode_tma_kernel<128, kDecodeKeys, 2, true>, 2, 128)
+                         : launch(attention_decode_tma_kernel<128, kDecodeKeys, 1, true>, 1, 128);
+        if (rc) return rc;
+    } else if (widest <= 64) {
+        constexpr int bytes = 5 * kRows * 64 * 2;
+        cudaFuncSetAttribute(attention_mma_kernel<64, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+        launch_chained(attention_mma_kernel<64, true>, grid, dim3(kAttnThreads), bytes, stream, p);
+    } else {
+        constexpr int bytes = 5 * kRows * 128 * 2;
+        cudaFuncSetAttribute(attention_mma_kernel<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+        launch_chained(attention_mma_kernel<128, true>, grid, dim3(kAttnThreads), bytes, stream, p);
+    }
+    MDMA_LAUNCH_OK("attention_mma (general)");
+    return 0;
+}
+#endif
 
 }  // namespace mdma

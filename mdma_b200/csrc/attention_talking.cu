@@ -4,7 +4,10 @@
 // k head is (if asked) divided by its root mean square, x / sqrt(mean(x^2) + eps), and multiplied by a weight vector
 // shared by all heads, THEN its first `rotary_dim` numbers are turned by the token's position (pairs (2i, 2i+1) or
 // (i, i + rotary_dim/2), cos and sin times `magnitude`).  q is written back in place; k and v go to the token's row
-// of the paged cache (value heads may have a size of their own).
+// of the paged cache (value heads may have a size and a number of their own, and may be the key heads' projections:
+// v_col == k_col).  With `v_norm` every value head is divided by its root mean square, without a weight.  With `splits`
+// > 0 the projection row is the sum of that many float partial rows of `row_width` numbers (a K-split product not yet
+// added up); the columns from `tail_col` on are then summed up too and stored in the row.
 //
 // talking_attention: raw scores s_g = (q_g . k_kv(g)) * scale of ALL query heads g for a key are mixed by a matrix,
 // s'_h = sum_g T[h, g] s_g, before the softmax of head h; a query at position p sees the keys up to p; the
@@ -27,7 +30,7 @@
 
 namespace mdma {
 
-constexpr int kTalkMaxDim = 256, kTalkMaxHeads = 32, kPrepWarpsT = 4;
+constexpr int kTalkMaxDim = 256, kTalkMaxHeads = 32, kPrepWarpsT = 4, kPrepTailCols = 128;
 
 __device__ __forceinline__ float talk_weight(const void* w, int dtype, int e) {
     if (w == nullptr) return 1.0f;
@@ -41,7 +44,8 @@ qk_norm_rotate_kernel(T* __restrict__ proj, int row_stride, int k_col, int v_col
                       float magnitude, const void* __restrict__ q_w, const void* __restrict__ k_w, int w_dtype, int norm,
                       float eps, T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ page_table,
                       int max_pages, int page_size, int n_heads, int n_kv_heads, int dim, int v_dim, int rotary_dim,
-                      int interleaved, int write_kv) {
+                      int interleaved, int write_kv, int n_v_heads, int v_norm, const float* __restrict__ partial, int splits,
+                      size_t split_stride, int row_width, int tail_col) {
     chain_release();
     chain_wait();
     __shared__ float sines[kTalkMaxDim / 2], cosines[kTalkMaxDim / 2];
@@ -57,29 +61,55 @@ qk_norm_rotate_kernel(T* __restrict__ proj, int row_stride, int k_col, int v_col
     }
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int total = n_heads + (write_kv ? 2 * n_kv_heads : 0);
+    const int heads_total = n_heads + (write_kv ? n_kv_heads + n_v_heads : 0);
     const int head = blockIdx.y * kPrepWarpsT + warp;
-    if (head >= total) return;
     T* row = proj + (size_t)t * row_stride;
+    const float* part = partial + (size_t)t * row_width;
+    auto input = [&](int col) -> float {
+        if (splits == 0) return to_float(row[col]);
+        float x = 0.f;
+#pragma unroll 4
+        for (int p = 0; p < splits; ++p) x += part[(size_t)p * split_stride + col];
+        return x;
+    };
+    if (head >= heads_total) {                          // columns behind the heads: completed only
+        if (splits == 0) return;
+        for (int i = 0, c = tail_col + (head - heads_total) * kPrepTailCols + lane; i < kPrepTailCols / 32; ++i, c += 32)
+            if (c < row_width) row[c] = from_float<T>(input(c));
+        return;
+    }
     size_t cache_row = 0;
     if (write_kv) {
         const int slot = seq_slot[tok_seq[t]];
-        cache_row = ((size_t)page_table[(size_t)slot * max_pages + pos / page_size] * page_size + (size_t)(pos % page_size)) * n_kv_heads;
+        cache_row = (size_t)page_table[(size_t)slot * max_pages + pos / page_size] * page_size + (size_t)(pos % page_size);
     }
-    if (head >= n_heads + n_kv_heads) {                 // a value head: copied as it is
-        const int g = head - n_heads - n_kv_heads;
-        const T* src = row + v_col + (size_t)g * v_dim;
-        T* dst = v_cache + (cache_row + g) * v_dim;
-        for (int d = lane; d < v_dim; d += 32) dst[d] = src[d];
+    if (head >= n_heads + n_kv_heads) {                 // a value head
+        const int g = head - n_heads - n_kv_heads, c0 = v_col + g * v_dim;
+        T* dst = v_cache + (cache_row * n_v_heads + g) * v_dim;
+        if (!v_norm) {
+            for (int d = lane; d < v_dim; d += 32) dst[d] = from_float<T>(input(c0 + d));
+            return;
+        }
+        float x[kTalkMaxDim / 32], sq = 0.f;
+#pragma unroll
+        for (int i = 0; i < kTalkMaxDim / 32; ++i) {
+            const int d = lane + 32 * i;
+            x[i] = d < v_dim ? input(c0 + d) : 0.f;
+            sq = fmaf(x[i], x[i], sq);
+        }
+        const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)v_dim + eps);
+#pragma unroll
+        for (int i = 0; i < kTalkMaxDim / 32; ++i)
+            if (lane + 32 * i < v_dim) dst[lane + 32 * i] = from_float<T>(x[i] * inv);
         return;
     }
     const bool is_q = head < n_heads;
-    T* src = is_q ? row + (size_t)head * dim : row + k_col + (size_t)(head - n_heads) * dim;
-    T* dst = is_q ? src : k_cache + (cache_row + (head - n_heads)) * dim;
+    const int c0 = is_q ? head * dim : k_col + (head - n_heads) * dim;
+    T* dst = is_q ? row + c0 : k_cache + (cache_row * n_kv_heads + (head - n_heads)) * dim;
     float* v = rows[warp];
     float sq = 0.f;
     for (int d = lane; d < dim; d += 32) {
-        v[d] = to_float(src[d]);
+        v[d] = input(c0 + d);
         sq = fmaf(v[d], v[d], sq);
     }
     if (norm) {
@@ -382,20 +412,26 @@ int mdma_qk_norm_rotate(void* proj, int dtype, int row_stride, int k_col, int v_
                         const int* seq_slot, const float* inv_freq, float magnitude, const void* q_w, const void* k_w,
                         int w_dtype, int norm, float eps, void* k_cache, void* v_cache, const int* page_table,
                         int max_pages, int page_size, int n_tokens, int n_heads, int n_kv_heads, int dim, int v_dim,
-                        int rotary_dim, int interleaved, int write_kv, cudaStream_t stream) {
-    MDMA_REQUIRE(n_tokens >= 0 && n_heads > 0 && n_kv_heads >= 0, "qk_norm_rotate: bad sizes");
+                        int rotary_dim, int interleaved, int write_kv, int n_v_heads, int v_norm, const float* partial,
+                        int splits, long split_stride, int row_width, int tail_col, cudaStream_t stream) {
+    MDMA_REQUIRE(n_tokens >= 0 && n_heads >= 0 && n_kv_heads >= 0 && n_v_heads >= 0, "qk_norm_rotate: bad sizes");
+    MDMA_REQUIRE(splits >= 0 && (splits == 0 || (partial && n_heads > 0 && tail_col >= 0 && row_width > 0)), "qk_norm_rotate: partial sums need a pointer and every head");
+    MDMA_REQUIRE(!v_norm || v_dim <= kTalkMaxDim, "qk_norm_rotate: value heads of %d are beyond the limit %d", v_dim, kTalkMaxDim);
     MDMA_REQUIRE(dim > 0 && dim <= kTalkMaxDim && v_dim > 0, "qk_norm_rotate: head size %d is beyond the limit %d", dim, kTalkMaxDim);
     MDMA_REQUIRE(rotary_dim >= 0 && rotary_dim % 2 == 0 && rotary_dim <= dim, "qk_norm_rotate: rotary_dim %d does not fit head size %d", rotary_dim, dim);
     MDMA_REQUIRE(rotary_dim == 0 || inv_freq, "qk_norm_rotate: a rotation needs its frequencies");
     MDMA_REQUIRE(w_dtype == kF32 || w_dtype == kBF16, "qk_norm_rotate: unknown weight dtype %d", w_dtype);
     MDMA_REQUIRE(!write_kv || (page_table && k_cache && v_cache && page_size > 0 && max_pages > 0), "qk_norm_rotate: no cache pages");
     if (n_tokens == 0) return 0;
-    const int total = n_heads + (write_kv ? 2 * n_kv_heads : 0);
+    const int tail = splits > 0 && tail_col < row_width ? (row_width - tail_col + kPrepTailCols - 1) / kPrepTailCols : 0;
+    const int total = n_heads + (write_kv ? n_kv_heads + n_v_heads : 0) + tail;
+    if (total == 0) return 0;
     MDMA_DISPATCH_DTYPE(dtype, T,
         launch_chained(qk_norm_rotate_kernel<T>, dim3(n_tokens, (total + kPrepWarpsT - 1) / kPrepWarpsT), dim3(kPrepWarpsT * 32),
                        0, stream, (T*)proj, row_stride, k_col, v_col, tok_seq, tok_pos, seq_slot, inv_freq, magnitude, q_w, k_w,
                        w_dtype, norm, eps, (T*)k_cache, (T*)v_cache, page_table, max_pages, page_size, n_heads, n_kv_heads,
-                       dim, v_dim, rotary_dim, interleaved, write_kv));
+                       dim, v_dim, rotary_dim, interleaved, write_kv, n_v_heads, v_norm, partial, splits, (size_t)split_stride,
+                       row_width, tail_col));
     MDMA_LAUNCH_OK("qk_norm_rotate");
     return 0;
 }

@@ -22,6 +22,11 @@
 // are the softmax.  Two blocks fit an SM, so one block's softmax runs under the other's MMAs.
 // Every wait is bounded.
 // Limits: head_dim a multiple of 16 up to 128, group size up to 128, page size a multiple of 64.
+//
+// EXT is the same kernel with further options: value heads of a size of their own, which keys a row sees (`KeyRule`:
+// kept first tokens, chunks; the key blocks before the gap and behind it are walked as one list), a soft cap on the
+// scores, several maps per head (query heads [head][map], key heads [kv head][map], one value head per kv head; a map is
+// a row tile of its own), float results.
 #include <cuda_fp16.h>
 
 #include <mutex>
@@ -43,7 +48,16 @@ struct AttnTcParams {
     int* status;
     const float* sink_log2;       // [n_heads] or null: 2^(sink_log2[head] - reference) joins the row's denominator once
     const float* slope_log2;      // [n_heads] or null: slope_log2[head] * (query position - key position) is taken off every score
+    // EXT only
+    int v_dim, maps;
+    KeyRule rule;
+    float cap_raw, cap_rate;      // a soft cap c on raw scores s: cap_raw tanh(s cap_rate' ) with cap_raw = c / scale; cap_rate = 2 scale log2(e) / c; 0: none
+    float* out_f32;               // results as float rows instead of `out`
 };
+// cap_raw * tanh(x), x = s * cap_rate / (2 log2(e)), as 1 - 2 / (1 + e^(2 x))
+__device__ __forceinline__ float capped_raw(float s, float cap_raw, float cap_rate) {
+    return fmaf(-2.0f * cap_raw, __fdividef(1.0f, 1.0f + ptx::ex2_approx(s * cap_rate)), cap_raw);
+}
 
 // shared memory map (bytes), all tiles 1024-aligned:
 //   Q: 2 halves x [128 rows x 128 B]           32 KB
@@ -56,6 +70,7 @@ constexpr int kSmemQ = 0, kSmemK = 2 * kQHalf, kSmemV = kSmemK + kKvStages * 2 *
               kSmemXch = kSmemBars + 256,          // the two halves of a row exchange their maxima here: 2 x 128 halves (16-bit)
               kAttnTcSmem = kSmemXch + 512;        // 112.75 KB: two blocks per SM (113 KB each at most)
 
+template <bool EXT>
 __global__ void __launch_bounds__(kTcThreadsA, 2)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const AttnTcParams p) {
@@ -78,7 +93,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 
     chain_release();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int seq = blockIdx.y, kvh = blockIdx.x;
+    const int seq = blockIdx.y;
+    const int key_head = blockIdx.x, maps = EXT ? p.maps : 1;      // key_head = kvh * maps + map
+    const int kvh = EXT ? key_head / maps : key_head, map = EXT ? key_head % maps : 0;
     if (threadIdx.x == 0) {
         if (base & 1023u) *abort_flag = 1;          // the tiles need 1024-byte alignment (checked again below)
         ptx::mbar_init(q_full, 1);
@@ -113,18 +130,22 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int n_tok = active ? min(p.tile_tokens, n_new - tok0) : 0;
     const int pos0 = p.seq_pos0[seq] + tok0;
     const int last_pos = pos0 + n_tok - 1;
-    const int D = p.head_dim, G = p.group;
-    const int first_key = p.window > 0 ? max(0, pos0 + 1 - p.window) : 0;
+    const int D = p.head_dim, G = p.group, DV = EXT ? p.v_dim : D;
+    const int first_key = EXT ? rule_first(p.rule, pos0) : p.window > 0 ? max(0, pos0 + 1 - p.window) : 0;
     const int b0 = first_key / kTcKeys, b1 = active ? last_pos / kTcKeys + 1 : b0;
-    const int nb = b1 - b0;
-    const int halves = (D + 63) / 64;
+    // blocks with kept first tokens in front of the window's: block i of the walk is block `block_of(i)` of the sequence
+    const int keep = EXT ? p.rule.keep_first : 0;
+    const int kb = EXT ? min((keep + kTcKeys - 1) / kTcKeys, b0) : 0;
+    auto block_of = [&](int i) { return EXT && i < kb ? i : b0 + i - kb; };
+    const int nb = active ? kb + b1 - b0 : 0;
+    const int halves = (D + 63) / 64, v_halves = EXT ? (DV + 63) / 64 : halves;
 
     if (active && warp == 0 && lane == 0) {
         // ---- TMA producer ---------------------------------------------------------
         const int* pages = p.page_table + (size_t)p.seq_slot[seq] * p.max_pages;
         ptx::mbar_expect_tx(q_full, halves * G * p.tile_tokens * 128);      // the box is G x tile_tokens rows of 128 bytes
         for (int h = 0; h < halves; ++h)
-            ptx::tma_load_4d(base + kSmemQ + h * kQHalf, &map_q, q_full, h * 64, kvh * G, row0_seq + tok0, 0);
+            ptx::tma_load_4d(base + kSmemQ + h * kQHalf, &map_q, q_full, h * 64, kvh * G, row0_seq + tok0, map);
         // S is computed for two key blocks at once (below), so the two key stages are filled and freed
         // together; a value stage is free after its own P V product.  The loads are issued in the order in
         // which their stages come free: K0 K1 V0 V1 | K2 K3 (S of blocks 0,1 done) V2 (P V 0 done) |
@@ -135,21 +156,21 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             if (i >= nb) return true;
             const int s = i % kKvStages;
             if (!ptx::mbar_wait(k_empty(s), ((i / kKvStages) & 1) ^ 1, abort_flag)) return false;
-            const int key0 = (b0 + i) * kTcKeys;
+            const int key0 = block_of(i) * kTcKeys;
             const int page = pages[key0 / p.page_size], row = key0 % p.page_size;
             ptx::mbar_expect_tx(k_full(s), halves * kKvHalf);
             for (int h = 0; h < halves; ++h)
-                ptx::tma_load_4d(base + kSmemK + (h * kKvStages + s) * kKvHalf, &map_k, k_full(s), h * 64, kvh, row, page);
+                ptx::tma_load_4d(base + kSmemK + (h * kKvStages + s) * kKvHalf, &map_k, k_full(s), h * 64, key_head, row, page);
             return true;
         };
         auto load_v = [&](int i) -> bool {
             if (i >= nb) return true;
             const int s = i % kKvStages;
             if (!ptx::mbar_wait(v_empty(s), ((i / kKvStages) & 1) ^ 1, abort_flag)) return false;
-            const int key0 = (b0 + i) * kTcKeys;
+            const int key0 = block_of(i) * kTcKeys;
             const int page = pages[key0 / p.page_size], row = key0 % p.page_size;
-            ptx::mbar_expect_tx(v_full(s), halves * kKvHalf);
-            for (int h = 0; h < halves; ++h)
+            ptx::mbar_expect_tx(v_full(s), v_halves * kKvHalf);
+            for (int h = 0; h < v_halves; ++h)
                 ptx::tma_load_4d(base + kSmemV + (s * 2 + h) * kKvHalf, &map_v, v_full(s), h * 64, kvh, row, page);
             return true;
         };
@@ -188,7 +209,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         }
     } else if (active && warp == 10 && lane == 0) {
         // ---- second MMA issuer: O += P(i) V(i), K dimension = keys ----------------------
-        const uint32_t idesc_o = ptx::idesc_bf16_f32_ex(kTcRows, D, 1);
+        const uint32_t idesc_o = ptx::idesc_bf16_f32_ex(kTcRows, DV, 1);
         for (int i = 0; i < nb; ++i) {
             const int s = i % kKvStages;
             if (!(ptx::mbar_wait(v_full(s), (i / kKvStages) & 1, abort_flag) && ptx::mbar_wait(p_ready, i & 1, abort_flag))) break;
@@ -210,7 +231,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const int t = r / G, g = r % G;
         const bool row_valid = t < n_tok;
         const int pos = pos0 + (row_valid ? t : n_tok - 1);
-        const int win = p.window > 0 ? pos + 1 - p.window : 0;
+        const int win = EXT ? rule_first(p.rule, pos) : p.window > 0 ? pos + 1 - p.window : 0;
         // the penalty on distance in the units of the raw scores (they are multiplied by scale_log2 later)
         const float slope_raw = p.slope_log2 != nullptr ? p.slope_log2[kvh * G + g] / p.scale_log2 : 0.f;
         float m_ref = -INFINITY, l = 0.f;                     // reference maximum (log2 domain), this half's running sum
@@ -237,7 +258,11 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             ptx::tmem_load_wait();
             ptx::tc_fence_before_sync();
             if (i & 1) ptx::mbar_arrive(s_read);              // both blocks of the pair are in registers: S may be overwritten
-            const int key0 = (b0 + i) * kTcKeys + half * 32;
+            const int key0 = block_of(i) * kTcKeys + half * 32;
+            if (EXT && p.cap_raw > 0.f) {
+#pragma unroll
+                for (int j = 0; j < 32; ++j) sv[j] = capped_raw(sv[j], p.cap_raw, p.cap_rate);
+            }
             if (slope_raw != 0.f) {
 #pragma unroll
                 for (int j = 0; j < 32; ++j) sv[j] -= slope_raw * (float)(pos - (key0 + j));
@@ -246,7 +271,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             if (need_mask) {
 #pragma unroll
                 for (int j = 0; j < 32; ++j)
-                    if (key0 + j > pos || key0 + j < win) sv[j] = -INFINITY;
+                    if (key0 + j > pos || (key0 + j < win && !(EXT && key0 + j < keep))) sv[j] = -INFINITY;
             }
             float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -285,7 +310,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 if (__any_sync(0xffffffffu, moved)) {          // rare: rescale this warp's rows of O (its column chunks)
 #pragma unroll
                     for (int c = 0; c < 4; ++c) {
-                        if ((c & 1) == half && c * 32 < D) {
+                        if ((c & 1) == half && c * 32 < DV) {
                             float v[32];
                             ptx::tmem_load_32_nowait(tmem_o + lane_base + c * 32, v);
                             ptx::tmem_load_wait();
@@ -302,15 +327,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 // window) belong to nobody: stale rows of an earlier sequence, possibly not finite.  Their
                 // probabilities are zero, but 0 * NaN is NaN, so the rows are cleared in shared memory before
                 // the product reads them.  Only the first and the last key block of a tile have any.
-                const int kb0 = (b0 + i) * kTcKeys;
-                if (kb0 + kTcKeys - 1 > last_pos || kb0 < first_key) {
+                const int kb0 = block_of(i) * kTcKeys;
+                if (kb0 + kTcKeys - 1 > last_pos || kb0 < first_key) {      // (with kept tokens: also their last block)
                     const int vs = i % kKvStages;
                     ok = __all_sync(0xffffffffu, ptx::mbar_wait(v_full(vs), (i / kKvStages) & 1, abort_flag));
                     if (!ok) break;
                     const int tid = (warp - 2) * 32 + lane;
-                    for (int e = tid; e < halves * kTcKeys * 8; e += 256) {
+                    for (int e = tid; e < v_halves * kTcKeys * 8; e += 256) {
                         const int h = e / (kTcKeys * 8), kr = (e >> 3) % kTcKeys, c = e & 7;
-                        if (kb0 + kr > last_pos || kb0 + kr < first_key)
+                        if (kb0 + kr > last_pos || (kb0 + kr < first_key && !(EXT && kb0 + kr < keep)))
                             *reinterpret_cast<uint4*>(base_ptr + kSmemV + (vs * 2 + h) * kKvHalf + kr * 128 + c * 16) = make_uint4(0u, 0u, 0u, 0u);
                     }
                 }
@@ -338,17 +363,27 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             if (half == 1) total = x[r];
             if (p.sink_log2 != nullptr) total += exp2f(p.sink_log2[kvh * G + g] - m_ref);
             const float inv = 1.0f / total;
-            __nv_bfloat16* dst = p.out + ((size_t)(row0_seq + tok0 + (row_valid ? t : 0)) * p.n_heads + kvh * G + g) * D;
+            const size_t out_row = EXT ? ((size_t)(row0_seq + tok0 + (row_valid ? t : 0)) * p.n_heads + kvh * G + g) * maps + map
+                                       : (size_t)(row0_seq + tok0 + (row_valid ? t : 0)) * p.n_heads + kvh * G + g;
+            __nv_bfloat16* dst = p.out + out_row * DV;
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
-                if ((c & 1) == half && c * 32 < D) {
+                if ((c & 1) == half && c * 32 < DV) {
                     float v[32];
                     ptx::tmem_load_32_nowait(tmem_o + lane_base + c * 32, v);
                     ptx::tmem_load_wait();
-                    if (row_valid) {
+                    if (EXT && p.out_f32 != nullptr) {
+                        if (row_valid) {
+                            float* fd = p.out_f32 + out_row * DV + c * 32;
+#pragma unroll
+                            for (int q = 0; q < 8; ++q)
+                                if (c * 32 + q * 4 < DV)
+                                    *reinterpret_cast<float4*>(fd + q * 4) = make_float4(v[4 * q] * inv, v[4 * q + 1] * inv, v[4 * q + 2] * inv, v[4 * q + 3] * inv);
+                        }
+                    } else if (row_valid) {
 #pragma unroll
                         for (int q = 0; q < 4; ++q) {
-                            if (c * 32 + q * 8 < D) {
+                            if (c * 32 + q * 8 < DV) {
                                 uint32_t w[4];
 #pragma unroll
                                 for (int j = 0; j < 4; ++j) {
@@ -417,12 +452,21 @@ int mdma_attention_tc_supported(int n_heads, int n_kv_heads, int head_dim, int p
     return (head_dim % 16 == 0 && head_dim >= 16 && head_dim <= 128 && g <= kTcRows && page_size % kTcKeys == 0) ? 1 : 0;
 }
 
+// What the kernel's EXT form takes beside the rest.
+struct AttnTcExt {
+    int v_dim, maps;
+    KeyRule rule;
+    float softcap;
+    float* out_f32;
+};
+
 // q: rows of the fused projection [tokens_cap, row_width], queries first; caches [pages, page_size, kv_heads, head_dim].
 static int attention_tc_run(const void* q, int q_stride, int q_rows_cap, const void* k_cache, const void* v_cache,
                       int n_pages, const int* seq_start, const int* seq_pos0, const int* seq_slot,
                       const int* page_table, int max_pages, int page_size, void* out, int n_tokens, int n_seqs,
                       int max_new, int n_heads, int n_kv_heads, int head_dim, int window, float scale,
-                      int* status, const float* sink_log2, cudaStream_t stream, const float* slope_log2 = nullptr) {
+                      int* status, const float* sink_log2, cudaStream_t stream, const float* slope_log2 = nullptr,
+                      const AttnTcExt* ext = nullptr) {
     MDMA_REQUIRE(mdma_attention_tc_supported(n_heads, n_kv_heads, head_dim, page_size),
                  "attention_tc: heads %d / kv heads %d / head_dim %d / page %d is outside its limits", n_heads, n_kv_heads, head_dim, page_size);
     MDMA_REQUIRE(q_stride % 8 == 0 && ((uintptr_t)q & 15) == 0, "attention_tc: query rows must be 16-byte aligned");
@@ -436,29 +480,44 @@ static int attention_tc_run(const void* q, int q_stride, int q_rows_cap, const v
     p.out = (__nv_bfloat16*)out; p.n_heads = n_heads; p.n_kv_heads = n_kv_heads; p.head_dim = head_dim;
     p.group = G; p.tile_tokens = kTcRows / G; p.window = window; p.n_tokens = n_tokens;
     p.scale_log2 = scale * 1.4426950408889634f; p.status = status; p.sink_log2 = sink_log2; p.slope_log2 = slope_log2;
+    p.v_dim = head_dim; p.maps = 1; p.rule = {window, 0, 0}; p.cap_raw = p.cap_rate = 0.f; p.out_f32 = nullptr;
+    if (ext != nullptr) {
+        p.v_dim = ext->v_dim; p.maps = ext->maps; p.rule = ext->rule; p.out_f32 = ext->out_f32;
+        if (ext->softcap > 0.f) {
+            p.cap_raw = ext->softcap / scale;
+            p.cap_rate = 2.0f * 1.4426950408889634f * scale / ext->softcap;
+        }
+    }
+    const int maps = p.maps, v_dim = p.v_dim;
     CUtensorMap mq, mk, mv;
     {   // queries: [tokens][heads][head_dim] inside rows of q_stride elements; box = 64 x G x tile_tokens
-        const uint64_t dims[4] = {(uint64_t)head_dim, (uint64_t)n_heads, (uint64_t)n_tokens, 1};
-        const uint64_t strides[3] = {(uint64_t)head_dim * 2, (uint64_t)q_stride * 2, (uint64_t)q_stride * 2 * (uint64_t)q_rows_cap};
+        // (several maps: heads lie `maps` head sizes apart, the last coordinate is the map)
+        const uint64_t dims[4] = {(uint64_t)head_dim, (uint64_t)n_heads, (uint64_t)n_tokens, (uint64_t)maps};
+        const uint64_t strides[3] = {(uint64_t)maps * head_dim * 2, (uint64_t)q_stride * 2,
+                                     maps > 1 ? (uint64_t)head_dim * 2 : (uint64_t)q_stride * 2 * (uint64_t)q_rows_cap};
         const uint32_t box[4] = {64, (uint32_t)G, (uint32_t)p.tile_tokens, 1};
         if (int rc = make_map_4d(&mq, q, dims, strides, box)) return rc;
     }
     {
-        const uint64_t dims[4] = {(uint64_t)head_dim, (uint64_t)n_kv_heads, (uint64_t)page_size, (uint64_t)n_pages};
-        const uint64_t strides[3] = {(uint64_t)head_dim * 2, (uint64_t)n_kv_heads * head_dim * 2,
-                                     (uint64_t)page_size * n_kv_heads * head_dim * 2};
-        const uint32_t box[4] = {64, 1, (uint32_t)kTcKeys, 1};
-        if (int rc = make_map_4d(&mk, k_cache, dims, strides, box)) return rc;
-        if (int rc = make_map_4d(&mv, v_cache, dims, strides, box)) return rc;
+        auto cache_map = [&](CUtensorMap* out, const void* cache, int heads, int dim) -> int {
+            const uint64_t dims[4] = {(uint64_t)dim, (uint64_t)heads, (uint64_t)page_size, (uint64_t)n_pages};
+            const uint64_t strides[3] = {(uint64_t)dim * 2, (uint64_t)heads * dim * 2, (uint64_t)page_size * heads * dim * 2};
+            const uint32_t box[4] = {64, 1, (uint32_t)kTcKeys, 1};
+            return make_map_4d(out, cache, dims, strides, box);
+        };
+        if (int rc = cache_map(&mk, k_cache, n_kv_heads * maps, head_dim)) return rc;
+        if (int rc = cache_map(&mv, v_cache, n_kv_heads, v_dim)) return rc;
     }
     static bool once = false;
     if (!once) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnTcSmem);
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnTcSmem);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnTcSmem);
         if (e != cudaSuccess) return fail("attention_tc: cannot reserve %d bytes of shared memory: %s", kAttnTcSmem, cudaGetErrorString(e));
         once = true;
     }
-    dim3 grid(n_kv_heads, n_seqs, (max_new + p.tile_tokens - 1) / p.tile_tokens);
-    cudaError_t e = launch_chained(attention_tc_kernel, grid, dim3(kTcThreadsA), kAttnTcSmem, stream, mq, mk, mv, p);
+    dim3 grid(n_kv_heads * maps, n_seqs, (max_new + p.tile_tokens - 1) / p.tile_tokens);
+    cudaError_t e = ext != nullptr ? launch_chained(attention_tc_kernel<true>, grid, dim3(kTcThreadsA), kAttnTcSmem, stream, mq, mk, mv, p)
+                                   : launch_chained(attention_tc_kernel<false>, grid, dim3(kTcThreadsA), kAttnTcSmem, stream, mq, mk, mv, p);
     if (e != cudaSuccess) return fail("attention_tc: launch failed: %s", cudaGetErrorString(e));
     return 0;
 }
@@ -493,6 +552,23 @@ int mdma_attention_tc_distance(const void* q, int q_stride, int q_rows_cap, cons
     return attention_tc_run(q, q_stride, q_rows_cap, k_cache, v_cache, n_pages, seq_start, seq_pos0, seq_slot, page_table,
                             max_pages, page_size, out, n_tokens, n_seqs, max_new, n_heads, n_kv_heads, head_dim, window,
                             scale, status, sink_log2, stream, slope_log2);
+}
+
+// The same with everything the EXT form takes: value heads of v_dim numbers, `maps` maps per head, a `KeyRule`, a soft
+// cap, and with `out_f32` float rows [tokens][heads][maps][v_dim] instead of bfloat16 ones.
+int mdma_attention_tc_general(const void* q, int q_stride, int q_rows_cap, const void* k_cache, const void* v_cache,
+                              int n_pages, const int* seq_start, const int* seq_pos0, const int* seq_slot,
+                              const int* page_table, int max_pages, int page_size, void* out, float* out_f32, int n_tokens,
+                              int n_seqs, int max_new, int n_heads, int n_kv_heads, int head_dim, int v_dim, int maps,
+                              int window, int keep_first, int chunk, float softcap, float scale, int* status,
+                              const float* sink_log2, const float* slope_log2, cudaStream_t stream) {
+    const AttnTcExt ext = {v_dim, maps, {window, keep_first, chunk}, softcap, out_f32};
+    MDMA_REQUIRE(rule_ok(ext.rule) && softcap >= 0.f && maps >= 1 && v_dim % 16 == 0 && v_dim >= 16 && v_dim <= 128,
+                 "attention_tc: value heads of %d, %d maps, window %d, kept %d, chunk %d are outside its limits", v_dim, maps, window, keep_first, chunk);
+    MDMA_REQUIRE(n_kv_heads * maps <= 65535, "attention_tc: grid too large");
+    return attention_tc_run(q, q_stride, q_rows_cap, k_cache, v_cache, n_pages, seq_start, seq_pos0, seq_slot, page_table,
+                            max_pages, page_size, out, n_tokens, n_seqs, max_new, n_heads, n_kv_heads, head_dim, window,
+                            scale, status, sink_log2, stream, slope_log2, &ext);
 }
 
 }  // extern "C"

@@ -143,6 +143,21 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
     return total;
 }
 
+// Which keys a query at position i sees, j <= i always: all of them; with `window` > 0 those with i - j < window, and with
+// `keep_first` also those with j < keep_first; with `chunk` > 0 (then no window) those of i's own chunk,
+// j / chunk == i / chunk.
+struct KeyRule {
+    int window, keep_first, chunk;
+};
+// the first key a query at `pos` sees, apart from the kept first ones
+__device__ __forceinline__ int rule_first(const KeyRule& r, int pos) {
+    if (r.chunk > 0) return pos / r.chunk * r.chunk;
+    return r.window > 0 ? max(0, pos + 1 - r.window) : 0;
+}
+static inline int rule_ok(const KeyRule& r) {
+    return r.window >= 0 && r.keep_first >= 0 && r.chunk >= 0 && (r.chunk == 0 || (r.window == 0 && r.keep_first == 0));
+}
+
 }  // namespace mdma
 
 // Dispatch on an element type code.

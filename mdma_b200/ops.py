@@ -526,15 +526,20 @@ def attention_distance_tiled_fits(n_heads: int, n_kv_heads: int, dim: int, v_dim
 
 def attention_distance(q, k_cache, v_cache, ctx, page_table, max_pages: int, page_size: int, slopes, gate, out,
                        n_heads: int, n_kv_heads: int, dim: int, v_dim: int, window: int, scale: float,
-                       tiled: bool = False, sinks=None, gate_heads: bool = False, out_scale: float = 1.0) -> None:
+                       tiled: bool = False, sinks=None, gate_heads: bool = False, out_scale: float = 1.0,
+                       keep_first: int = 0, chunk: int = 0, softcap: float = 0.0, maps: int = 1) -> None:
     """Softmax attention with score (q.k) * scale - slopes[h] * distance over the paged cache; q: rows whose first
     n_heads * dim columns are the queries; `gate` (rows of n_heads * v_dim, optional): the result is multiplied by
     its sigmoid; out [T, n_heads * v_dim].  `tiled`: the kernel that stages keys and values per tile of query rows.
     `sinks` [n_heads] floats: exp(sink) joins each head's normaliser once; `gate_heads`: the gate has one number per
-    head (rows of n_heads); `out_scale` multiplies the result."""
+    head (rows of n_heads); `out_scale` multiplies the result.  The kernel that is not tiled also takes: `keep_first`, with
+    a window the first tokens stay visible; `chunk`, a query sees the keys of its own chunk of positions only; `softcap` c,
+    c tanh(. / c) on the scores before the penalty; `maps` m, query heads [head][map] and key heads [kv head][map] with one
+    value head per kv head, results [head][map]; `out` as float rows whatever the queries' dtype."""
     _need_cuda(q, k_cache, v_cache, page_table, slopes, gate, out)
-    assert q.stride(1) == 1 and out.is_contiguous() and out.dtype == q.dtype == k_cache.dtype == v_cache.dtype
-    assert out.shape[1] == n_heads * v_dim and out.shape[0] >= ctx.n_tokens
+    assert q.stride(1) == 1 and out.is_contiguous() and q.dtype == k_cache.dtype == v_cache.dtype
+    assert out.dtype in (q.dtype, torch.float32)
+    assert out.shape[1] == n_heads * maps * v_dim and out.shape[0] >= ctx.n_tokens
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == n_heads and slopes.is_contiguous())
     assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape[1] >= (n_heads if gate_heads else n_heads * v_dim))
     assert sinks is None or (sinks.is_cuda and sinks.dtype == torch.float32 and sinks.numel() == n_heads and sinks.is_contiguous())
@@ -543,7 +548,8 @@ def attention_distance(q, k_cache, v_cache, ctx, page_table, max_pages: int, pag
           _ptr(page_table), _i(max_pages), _i(page_size), _ptr(slopes), _ptr(gate),
           _i(gate.stride(0) if gate is not None else 0), _ptr(out), _i(ctx.n_tokens), _i(ctx.n_seqs), _i(ctx.max_new),
           _i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim), _i(window), _f(scale), _i(int(tiled)), _ptr(sinks),
-          _i(int(gate_heads)), _f(out_scale), _stream())
+          _i(int(gate_heads)), _f(out_scale), _i(keep_first), _i(chunk), _f(softcap), _i(maps),
+          _i(int(out.dtype == torch.float32)), _stream())
 
 
 # ---- routed feed-forward (csrc/routed_ffn.cu) -----------------------------------------------------------------------
@@ -797,10 +803,17 @@ def rotate_heads(q, n_heads: int, head_pitch: int, offset: int, rotary_dim: int,
 def qk_norm_rotate(proj, k_col: int, v_col: int, tok_seq, tok_pos, seq_slot, inv_freq, magnitude: float, q_w, k_w,
                    norm: bool, eps: float, k_cache, v_cache, page_table, max_pages: int, page_size: int, n_tokens: int,
                    n_heads: int, n_kv_heads: int, dim: int, v_dim: int, rotary_dim: int, interleaved: bool,
-                   write_kv: bool) -> None:
+                   write_kv: bool, n_v_heads: Optional[int] = None, v_norm: bool = False,
+                   partial: Optional[torch.Tensor] = None, splits: int = 0, split_stride: int = 0, row_width: int = 0,
+                   tail_col: int = 0) -> None:
     """Rows [q heads | k heads at k_col | v heads at v_col]: q and k heads are (with `norm`) divided by their root mean
     square and multiplied by q_w / k_w [dim], then their first `rotary_dim` numbers are turned by the token's position;
-    q in place, k and v to the token's cache row (`write_kv`)."""
+    q in place, k and v to the token's cache row (`write_kv`).  `n_v_heads` (as many as k heads): value heads; v_col may
+    be k_col (values that are the keys' projections); `v_norm`: value heads are divided by their root mean square.  With
+    `partial` [splits, rows, row_width] floats the rows are their sums, and columns from `tail_col` on are stored too."""
+    n_v_heads = n_kv_heads if n_v_heads is None else n_v_heads
+    partial_splits = splits if partial is not None else 0
+    _need_cuda(partial)
     _need_cuda(proj, tok_seq, tok_pos, seq_slot, inv_freq, q_w, k_w, k_cache, v_cache, page_table)
     assert proj.stride(1) == 1 and (inv_freq is None or (inv_freq.dtype == torch.float32 and inv_freq.numel() >= rotary_dim // 2))
     w_dtype = F32
@@ -810,11 +823,14 @@ def qk_norm_rotate(proj, k_col: int, v_col: int, tok_seq, tok_pos, seq_slot, inv
     if write_kv:
         assert k_cache.dtype == proj.dtype == v_cache.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
         assert k_cache.shape[-1] == dim and v_cache.shape[-1] == v_dim
-        assert proj.shape[1] >= v_col + n_kv_heads * v_dim and v_col >= k_col + n_kv_heads * dim >= 0
+        assert k_cache.shape[-2] == n_kv_heads and v_cache.shape[-2] == n_v_heads
+        assert proj.shape[1] >= v_col + n_v_heads * v_dim and (v_col >= k_col + n_kv_heads * dim >= 0 or v_col == k_col)
     _call("core", "mdma_qk_norm_rotate", _ptr(proj), _i(dtype_code(proj.dtype)), _i(proj.stride(0)), _i(k_col), _i(v_col),
           _ptr(tok_seq), _ptr(tok_pos), _ptr(seq_slot), _ptr(inv_freq), _f(magnitude), _ptr(q_w), _ptr(k_w), _i(w_dtype),
           _i(int(norm)), _f(eps), _ptr(k_cache), _ptr(v_cache), _ptr(page_table), _i(max_pages), _i(page_size), _i(n_tokens),
-          _i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim), _i(rotary_dim), _i(int(interleaved)), _i(int(write_kv)), _stream())
+          _i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim), _i(rotary_dim), _i(int(interleaved)), _i(int(write_kv)),
+          _i(n_v_heads), _i(int(v_norm)), _ptr(partial), _i(partial_splits), ctypes.c_long(split_stride), _i(row_width),
+          _i(tail_col), _stream())
 
 
 def talking_attention_tiled_fits(n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
