@@ -29,7 +29,8 @@ LIBRARIES = {
     "core": (["elementwise.cu", "gemm_simt.cu", "attention_simple.cu", "sampling.cu", "sequence_mix.cu",
              "latent_attention.cu", "rglru.cu", "attention_distance.cu", "routed_ffn.cu", "attention_prepare.cu",
              "linear_attention.cu", "group_norm.cu", "rotary_latent.cu", "attention_talking.cu",
-             "delta_rule.cu", "delta_chunk.cu", "attention_mixed_weights.cu"], ["common.cuh", "delta_rule.cuh"], []),
+             "delta_rule.cu", "delta_chunk.cu", "attention_mixed_weights.cu", "attention_finish.cu", "matrix_memory.cu"],
+             ["common.cuh", "delta_rule.cuh", "float4.cuh"], []),
     "tensor": (["gemm_tcgen05.cu", "attention_mma.cu", "attention_tc.cu", "attention_talking_mma.cu",
                 "attention_mixed_weights_mma.cu"], ["common.cuh", "ptx.cuh", "attention_mma.cuh"], []),
     "noalloc": (["attention_noalloc.cu"], ["common.cuh", "ptx.cuh", "attention_mma.cuh", "attention_noalloc.h"], []),

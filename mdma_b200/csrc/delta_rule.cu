@@ -15,7 +15,8 @@
 // all rows of the step; every sum has one fixed order, so the result does not depend on how rows were cut into steps.
 // The 32-bit engine's walk, and short portions.
 //
-// gated_head_rmsnorm: out = o_h / sqrt(mean(o_h^2) + eps) [* w] * act(gate), per head, act = sigmoid or silu.
+// gated_head_rmsnorm: out = o_h / sqrt(mean(o_h^2) + eps) [* w] * act(gate) * scale, per head, act = sigmoid or silu; w is one
+// head's (all heads share it) or the whole row's.
 #include "delta_rule.cuh"
 
 namespace mdma {
@@ -356,7 +357,8 @@ static int tok_rows(int dim, int vdim) {
 template <typename TG, typename TO>
 __global__ void __launch_bounds__(256)
 gated_head_rmsnorm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int gate_stride, const void* __restrict__ w,
-                          int w_dtype, TO* __restrict__ out, int n_rows, int heads, int vdim, float eps, int gate_act) {
+                          int w_dtype, TO* __restrict__ out, int n_rows, int heads, int vdim, float eps, int gate_act, int w_heads,
+                          float scale) {
     chain_release();
     chain_wait();
     const int pair = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -365,10 +367,11 @@ gated_head_rmsnorm_kernel(const float* __restrict__ o, const TG* __restrict__ ga
     const float* row = o + (size_t)pair * vdim;
     float sq = 0.f;
     for (int d = lane; d < vdim; d += 32) sq = fmaf(row[d], row[d], sq);
-    const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)vdim + eps);
+    const float inv = scale / sqrtf(warp_sum(sq) / (float)vdim + eps);
+    const int w0 = w_heads ? h * vdim : 0;
     for (int d = lane; d < vdim; d += 32) {
         const float g = to_float(gate[(size_t)t * gate_stride + h * vdim + d]);
-        const float y = row[d] * inv * (w ? delta_weight(w, w_dtype, d) : 1.0f);
+        const float y = row[d] * inv * (w ? delta_weight(w, w_dtype, w0 + d) : 1.0f);
         out[(size_t)pair * vdim + d] = from_float<TO>(y * (gate_act ? delta_silu(g) : delta_sigmoid(g)));
     }
 }
@@ -418,13 +421,14 @@ int mdma_delta_scan(const float* q, const float* k, const float* v, const float*
 
 // `gate_act` 0: sigmoid, 1: silu; `w` (vdim numbers, shared by the heads) may be null
 int mdma_gated_head_rmsnorm(const float* o, const void* gate, int g_dtype, int gate_stride, const void* w, int w_dtype, void* out,
-                            int out_dtype, int n_rows, int heads, int vdim, float eps, int gate_act, cudaStream_t stream) {
+                            int out_dtype, int n_rows, int heads, int vdim, float eps, int gate_act, int w_heads, float scale,
+                            cudaStream_t stream) {
     MDMA_REQUIRE(n_rows >= 0 && heads > 0 && vdim > 0, "gated_head_rmsnorm: bad sizes");
     if (n_rows == 0) return 0;
     const unsigned blocks = (unsigned)(((long)n_rows * heads + 7) / 8);
     MDMA_DISPATCH_DTYPE(g_dtype, TG, MDMA_DISPATCH_DTYPE(out_dtype, TO,
         launch_chained(gated_head_rmsnorm_kernel<TG, TO>, dim3(blocks), dim3(256), 0, stream, o, (const TG*)gate, gate_stride, w,
-                       w_dtype, (TO*)out, n_rows, heads, vdim, eps, gate_act)));
+                       w_dtype, (TO*)out, n_rows, heads, vdim, eps, gate_act, w_heads, scale)));
     MDMA_LAUNCH_OK("gated_head_rmsnorm");
     return 0;
 }

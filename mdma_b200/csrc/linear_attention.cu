@@ -20,6 +20,7 @@
 //
 // gated_rmsnorm: out = o / sqrt(mean(o^2) + eps) * w * sigmoid(g) * scale over the heads side by side.
 #include "common.cuh"
+#include "float4.cuh"
 
 namespace mdma {
 
@@ -184,15 +185,6 @@ constexpr int kAPitch = kChunk + 4;
 enum LinPass : int { kLinWhole = 0, kLinLocal = 1, kLinFrom = 2 };
 constexpr int kLinSingleRows = 2;      // value of the launcher's `chunked` that asks for the single-row kernel
 
-__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ void st4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void fma4(float4& acc, float a, const float4& b) {
-    acc.x = fmaf(a, b.x, acc.x); acc.y = fmaf(a, b.y, acc.y); acc.z = fmaf(a, b.z, acc.z); acc.w = fmaf(a, b.w, acc.w);
-}
-__device__ __forceinline__ void scale4(float4& v, float a) { v.x *= a; v.y *= a; v.z *= a; v.w *= a; }
-__device__ __forceinline__ float dot4(const float4& a, const float4& b, float acc) {
-    return fmaf(a.w, b.w, fmaf(a.z, b.z, fmaf(a.y, b.y, fmaf(a.x, b.x, acc))));
-}
 __device__ __forceinline__ void copy16_async(void* dst_shared, const void* src_global) {
     const unsigned d = (unsigned)__cvta_generic_to_shared(dst_shared);
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" :: "r"(d), "l"(src_global) : "memory");

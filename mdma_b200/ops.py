@@ -976,17 +976,17 @@ def delta_chunks(proj, raw, conv_w, taps: int, a_log, dt_bias, conv_state, scrat
 
 
 def gated_head_rmsnorm(o: torch.Tensor, gate: torch.Tensor, w: Optional[torch.Tensor], out: torch.Tensor, n_rows: int,
-                       heads: int, vdim: int, eps: float, gate_act: str = "sigmoid") -> None:
-    """out = o_h / sqrt(mean(o_h^2) + eps) * w * act(gate) head by head; o float rows of heads * vdim, `w` [vdim] shared by
-    the heads (None: no weight), gate may be a view of wider rows; act "sigmoid" or "silu"."""
+                       heads: int, vdim: int, eps: float, gate_act: str = "sigmoid", scale: float = 1.0) -> None:
+    """out = o_h / sqrt(mean(o_h^2) + eps) * w * act(gate) * scale head by head; o float rows of heads * vdim, `w` [vdim]
+    shared by the heads or [heads * vdim] (None: no weight), gate may be a view of wider rows; act "sigmoid" or "silu"."""
     _need_cuda(o, gate, w, out)
     width = heads * vdim
     assert o.dtype == torch.float32 and o.is_contiguous() and out.is_contiguous() and o.shape[1] == out.shape[1] == width
-    assert gate.stride(1) == 1 and gate.shape[1] >= width and (w is None or (w.numel() == vdim and w.is_contiguous()))
+    assert gate.stride(1) == 1 and gate.shape[1] >= width and (w is None or (w.numel() in (vdim, width) and w.is_contiguous()))
     assert gate_act in ("sigmoid", "silu")
     _call("core", "mdma_gated_head_rmsnorm", _ptr(o), _ptr(gate), _i(dtype_code(gate.dtype)), _i(gate.stride(0)), _ptr(w),
           _i(dtype_code(w.dtype) if w is not None else F32), _ptr(out), _i(dtype_code(out.dtype)), _i(n_rows), _i(heads),
-          _i(vdim), _f(eps), _i(int(gate_act == "silu")), _stream())
+          _i(vdim), _f(eps), _i(int(gate_act == "silu")), _i(int(w is not None and w.numel() == width)), _f(scale), _stream())
 
 
 # ---- attention whose heads' weights are mixed after the softmax (csrc/attention_mixed_weights.cu) ------------------------
