@@ -7,8 +7,8 @@ head_dim]` for keys and one for values (of `v_dim` numbers a head where that
 differs from the keys'; none for a need with `values=False`: one vector per
 token that serves as both), a free list of pages and one page
 table `[slots, max_pages]`.  A sequence holds a slot, and in every group the
-pages that cover its length; groups with a window give pages back once every
-key in them has left the window (except those of the first `keep_first` tokens).  Slots and pages go back to the free lists
+pages that cover its length; groups with a window (or chunks) give pages back once
+no later token sees a key in them (those of the first `keep_first` tokens stay).  Slots and pages go back to the free lists
 when a sequence ends and are handed out again.  Next to the pages lies
 fixed-size per-sequence state `[slots, ...]` for sites that declare some; it
 is zeroed when a slot is taken.
@@ -37,6 +37,19 @@ class KVNeed:
     values: bool = True      # False: one vector per token only (a latent that serves as key and value)
     v_dim: int = 0           # size of a value head when it differs from the key's (0: the same)
     keep_first: int = 0      # with a window: the first tokens' keys stay visible to every later token
+    chunk: int = 0           # n: only keys of the query's own chunk of n positions are read (then no window)
+    n_v_heads: int = 0       # value heads where their number differs from the keys' (0: the same)
+
+    @property
+    def bounded(self) -> bool:
+        """Whether keys go out of sight of every later token."""
+        return self.window > 0 or self.chunk > 0
+
+    def first_key(self, pos: int) -> int:
+        """The earliest key a query at `pos` reads, apart from the kept first ones."""
+        if self.chunk:
+            return pos // self.chunk * self.chunk
+        return max(0, pos + 1 - self.window) if self.window else 0
 
 
 @dataclass(frozen=True)
@@ -69,7 +82,7 @@ class CacheGroup:
         self.seq_pages: dict[int, dict[int, int]] = {}      # slot -> {page index in sequence: page}
         self.dirty: set[int] = set()
         shape = (len(sites), n_pages, page_size, need.n_kv_heads, need.head_dim)
-        v_shape = shape[:-1] + (need.v_dim or need.head_dim,)
+        v_shape = shape[:3] + (need.n_v_heads or need.n_kv_heads, need.v_dim or need.head_dim)
         self.bytes = ((int(np.prod(shape)) + (int(np.prod(v_shape)) if need.values else 0))
                       * torch.empty((), dtype=dtype).element_size())
         # `alloc(shape, dtype)` hands out zeroed device memory, or None when only sizes are wanted
@@ -82,10 +95,8 @@ class CacheGroup:
         have = self.seq_pages.setdefault(slot, {})
         if new_len <= 0:
             return
-        first_needed = 0
-        if self.need.window:
-            # the earliest key any token of this step reads
-            first_needed = max(0, old_len + 1 - self.need.window) // self.page_size
+        # the earliest key any token of this step reads
+        first_needed = self.need.first_key(old_len) // self.page_size
         last = (new_len - 1) // self.page_size
         if last >= self.max_pages:
             raise CacheFull(f"a sequence of {new_len} tokens needs more than {self.max_pages} pages")
@@ -100,12 +111,12 @@ class CacheGroup:
             self.dirty.add(slot)
 
     def trim(self, slot: int, length: int) -> None:
-        """Give back pages whose keys have all left the window of every later token (the first tokens that the need
-        keeps stay)."""
-        if not self.need.window:
+        """Give back pages whose keys no later token sees: they have left the window or lie in an earlier chunk (the
+        first tokens that the need keeps stay)."""
+        if not self.need.bounded:
             return
         have = self.seq_pages.get(slot, {})
-        first_live = max(0, length + 1 - self.need.window) // self.page_size
+        first_live = self.need.first_key(length) // self.page_size
         for p in [p for p in have if self.kept_pages <= p < first_live]:
             self.pages.release(have.pop(p))
 
@@ -199,7 +210,7 @@ class SequenceCache:
                     return (f"sequence in slot {slot} would reach {old + n_new} tokens, "
                             f"beyond the context of {self.max_context}")
                 have = g.seq_pages.get(slot, {})
-                first = max(0, old + 1 - g.need.window) // self.page_size if g.need.window else 0
+                first = g.need.first_key(old) // self.page_size
                 if old > 0:                    # pages up to the one that holds position old - 1 are held
                     first = max(first, (old - 1) // self.page_size)
                 last = (old + n_new - 1) // self.page_size
@@ -240,8 +251,8 @@ class SequenceCache:
             raise ValueError("a cache with fixed-size per-sequence state cannot be rewound")
         for g in self.groups:
             have = g.seq_pages.get(slot, {})
-            if g.need.window:
-                first_needed = max(0, length + 1 - g.need.window) // self.page_size
+            if g.need.bounded:
+                first_needed = g.need.first_key(length) // self.page_size
                 last = (length - 1) // self.page_size if length else -1
                 if any(p not in have for p in range(first_needed, last + 1)):
                     raise ValueError("a windowed group has already released pages of the kept part")

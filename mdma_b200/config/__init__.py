@@ -49,11 +49,13 @@ from . import mogevik_arch  # noqa: E402,F401  registers the Mogevik architectur
 from . import tubusun_arch  # noqa: E402,F401  registers the Tubusun architecture
 from . import fizadra_arch  # noqa: E402,F401  registers the Fizadra architecture
 from . import degavik_arch  # noqa: E402,F401  registers the Degavik architecture
+from . import salipel_arch  # noqa: E402,F401  registers the Salipel architecture
 from .degavik import DegavikConfig  # noqa: E402
 from .fizadra import FizadraConfig  # noqa: E402
 from .gevonex import GevonexConfig  # noqa: E402
 from .mogevik import MogevikConfig  # noqa: E402
+from .salipel import SalipelConfig  # noqa: E402
 from .tubusun import TubusunConfig  # noqa: E402
 
-__all__ = ["Architecture", "ConfigError", "DegavikConfig", "FizadraConfig", "GevonexConfig", "LlamaConfig", "MogevikConfig", "RopeScaling", "RegistryError", "TubusunConfig",
+__all__ = ["Architecture", "ConfigError", "DegavikConfig", "FizadraConfig", "GevonexConfig", "LlamaConfig", "MogevikConfig", "RopeScaling", "RegistryError", "SalipelConfig", "TubusunConfig",
            "architecture_name", "load_config", "read_config_json"]

@@ -8,11 +8,11 @@
 //     largest c (1: its largest); only the `keep_groups` best groups stay eligible (the others count as
 //     minus infinity)
 //     the `top` eligible experts with the largest c are chosen (ties: the lower number)
-//     weight_j = s[chosen_j] / (sum of the chosen s + 1e-20), or s[chosen_j] itself (`renormalize` 0)
+//     weight_j = s[chosen_j] / (sum of the chosen s + 1e-20), or s[chosen_j] itself (`renormalize` 0), times a constant
 // and, if the layer has a shared expert with a gate, sg = sigmoid(g . h), one number per token.
 //
 // Experts: expert e maps h to D_e pair(G_e h, U_e h), pair(g, u) = SiLU(g) * u or another gated form of
-// `gated_pair`; the last `n_identity` routed
+// `gated_pair`, or without U (a null pointer) to D_e act(G_e h); the last `n_identity` routed
 // outputs have no matrices, their output is h itself.  The matrices of all experts are stacked:
 // G and U [experts * ff, width], D [experts * width, ff].
 //
@@ -66,7 +66,7 @@ template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(256)
 route_kernel(const TA* __restrict__ h, int h_stride, const TW* __restrict__ router, const TC* __restrict__ correction,
              const TW* __restrict__ shared_gate, int width, int n_routed, int top, int n_groups, int keep_groups,
-             int scoring, int group_top, int renormalize, int logit_bias,
+             int scoring, int group_top, int renormalize, int logit_bias, float weight_scale,
              int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ shared_scale) {
     chain_release();
     chain_wait();
@@ -142,7 +142,7 @@ route_kernel(const TA* __restrict__ h, int h_stride, const TW* __restrict__ rout
     }
     for (int k = 0; k < top; ++k) {
         chosen[(size_t)t * top + k] = pick[k];
-        weights[(size_t)t * top + k] = pick[k] < 0 ? 0.f : renormalize ? z[pick[k]] / (total + 1e-20f) : z[pick[k]];
+        weights[(size_t)t * top + k] = pick[k] < 0 ? 0.f : weight_scale * (renormalize ? z[pick[k]] / (total + 1e-20f) : z[pick[k]]);
     }
 }
 
@@ -165,6 +165,13 @@ expert_gate_up_kernel(const TA* __restrict__ h, int h_stride, const TW* __restri
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
     const bool vec = width % 8 == 0 && (((uintptr_t)G | (uintptr_t)U) & 15) == 0;
+    if (U == nullptr) {
+        for (int f = blockIdx.y * n_warps + warp; f < ff; f += gridDim.y * n_warps) {
+            const float z = warp_dot(hs, G + ((size_t)e * ff + f) * width, width, lane, vec);
+            if (lane == 0) act[(size_t)pair * ff + f] = from_float<TA>(gate_activation(z, pair_act));
+        }
+        return;
+    }
     for (int f = blockIdx.y * n_warps + warp; f < ff; f += gridDim.y * n_warps) {
         const TW* g = G + ((size_t)e * ff + f) * width;
         const TW* u = U + ((size_t)e * ff + f) * width;
@@ -317,7 +324,7 @@ expert_gate_up_sorted_kernel(const TA* __restrict__ h, int h_stride, const TW* _
             const bool ok = f0 + f < ff && k0 + k < width;
             const size_t at = ((size_t)e * ff + f0 + f) * width + k0 + k;
             gs[k][f] = ok ? to_float(G[at]) : 0.f;
-            us[k][f] = ok ? to_float(U[at]) : 0.f;
+            us[k][f] = ok && U != nullptr ? to_float(U[at]) : 0.f;
         }
         __syncthreads();
         float pg[2][4] = {}, pu[2][4] = {};
@@ -346,7 +353,7 @@ expert_gate_up_sorted_kernel(const TA* __restrict__ h, int h_stride, const TW* _
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int f = f0 + fx * 4 + j;
-            if (f < ff) act[(size_t)pr * ff + f] = from_float<TA>(gated_pair(ag[i][j], au[i][j], pair_act, act_limit, act_alpha));
+            if (f < ff) act[(size_t)pr * ff + f] = from_float<TA>(U == nullptr ? gate_activation(ag[i][j], pair_act) : gated_pair(ag[i][j], au[i][j], pair_act, act_limit, act_alpha));
         }
     }
 }
@@ -446,8 +453,8 @@ extern "C" {
 
 int mdma_route(const void* h, int h_dtype, int h_stride, const void* router, int w_dtype, const void* correction,
                int c_dtype, const void* shared_gate, int n_tokens, int width, int n_routed, int top, int n_groups,
-               int keep_groups, int scoring, int group_top, int renormalize, int logit_bias, int* chosen, float* weights,
-               float* shared_scale, cudaStream_t stream) {
+               int keep_groups, int scoring, int group_top, int renormalize, int logit_bias, float weight_scale, int* chosen,
+               float* weights, float* shared_scale, cudaStream_t stream) {
     MDMA_REQUIRE(!logit_bias || correction, "route: a bias on the logits needs its numbers");
     MDMA_REQUIRE(scoring >= 0 && scoring <= 1 && group_top >= 1 && group_top <= kMaxGroupTop,
                  "route: scoring %d, a group's score over its %d largest (at most %d)", scoring, group_top, kMaxGroupTop);
@@ -462,7 +469,7 @@ int mdma_route(const void* h, int h_dtype, int h_stride, const void* router, int
         MDMA_DISPATCH_DTYPE(c_dtype, TC,
             launch_chained(route_kernel<TA, TW, TC>, dim3(n_tokens), dim3(256), 0, stream, (const TA*)h, h_stride,
                            (const TW*)router, (const TC*)correction, (const TW*)shared_gate, width, n_routed, top,
-                           n_groups, keep_groups, scoring, group_top, renormalize, logit_bias, chosen, weights, shared_scale)));
+                           n_groups, keep_groups, scoring, group_top, renormalize, logit_bias, weight_scale, chosen, weights, shared_scale)));
     MDMA_LAUNCH_OK("route");
     return 0;
 }

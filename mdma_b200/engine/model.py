@@ -192,7 +192,8 @@ class DecoderModel:
                 if ctx.rt.gemm == "tensor":
                     from .. import ops_tensor
                     ops_tensor.flush_pending(x.device, ctx.rt.tc)
-                self.on_layer(n, x[:ctx.n_tokens])
+                rows = x[:ctx.n_tokens]
+                self.on_layer(n, rows if self.spec.stream_unit == 1.0 else rows * self.spec.stream_unit)
         if ctx.rt.gemm == "tensor":
             from .. import ops_tensor
             ops_tensor.flush_pending(x.device, ctx.rt.tc)

@@ -554,10 +554,11 @@ def attention_distance(q, k_cache, v_cache, ctx, page_table, max_pages: int, pag
 
 # ---- routed feed-forward (csrc/routed_ffn.cu) -----------------------------------------------------------------------
 def route(h, router, correction, shared_gate, n_tokens: int, top: int, n_groups: int, keep_groups: int, chosen, weights,
-          shared_scale, scoring: str = "softmax", group_top: int = 1, renormalize: bool = True, logit_bias=None) -> None:
+          shared_scale, scoring: str = "softmax", group_top: int = 1, renormalize: bool = True, logit_bias=None,
+          weight_scale: float = 1.0) -> None:
     """Per token: scores over the router's logits (`scoring`: "softmax" over all, or "sigmoid" of each), choice among the
     best groups (a group's score: the sum of its `group_top` largest), `top` experts and their weights (their scores,
-    divided by their sum if `renormalize`); with `shared_gate` [width] also sigmoid(shared_gate . h) into `shared_scale`.
+    divided by their sum if `renormalize`, times `weight_scale`); with `shared_gate` [width] also sigmoid(shared_gate . h) into `shared_scale`.
     `logit_bias` [n_routed] (in the place of `correction`) joins the logits themselves."""
     assert scoring in ("softmax", "sigmoid") and (correction is None or logit_bias is None)
     biased = logit_bias is not None
@@ -571,22 +572,22 @@ def route(h, router, correction, shared_gate, n_tokens: int, top: int, n_groups:
     _call("core", "mdma_route", _ptr(h), _i(dtype_code(h.dtype)), _i(h.stride(0)), _ptr(router), _i(dtype_code(router.dtype)),
           _ptr(correction), _i(dtype_code(correction.dtype) if correction is not None else F32), _ptr(shared_gate),
           _i(n_tokens), _i(width), _i(n_routed), _i(top), _i(n_groups), _i(keep_groups), _i(int(scoring == "sigmoid")),
-          _i(group_top), _i(int(renormalize)), _i(int(biased)), _ptr(chosen), _ptr(weights), _ptr(shared_scale), _stream())
+          _i(group_top), _i(int(renormalize)), _i(int(biased)), _f(weight_scale), _ptr(chosen), _ptr(weights), _ptr(shared_scale), _stream())
 
 
 def experts(h, gate_w, up_w, down_w, chosen, weights, n_tokens: int, n_experts: int, top: int, ff: int, act, x,
             sorted_scratch=None, pair_act: int = ACT_SILU, act_limit: float = 0.0, act_alpha: float = 1.0) -> None:
     """x += sum over each token's chosen experts of weight * expert(h) (identity experts: weight * h).  gate_w, up_w
-    [experts * ff, width], down_w [experts * width, ff]; act [tokens * top, ff] scratch in h's dtype.
+    (None: experts without a gate, act(gate_w h)) [experts * ff, width], down_w [experts * width, ff]; act [tokens * top, ff] scratch in h's dtype.
     `sorted_scratch` = (first [2 * (experts + 1)] ints, order, y): the expert-by-expert kernels (steps of many tokens); else token by token."""
     _need_cuda(h, gate_w, up_w, down_w, chosen, weights, act, x)
     width = h.shape[1]
     assert h.stride(1) == 1 and x.dtype == torch.float32 and x.is_contiguous() and x.shape[1] == width
     assert act.is_contiguous() and act.dtype == h.dtype and act.shape[1] == ff
     if n_experts:
-        assert gate_w.is_contiguous() and up_w.is_contiguous() and down_w.is_contiguous()
-        assert tuple(gate_w.shape) == (n_experts * ff, width) == tuple(up_w.shape) and tuple(down_w.shape) == (n_experts * width, ff)
-        assert gate_w.dtype == up_w.dtype == down_w.dtype
+        assert gate_w.is_contiguous() and down_w.is_contiguous() and gate_w.dtype == down_w.dtype
+        assert tuple(gate_w.shape) == (n_experts * ff, width) and tuple(down_w.shape) == (n_experts * width, ff)
+        assert up_w is None or (up_w.is_contiguous() and up_w.shape == gate_w.shape and up_w.dtype == gate_w.dtype)
     wd = dtype_code(gate_w.dtype) if n_experts else dtype_code(h.dtype)
     if sorted_scratch is None:
         _call("core", "mdma_experts_by_token", _ptr(h), _i(dtype_code(h.dtype)), _i(h.stride(0)), _ptr(gate_w), _ptr(up_w),
@@ -1004,3 +1005,82 @@ def mixed_weights_attention(q, k_cache, v_cache, mix, factor, softcap: float, ct
           _ptr(mix), _ptr(factor), _f(softcap), _ptr(ctx.tok_seq), _ptr(ctx.tok_pos), _ptr(ctx.seq_slot), _ptr(page_table),
           _i(max_pages), _i(page_size), _ptr(out), _i(ctx.n_tokens), _i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim),
           _i(window), _i(keep_first), _stream())
+
+
+# ---- what follows attention before its output product (csrc/attention_finish.cu) -----------------------------------------
+def attention_finish(out: torch.Tensor, n_tokens: int, n_heads: int, v_dim: int, rows: Optional[torch.Tensor] = None,
+                     partial: Optional[tuple] = None, sink_log2=None, gate=None, maps: int = 1, lam: float = 0.0,
+                     norm_scale: float = 1.0, eps: float = 0.0, out_scale: float = 1.0) -> None:
+    """out [tokens, heads * v_dim] from attention's rows [tokens, heads * maps * v_dim] or, with `partial` = (sums, maxima and
+    sums of weights, runs), from partial sums over runs of keys, merged in order (`sink_log2` joins the denominators once).
+    Two maps: a_1 - lam a_2, divided by its root mean square over the head, times norm_scale.  Then times sigmoid(gate)
+    (rows of heads * v_dim, may be a view of wider rows) and out_scale.  All in float."""
+    _need_cuda(out, rows, sink_log2, gate)
+    assert out.is_contiguous() and out.shape[1] == n_heads * v_dim and out.shape[0] >= n_tokens
+    assert gate is None or (gate.dtype == out.dtype and gate.stride(1) == 1 and gate.shape[1] >= n_heads * v_dim)
+    part_o = part_ml = None
+    splits = 0
+    if partial is not None:
+        part_o, part_ml, splits = partial
+        assert part_o.numel() >= n_tokens * n_heads * maps * splits * v_dim and part_ml.numel() >= n_tokens * n_heads * maps * splits * 2
+        assert part_o.dtype == part_ml.dtype == torch.float32
+    else:
+        assert rows.is_contiguous() and rows.shape[1] == n_heads * maps * v_dim and rows.shape[0] >= n_tokens
+    _call("core", "mdma_attention_finish", _ptr(rows), _i(dtype_code(rows.dtype) if rows is not None else F32), _ptr(part_o),
+          _ptr(part_ml), _i(splits), _ptr(sink_log2), _ptr(gate), _i(gate.stride(0) if gate is not None else 0), _ptr(out),
+          _i(dtype_code(out.dtype)), _i(n_tokens), _i(n_heads), _i(maps), _i(v_dim), _f(lam), _f(norm_scale), _f(eps),
+          _f(out_scale), _stream())
+
+
+# ---- a matrix memory with exponential gates (csrc/matrix_memory.cu) --------------------------------------------------------
+def matrix_memory_state_floats(heads: int, dim: int, vdim: int) -> int:
+    """Floats of a sequence's state: S, then n and m once per part of the columns (the layout of csrc/matrix_memory.cu; kept
+    here so that a memory plan needs no compiled library)."""
+    cols = min(vdim, 64)
+    while cols > 1 and dim * cols > 12288:
+        cols = (cols + 1) // 2
+    floats = heads * (dim * vdim + -(-vdim // cols) * (-(-(dim + 2) // 4) * 4))
+    return -(-floats // 4) * 4
+
+
+def matrix_memory(proj, cols, i_bias, f_bias, cap: float, q_scale: float, ctx, state, out, heads: int, dim: int, vdim: int,
+                  chunked: bool = False, run_rows: int = 0, max_runs: int = 1, scratch=None) -> None:
+    """The recurrence over each sequence's rows.  `proj`: float rows with q, k, v, the input gate's and the forget gate's
+    numbers at the columns `cols`; `state` rows of `matrix_memory_state_floats` floats are read and brought up to date; out
+    [T, heads * vdim] floats.  `chunked`: a chunk of rows at a time, with `run_rows` > 0 in runs of that many rows side by
+    side (`max_runs`: the most runs of a sequence, 256 at most; `scratch`: n_seqs * max_runs states).  Equal up to rounding."""
+    _need_cuda(proj, i_bias, f_bias, state, out, scratch)
+    q_col, k_col, v_col, i_col, f_col = cols
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and i_bias.numel() == f_bias.numel() == heads
+    assert proj.shape[1] >= max(q_col + heads * dim, k_col + heads * dim, v_col + heads * vdim, i_col + heads, f_col + heads)
+    assert out.dtype == torch.float32 and out.is_contiguous() and out.shape[1] == heads * vdim
+    assert run_rows == 0 or (chunked and scratch is not None and scratch.dtype == torch.float32 and scratch.is_contiguous())
+    sp, ss = _state(state)
+    assert state.shape[1] >= matrix_memory_state_floats(heads, dim, vdim)
+    _call("core", "mdma_matrix_memory", _ptr(proj), _i(proj.stride(0)), _i(q_col), _i(k_col), _i(v_col), _i(i_col), _i(f_col),
+          _ptr(i_bias), _ptr(f_bias), _i(_same_dtype(i_bias, f_bias)), _f(cap), _f(q_scale), _ptr(ctx.seq_start), _ptr(ctx.seq_slot),
+          sp, ss, _ptr(out), _i(ctx.n_seqs), _i(heads), _i(dim), _i(vdim), _i(int(chunked)), _i(run_rows), _i(max_runs),
+          _ptr(scratch), ctypes.c_long(scratch.numel() if scratch is not None else 0), _stream(), launches=2 if run_rows > 0 else 1)
+
+
+def matrix_memory_token_fits(dim: int, vdim: int) -> bool:
+    lib = _build._loaded.get("core") or _build.load("core")
+    return bool(lib.mdma_matrix_memory_token_fits(_i(dim), _i(vdim)))
+
+
+def matrix_memory_token(proj, cols, g_col: int, i_bias, f_bias, cap: float, q_scale: float, norm_w, ctx, state, out, heads: int,
+                        dim: int, vdim: int, eps: float, out_scale: float = 1.0, partial=None, splits: int = 0,
+                        split_stride: int = 0) -> None:
+    """Single tokens of the serving engine, from the projection rows (or with `partial` the sums of a K-split product's
+    partial rows) to the normed, gated heads times `out_scale` in `out` (bfloat16); state brought up to date."""
+    _need_cuda(proj, i_bias, f_bias, norm_w, state, out, partial)
+    q_col, k_col, v_col, i_col, f_col = cols
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and i_bias.numel() == f_bias.numel() == heads and ctx.max_new == 1
+    assert out.dtype == torch.bfloat16 and out.is_contiguous() and out.shape[1] == heads * vdim
+    assert norm_w.numel() == heads * vdim and norm_w.is_contiguous()
+    sp, ss = _state(state)
+    assert state.shape[1] >= matrix_memory_state_floats(heads, dim, vdim)
+    _call("core", "mdma_matrix_memory_token", _ptr(proj), _i(proj.stride(0)), _ptr(partial), _i(splits if partial is not None else 0),
+          ctypes.c_long(split_stride), _i(proj.shape[1]), _i(q_col), _i(k_col), _i(v_col), _i(g_col), _i(i_col), _i(f_col),
+          _ptr(i_bias), _ptr(f_bias), _i(_same_dtype(i_bias, f_bias)), _f(cap), _f(q_scale), _ptr(norm_w), _i(dtype_code(norm_w.dtype)),
+          _ptr(ctx.seq_slot), sp, ss, _ptr(out), _i(ctx.n_seqs), _i(heads), _i(dim), _i(vdim), _f(eps), _f(out_scale), _stream())

@@ -215,13 +215,16 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int = ops.GE
 
 def gemm_runs(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, first: list, n_features: int,
               mode: int = ops.GEMM_STORE, w2: Optional[torch.Tensor] = None, st: Optional[TensorState] = None,
-              act: int = ops.ACT_SILU, act_limit: float = 0.0, act_alpha: float = 1.0) -> None:
+              act: int = ops.ACT_SILU, act_limit: float = 0.0, act_alpha: float = 1.0, store_act: bool = False) -> None:
     """Run r = 0.. of rows: out[first[r]:first[r+1]] = a[first[r]:first[r+1]] @ w[r * n_features:(r+1) * n_features].T
-    (gated mode: act(gate) * up with w2 stacked likewise).  `first`: a host list of len(runs) + 1 row numbers.  One
+    (gated mode: act(gate) * up with w2 stacked likewise; `store_act`: act of a stored product).  `first`: a host list of len(runs) + 1 row numbers.  One
     call for all runs: the loop over the products is in the library."""
     _need_cuda(a, w, out, w2)
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("the tensor-core product takes bfloat16 operands")
+    if store_act:
+        assert mode == ops.GEMM_STORE
+        act = act | 0x100
     n_runs = len(first) - 1
     K = w.shape[1]
     assert a.dim() == 2 and a.stride(1) == 1 and out.stride(1) == 1 and w.is_contiguous() and a.shape[1] == K
@@ -517,3 +520,63 @@ def mixed_weights_attention(ctx, q: torch.Tensor, view, mix: torch.Tensor, facto
           _f(softcap), _ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(ctx.seq_slot), _ptr(view.page_table), _i(view.max_pages),
           _i(view.page_size), _ptr(out), _ptr(scratch), _i(slab), _i(ctx.n_tokens), _i(ctx.n_seqs), _i(ctx.max_new), _i(n_heads),
           _i(n_kv_heads), _i(dim), _i(v_dim), _i(window), _i(keep_first), _stream(), launches=2 * -(-ctx.n_tokens // slab))
+
+
+# ---- attention with further options: kept tokens, chunks, a soft cap, maps (the EXT forms) ----------------------------------
+def attention_general_supported(n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
+    return attention_supported(n_heads, n_kv_heads, dim) and attention_supported(n_heads, n_kv_heads, v_dim)
+
+
+def attention_general(ctx, q: torch.Tensor, view, n_heads: int, n_kv_heads: int, dim: int, v_dim: int, scale: float,
+                      out: Optional[torch.Tensor] = None, out_f32: Optional[torch.Tensor] = None, maps: int = 1, window: int = 0,
+                      keep_first: int = 0, chunk: int = 0, softcap: float = 0.0, sink_log2: Optional[torch.Tensor] = None,
+                      slope_log2: Optional[torch.Tensor] = None, splits: Optional[int] = None, impl: Optional[str] = None,
+                      st: Optional[TensorState] = None):
+    """`attention` with value heads of `v_dim` numbers and: `keep_first`, with a window the first tokens stay visible;
+    `chunk`, a query sees the keys of its own chunk of positions only; `softcap` c, c tanh(. / c) on the scores before the
+    penalty; `maps` m, query heads [head][map], key heads [kv head][map], one value head per kv head.  Returns None when the
+    finished rows [tokens][head][map] are in `out` (bfloat16) or `out_f32`, else (sums, maxima and sums of weights, runs) in
+    the state's scratch, for `ops.attention_finish` (which then takes the sink too)."""
+    _need_cuda(q, view.k, view.v, out, out_f32, view.page_table, sink_log2, slope_log2)
+    if q.dtype != torch.bfloat16 or view.k.dtype != torch.bfloat16:
+        raise KernelError("the tensor-core attention takes bfloat16")
+    assert (out is None) != (out_f32 is None)
+    rows = out if out is not None else out_f32
+    assert rows.dtype == (torch.bfloat16 if out is not None else torch.float32) and rows.is_contiguous()
+    assert rows.shape[1] == n_heads * maps * v_dim and rows.shape[0] >= ctx.n_tokens
+    assert q.stride(1) == 1 and view.k.is_contiguous() and view.v.is_contiguous()
+    assert view.k.shape[-2:] == (n_kv_heads * maps, dim) and view.v.shape[-2:] == (n_kv_heads, v_dim)
+    for t in (sink_log2, slope_log2):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n_heads)
+    st = st or _device_state(q.device)
+    flush_pending(q.device, st)
+    group = n_heads // n_kv_heads
+    if impl is None:
+        impl = "tc" if ctx.max_new * group > 64 and splits is None and attention_tc_supported(n_heads, n_kv_heads, dim, view.page_size) else "mma"
+    common = (_i(ctx.n_tokens), _i(ctx.n_seqs), _i(ctx.max_new), _i(n_heads), _i(n_kv_heads), _i(dim), _i(v_dim), _i(maps),
+              _i(window), _i(keep_first), _i(chunk), _f(softcap), _f(scale))
+    meta = (_ptr(ctx.seq_start), _ptr(ctx.seq_pos0), _ptr(ctx.seq_slot), _ptr(view.page_table), _i(view.max_pages), _i(view.page_size),
+            _ptr(out), _ptr(out_f32))
+    if impl == "tc":
+        _call("tensor", "mdma_attention_tc_general", _ptr(q), _i(q.stride(0)), _i(q.shape[0]), _ptr(view.k), _ptr(view.v),
+              _i(view.k.shape[0]), *meta, *common, _ptr(st.status), _ptr(sink_log2), _ptr(slope_log2), _stream())
+        return None
+    if splits is None:
+        # keys a row can see at most: the choice follows the capacity and the rounded context, as `attention_splits` does
+        seen = -(-ctx.max_len // 1024) * 1024
+        if chunk:
+            seen = min(seen, chunk)
+        elif window:
+            seen = min(seen, window + keep_first)
+        splits = attention_splits(ctx.n_seqs, ctx.max_new, ctx.max_len, n_heads * maps, n_kv_heads * maps, st.sms,
+                                  getattr(ctx, "most_seqs", None))
+        splits = max(1, min(splits, -(-seen // 64)))
+    need = ctx.n_tokens * n_heads * maps * splits * (v_dim + 2) if splits > 1 else 0
+    st.need(need, "attention over split keys")
+    _call("tensor", "mdma_attention_mma_general", _ptr(q), _i(q.stride(0)), _ptr(view.k), _ptr(view.v), _i(view.k.shape[0]), *meta,
+          *common, _i(splits), _ptr(st.scratch), ctypes.c_long(st.scratch.numel()), _ptr(st.status), _ptr(sink_log2), _ptr(slope_log2),
+          _stream())
+    if splits == 1:
+        return None
+    sums = ctx.n_tokens * n_heads * maps * splits * v_dim
+    return st.scratch[:sums], st.scratch[sums:need], splits

@@ -1,6 +1,6 @@
 """Parts a layer is put together from; importing this package registers them."""
-from . import (attention, block, delta_rule, distance_attention, embedding, gating, latent_attention, linear_attention, mlp, norm, recurrent,  # noqa: F401
-               rotary, routed_mlp, talking_attention)
+from . import (attention, block, delta_rule, distance_attention, embedding, gating, general_attention, latent_attention,  # noqa: F401
+               linear_attention, matrix_memory, mlp, norm, recurrent, rotary, routed_mlp, talking_attention)
 from .base import Part, Runtime
 from .linear import Linear
 

@@ -146,6 +146,8 @@ class ParallelBlock:
     """One norm, two readers:  h = norm(x);  x += mixer(h) + feed_forward(h)  (the feed-forward may be absent).
     Both sublayers add into the float residual stream, the mixer first."""
 
+    handles_pending = True      # completes x itself where a product left partial sums
+
     def __init__(self, spec: LayerSpec):
         self.spec = spec
         self.mixer_norm = NORMS.get(spec.mixer_norm.kind)(spec.mixer_norm)
@@ -162,6 +164,7 @@ class ParallelBlock:
 
     def forward(self, ctx, x, view, owns_cache=True):
         h = ctx.buf("normed", x.shape[1])
+        PreNormBlock._settle(ctx, x, self.mixer_norm)
         self.mixer_norm.forward(ctx, x, h)
         self.mixer.forward(ctx, h, x, view, owns_cache)
         if self.ffn is not None:

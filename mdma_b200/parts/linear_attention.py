@@ -192,8 +192,13 @@ class SideBySide(Part):
         return [m for m, _, _ in self.members]
 
     def attention_shapes(self):
-        return [(m.n_heads, m.n_kv_heads, m.head_dim) for m, _, _ in self.members
-                if all(hasattr(m, a) for a in ("n_heads", "n_kv_heads", "head_dim"))]
+        shapes = []
+        for m, _, _ in self.members:
+            if hasattr(m, "attention_shapes"):
+                shapes.extend(m.attention_shapes())
+            elif all(hasattr(m, a) for a in ("n_heads", "n_kv_heads", "head_dim")):
+                shapes.append((m.n_heads, m.n_kv_heads, m.head_dim))
+        return shapes
 
     def workspace(self):
         return {"side_scratch": (self.hidden, "f32")} if any(not folded for _, _, folded in self.members) else {}

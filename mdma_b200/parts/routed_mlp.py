@@ -6,9 +6,10 @@ The routed outputs form `groups` equal groups of neighbours; a group's score is 
 largest c (1, the default: its largest), and only
 members of the `keep_groups` best groups can be chosen (the others count as minus infinity).  The
 `top` eligible outputs with the largest c are chosen; their weights are their s divided by the sum of
-the chosen s (+ 1e-20), or with `renormalize` off their s as they are.  The first `experts` routed outputs are experts,
+the chosen s (+ 1e-20), or with `renormalize` off their s as they are, times `weight_scale` (1).  The first `experts` routed outputs are experts,
 D_e (silu(G_e h) * (U_e h)), or with `activation` "swish_limit" D_e (g sigmoid(act_alpha g) (u + 1)) where
-g = min(G_e h, act_limit) and u = U_e h kept within +-act_limit;
+g = min(G_e h, act_limit) and u = U_e h kept within +-act_limit; with `gated` off they have no gate, D_e act(U_e h),
+`activation` also "relu_squared", and no tensor `gate`;
 the last `identity` ones have no matrices and return h itself.  The result is the weighted sum.  A
 shared expert of the same form (`shared_ff` > 0) runs for every token and is added, multiplied by
 sigmoid(g . h), one number per token (`shared_gate`).
@@ -60,11 +61,15 @@ class RoutedMLP(Part):
         self.group_top = int(p.get("group_top", 1) or 1)
         self.renormalize = bool(p.get("renormalize", True))
         self.activation = str(p.get("activation", "silu"))
+        self.gated, self.weight_scale = bool(p.get("gated", True)), float(p.get("weight_scale", 1.0))
         self.act_limit, self.act_alpha = float(p.get("act_limit", 0.0) or 0.0), float(p.get("act_alpha", 1.0))
         if self.scoring not in ("softmax", "sigmoid") or not 1 <= self.group_top <= 8:
             raise ValueError(f"router scoring {self.scoring!r} with groups scored by their {self.group_top} largest is not implemented")
-        if self.activation not in ("silu", "gelu_tanh", "gelu", "swish_limit"):
+        if self.activation not in (("silu", "gelu_tanh", "gelu", "swish_limit") if self.gated else ("silu", "gelu_tanh", "gelu", "relu_squared")):
             raise ValueError(f"expert activation {self.activation!r} is not implemented")
+        if not self.gated and self.shared_ff:
+            raise ValueError("a shared expert goes with gated experts")
+        self.parts = ("gate", "up", "down") if self.gated else ("up", "down")
         self.pair_act = ops.ACTIVATIONS[self.activation]
         self.n_routed = self.n_experts + self.n_identity
         if not 0 < self.top <= min(self.n_routed, self.MAX_TOP) or self.n_routed > self.MAX_ROUTED:
@@ -77,7 +82,8 @@ class RoutedMLP(Part):
         W, F = self.hidden, self.ff
         specs = {}
         for e in range(self.n_experts):
-            specs[f"e{e}.gate"] = TensorSpec((F, W))
+            if self.gated:
+                specs[f"e{e}.gate"] = TensorSpec((F, W))
             specs[f"e{e}.up"] = TensorSpec((F, W))
             specs[f"e{e}.down"] = TensorSpec((W, F))
         specs["router"] = TensorSpec((self.n_routed, W))
@@ -96,7 +102,7 @@ class RoutedMLP(Part):
     def fused_tensors(self):
         if not self.n_experts:
             return {}
-        return {f"experts.{part}": tuple(f"e{e}.{part}" for e in range(self.n_experts)) for part in ("gate", "up", "down")}
+        return {f"experts.{part}": tuple(f"e{e}.{part}" for e in range(self.n_experts)) for part in self.parts}
 
     def device_tensors(self):
         return {"first": ((2 * (self.n_experts + 1),), torch.int32)}          # the experts' starts in the sorted list, and counters
@@ -121,12 +127,14 @@ class RoutedMLP(Part):
         self.w_gate = self.w_up = self.w_down = None
         if self.n_experts:
             stacked = {}
-            for part in ("gate", "up", "down"):
+            for part in self.parts:
                 t = tensors.get(f"experts.{part}")
                 if t is None:
                     t = torch.cat([tensors[f"e{e}.{part}"] for e in range(self.n_experts)], dim=0).contiguous()
                 stacked[part] = t
-            self.w_gate, self.w_up, self.w_down = stacked["gate"], stacked["up"], stacked["down"]
+            # the first product's matrices, the second factor's (None without a gate), the last product's
+            self.w_gate, self.w_up = (stacked["gate"], stacked["up"]) if self.gated else (stacked["up"], None)
+            self.w_down = stacked["down"]
         self.router = tensors["router"]
         self.correction_values, self.bias_values = tensors.get("correction"), tensors.get("router.b")
         self.shared_up = self.shared_down = self.sg = None
@@ -164,7 +172,8 @@ class RoutedMLP(Part):
         act = ctx.buf(names[3], self.top * self.ff)
         scale = ctx.buf(names[6], 1, torch.float32)
         ops.route(h, self.router, self.correction_values, self.sg, n, self.top, self.groups, self.keep_groups, chosen,
-                  weight, scale if self.sg is not None else None, self.scoring, self.group_top, self.renormalize, self.bias_values)
+                  weight, scale if self.sg is not None else None, self.scoring, self.group_top, self.renormalize, self.bias_values,
+                  self.weight_scale)
         if (self.by_products and n >= self.PRODUCTS_FROM and not getattr(ctx, "decode_only", False)
                 and not torch.cuda.is_current_stream_capturing()):
             self._experts_by_products(ctx, h, x, chosen, weight, act, names)
@@ -191,8 +200,11 @@ class RoutedMLP(Part):
         ops.experts_gather(h, chosen, n, self.n_experts, self.top, self.first, order, where, rows)
         first = self.first[:self.n_experts + 1].tolist()     # how many rows each expert got: read on the host
         from .. import ops_tensor
-        ops_tensor.gemm_runs(rows, self.w_gate, act, first, self.ff, ops.GEMM_SWIGLU, self.w_up, st=self.rt.tc,
-                             act=self.pair_act, act_limit=self.act_limit, act_alpha=self.act_alpha)
+        if self.gated:
+            ops_tensor.gemm_runs(rows, self.w_gate, act, first, self.ff, ops.GEMM_SWIGLU, self.w_up, st=self.rt.tc,
+                                 act=self.pair_act, act_limit=self.act_limit, act_alpha=self.act_alpha)
+        else:
+            ops_tensor.gemm_runs(rows, self.w_gate, act, first, self.ff, ops.GEMM_STORE, st=self.rt.tc, act=self.pair_act, store_act=True)
         ops_tensor.gemm_runs(act, self.w_down, y, first, self.hidden, ops.GEMM_STORE, st=self.rt.tc)
         ops.experts_combine(y, h, chosen, weight, where, n, self.n_experts, self.top, x)
 

@@ -79,3 +79,6 @@ class ModelSpec:
     lm_head: PartSpec
     stop_token_ids: tuple = ()
     junctions: list[PartSpec] = field(default_factory=list)
+    # the residual stream is kept in units of this number (an architecture that multiplies every sublayer's result by a
+    # constant keeps the stream divided by it)
+    stream_unit: float = 1.0
