@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl reference]
     python bench.py --shape llama-2-7b | llama-3.2-1b [--batch B] [--prompt-len P] [--prefill-tokens T]
-    python bench.py --compare gevonex|mogevik|tubusun|fizadra|degavik [--compare-widths 1024,2048,4096] [--compare-layers 4]
+    python bench.py --compare gevonex|mogevik|tubusun|fizadra|degavik|salipel [--compare-widths 1024,2048,4096] [--compare-layers 4]
 
 Prints ONE JSON line.  The default run has the layer sizes of the
 Llama-3.1-8B shape with random bfloat16 weights, a batch of 8 sequences
@@ -247,6 +247,26 @@ def degavik_config(width: int, layers: int, vocab: int) -> dict:
             "layers": [{"type": kinds[i % 4], "mixer": mixers[kinds[i % 4]], "mlp": moe if i % 2 else dense} for i in range(layers)]}
 
 
+def salipel_config(width: int, layers: int, vocab: int) -> dict:
+    """A Salipel of `layers` layers (chunked attention, differential attention, the pair, differential attention, ...) whose
+    sizes follow the width: query heads of 128 in groups of four over chunks of 1,024; heads of two maps of 64 over values of
+    128 with a soft cap; a window of 1,024 that keeps four tokens beside memory heads of 128 x 128; in turns sixteen
+    experts of 3/4 width, four per token, and a dense gated feed-forward of 8/3 width."""
+    heads = max(1, width // 128)
+    sizes = {"heads": heads, "kv_heads": max(1, heads // 4)}
+    mixers = {"attention": {**sizes, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024}},
+              "attention_2": {**sizes, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.5, "softcap": 50.0,
+                              "rot": {"dims": 64, "base": 10000.0}},
+              "parallel": {"left": {**sizes, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024, "keep_first": 4},
+                                    "rot": {"dims": 64, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+                           "right": {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 15.0}, "left_scale": 0.8, "right_scale": 0.6}}
+    kinds = ["attention", "attention_2", "parallel", "attention_2"]
+    moe = {"kind": "moe", "expert": {"ff": 3 * width // 4}, "router": {"experts": 16, "top": 4, "scale": 1.0}}
+    dense = {"kind": "dense", "ff": (8 * width // 3 + 255) // 256 * 256}
+    return {"architecture": "Salipel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+            "layers": [{"type": kinds[i % 4], "mixer": mixers[kinds[i % 4]], "mlp": dense if i % 2 else moe} for i in range(layers)]}
+
+
 def expert_share(cfg: dict, name: str, draws: int) -> float:
     """The share of an expert's matrix that a step of `draws` tokens reads (decode: distinct experts among the
     draws, chosen evenly) or, with draws = 0, the share of tokens that use it (prefill)."""
@@ -293,7 +313,7 @@ def compare(args) -> int:
                 n = 1
                 for d in ts.shape:
                     n *= d
-                routed = cfg.get("architecture") in ("Degavik", "Mogevik", "Tubusun")
+                routed = cfg.get("architecture") in ("Degavik", "Mogevik", "Salipel", "Tubusun")
                 matrix_bytes += 2 * n * (expert_share(cfg, name, batch) if routed else 1.0)
                 prefill_elements += n * (expert_share(cfg, name, 0) if routed else 1.0)
         # what a decode step moves besides the matrices: every live sequence's fixed-size state is read and written,
@@ -352,19 +372,21 @@ def compare(args) -> int:
     rows = []
     for width in [int(w) for w in args.compare_widths.split(",")]:
         row = {"width": width, "layers": args.compare_layers, "vocab": vocab, "batch": args.batch}
+        if args.compare == "salipel":
+            row["salipel"] = measure(salipel_config(width, args.compare_layers, vocab), args.batch)
         if args.compare == "degavik":
             row["degavik"] = measure(degavik_config(width, args.compare_layers, vocab), args.batch)
         if args.compare in ("fizadra", "degavik"):
             row["fizadra"] = measure(fizadra_config(width, args.compare_layers, vocab), args.batch)
-        if args.compare in ("tubusun", "degavik"):
+        if args.compare in ("tubusun", "degavik", "salipel"):
             row["tubusun"] = measure(tubusun_config(width, args.compare_layers, vocab), args.batch)
         if args.compare in ("mogevik", "tubusun"):
             row["mogevik"] = measure(mogevik_config(width, args.compare_layers, vocab), args.batch)
-        if args.compare not in ("tubusun", "degavik"):
+        if args.compare not in ("tubusun", "degavik", "salipel"):
             row["gevonex"] = measure(gevonex_config(width, args.compare_layers, vocab), args.batch)
         row["llama"] = measure(llama_like(width, args.compare_layers, vocab), args.batch)
         rows.append(row)
-    beside = {"degavik": "degavik beside tubusun, fizadra and llama", "fizadra": "fizadra beside gevonex and llama", "tubusun": "tubusun beside mogevik and llama", "mogevik": "mogevik beside gevonex and llama",
+    beside = {"salipel": "salipel beside tubusun and llama", "degavik": "degavik beside tubusun, fizadra and llama", "fizadra": "fizadra beside gevonex and llama", "tubusun": "tubusun beside mogevik and llama", "mogevik": "mogevik beside gevonex and llama",
               "gevonex": "gevonex beside llama"}[args.compare]
     print(json.dumps({"compare": beside + " at equal width, depth and vocabulary", "dtype": args.dtype,
                       "prefill_tokens": T, "decode_after_prompts_of": prompt, "peaks": peak_src,
@@ -393,7 +415,7 @@ def main() -> int:
     ap.add_argument("--prefill-only", action="store_true", help="run only the 2,048-token prefill (profiling runs)")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
                     help="float32: the true 32-bit engine (CUDA-core kernels), for the record; the headline is bfloat16")
-    ap.add_argument("--compare", default=None, choices=["gevonex", "mogevik", "tubusun", "fizadra", "degavik"],
+    ap.add_argument("--compare", default=None, choices=["gevonex", "mogevik", "tubusun", "fizadra", "degavik", "salipel"],
                     help="another program: the named architecture beside a Llama of equal size (see the header)")
     ap.add_argument("--compare-widths", default="1024,2048,4096")
     ap.add_argument("--compare-layers", type=int, default=4)

@@ -10,7 +10,7 @@
 
 namespace mdma {
 
-constexpr int kFinWarps = 8, kFinMaxDim = 256, kFinPerLane = kFinMaxDim / 32;
+constexpr int kFinWarps = 8, kFinMaxDim = 256;
 
 struct FinishParams {
     const void* rows;                  // finished rows (splits 0)
@@ -22,7 +22,25 @@ struct FinishParams {
     float out_scale;
 };
 
-template <typename TI, typename TO>
+// four neighbouring numbers (the address is aligned to them)
+__device__ __forceinline__ void fin_load4(const float* p, float* v) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void fin_load4(const __nv_bfloat16* p, float* v) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.y));
+    v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+}
+__device__ __forceinline__ void fin_store4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void fin_store4(__nv_bfloat16* p, const float* v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
+// VEC: heads of a multiple of four numbers, every row aligned to four; a lane owns the quads 4 lane + 128 i, else the
+// numbers lane + 32 i.  NQ: quads a lane owns at most (1: heads up to 128).
+template <typename TI, typename TO, bool VEC, int NQ>
 __global__ void __launch_bounds__(kFinWarps * 32)
 attention_finish_kernel(const FinishParams p, const TO* __restrict__ gate, TO* __restrict__ out) {
     chain_release();
@@ -30,30 +48,40 @@ attention_finish_kernel(const FinishParams p, const TO* __restrict__ gate, TO* _
     const int unit = blockIdx.x * kFinWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (unit >= p.n_tokens * p.n_heads) return;
     const int t = unit / p.n_heads, h = unit % p.n_heads;
-    // a lane's numbers: quads 4 lane + 128 i where rows allow it, else lane + 32 i
-    const bool quads = p.v_dim % 4 == 0;
-    auto at = [&](int i) { return quads ? (i >> 2) * 128 + lane * 4 + (i & 3) : lane + 32 * i; };
-    float o[kFinPerLane];
+    // f(number of the head, four of the lane's values at that place and how many of them are there)
+    auto quads = [&](auto&& f) {
 #pragma unroll
-    for (int i = 0; i < kFinPerLane; ++i) o[i] = 0.f;
+        for (int c = 0; c < NQ; ++c) {
+            if (VEC) {
+                const int d = c * 128 + lane * 4;
+                if (d < p.v_dim) f(d, 4 * c, 4);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int d = lane + 32 * (4 * c + i);
+                    if (d < p.v_dim) f(d, 4 * c + i, 1);
+                }
+            }
+        }
+    };
+    auto load = [](auto* src, float* v) {
+        if constexpr (VEC) fin_load4(src, v);
+        else v[0] = to_float(*src);
+    };
+    float o[4 * NQ];
+#pragma unroll
+    for (int i = 0; i < 4 * NQ; ++i) o[i] = 0.f;
     for (int j = 0; j < p.maps; ++j) {
         const size_t row = (size_t)unit * p.maps + j;
         const float f = j == 0 ? 1.0f : -p.lambda;
         if (p.splits == 0) {
             const TI* src = reinterpret_cast<const TI*>(p.rows) + row * p.v_dim;
-            if (quads && sizeof(TI) == 4) {
+            quads([&](int d, int i, int n) {
+                float v[4];
+                load(src + d, v);
 #pragma unroll
-                for (int c = 0; c < kFinPerLane / 4; ++c)
-                    if (at(4 * c) < p.v_dim) {
-                        const float4 v = *reinterpret_cast<const float4*>(src + at(4 * c));
-                        o[4 * c] = fmaf(f, v.x, o[4 * c]); o[4 * c + 1] = fmaf(f, v.y, o[4 * c + 1]);
-                        o[4 * c + 2] = fmaf(f, v.z, o[4 * c + 2]); o[4 * c + 3] = fmaf(f, v.w, o[4 * c + 3]);
-                    }
-            } else {
-#pragma unroll
-                for (int i = 0; i < kFinPerLane; ++i)
-                    if (at(i) < p.v_dim) o[i] = fmaf(f, to_float(src[at(i)]), o[i]);
-            }
+                for (int e = 0; e < (VEC ? 4 : 1); ++e) o[i + e] = fmaf(f, v[e], o[i + e]);
+            });
             continue;
         }
         const float* ml = p.part_ml + row * p.splits * 2;
@@ -61,36 +89,45 @@ attention_finish_kernel(const FinishParams p, const TO* __restrict__ gate, TO* _
         for (int s = 0; s < p.splits; ++s) m = fmaxf(m, ml[2 * s]);
         for (int s = 0; s < p.splits; ++s) if (ml[2 * s] != -INFINITY) l += exp2f(ml[2 * s] - m) * ml[2 * s + 1];
         if (p.sink_log2) l += exp2f(p.sink_log2[h] - m);
-        float a[kFinPerLane];
+        const float share = f / l;
+        float a[4 * NQ];
 #pragma unroll
-        for (int i = 0; i < kFinPerLane; ++i) a[i] = 0.f;
+        for (int i = 0; i < 4 * NQ; ++i) a[i] = 0.f;
         for (int s = 0; s < p.splits; ++s) {
             if (ml[2 * s] == -INFINITY) continue;                       // a run without a visible key
             const float w = exp2f(ml[2 * s] - m);
             const float* src = p.part_o + (row * p.splits + s) * p.v_dim;
+            quads([&](int d, int i, int n) {
+                float v[4];
+                load(src + d, v);
 #pragma unroll
-            for (int i = 0; i < kFinPerLane; ++i)
-                if (at(i) < p.v_dim) a[i] = fmaf(w, src[at(i)], a[i]);
+                for (int e = 0; e < (VEC ? 4 : 1); ++e) a[i + e] = fmaf(w, v[e], a[i + e]);
+            });
         }
 #pragma unroll
-        for (int i = 0; i < kFinPerLane; ++i) o[i] = fmaf(f, a[i] / l, o[i]);
+        for (int i = 0; i < 4 * NQ; ++i) o[i] = fmaf(share, a[i], o[i]);
     }
     float scale = p.out_scale;
     if (p.maps > 1) {
         float sq = 0.f;
 #pragma unroll
-        for (int i = 0; i < kFinPerLane; ++i) sq = fmaf(o[i], o[i], sq);
+        for (int i = 0; i < 4 * NQ; ++i) sq = fmaf(o[i], o[i], sq);
         scale *= p.norm_scale / sqrtf(warp_sum(sq) / (float)p.v_dim + p.eps);
     }
     TO* dst = out + (size_t)unit * p.v_dim;
     const TO* g = gate ? gate + (size_t)t * p.gate_stride + (size_t)h * p.v_dim : nullptr;
+    quads([&](int d, int i, int n) {
+        float v[4] = {1.f, 1.f, 1.f, 1.f};
+        if (g) {
+            load(g + d, v);
 #pragma unroll
-    for (int i = 0; i < kFinPerLane; ++i) {
-        if (at(i) >= p.v_dim) continue;
-        float v = o[i] * scale;
-        if (g) v *= 1.0f / (1.0f + expf(-to_float(g[at(i)])));
-        dst[at(i)] = from_float<TO>(v);
-    }
+            for (int e = 0; e < (VEC ? 4 : 1); ++e) v[e] = 1.0f / (1.0f + expf(-v[e]));
+        }
+#pragma unroll
+        for (int e = 0; e < (VEC ? 4 : 1); ++e) v[e] *= o[i + e] * scale;
+        if constexpr (VEC) fin_store4(dst + d, v);
+        else dst[d] = from_float<TO>(v[0]);
+    });
 }
 
 }  // namespace mdma
@@ -111,8 +148,16 @@ int mdma_attention_finish(const void* rows, int rows_dtype, const float* part_o,
     if (n_tokens == 0) return 0;
     const FinishParams p = {rows, part_o, part_ml, splits, sink_log2, n_tokens, n_heads, maps, v_dim, lambda, norm_scale, eps, gate_stride, out_scale};
     const unsigned blocks = (unsigned)(((long)n_tokens * n_heads + kFinWarps - 1) / kFinWarps);
-    MDMA_DISPATCH_DTYPE(rows_dtype, TI, MDMA_DISPATCH_DTYPE(out_dtype, TO,
-        launch_chained(attention_finish_kernel<TI, TO>, dim3(blocks), dim3(kFinWarps * 32), 0, stream, p, (const TO*)gate, (TO*)out)));
+    const uintptr_t all = (uintptr_t)rows | (uintptr_t)part_o | (uintptr_t)out;
+    const bool vec = v_dim % 4 == 0 && (all & 15) == 0 && ((uintptr_t)gate & (out_dtype == kF32 ? 15 : 7)) == 0 && (!gate || gate_stride % 4 == 0);
+#define MDMA_FINISH(VEC, NQ)                                                                                                       \
+    launch_chained(attention_finish_kernel<TI, TO, VEC, NQ>, dim3(blocks), dim3(kFinWarps * 32), 0, stream, p, (const TO*)gate, (TO*)out)
+    MDMA_DISPATCH_DTYPE(rows_dtype, TI, MDMA_DISPATCH_DTYPE(out_dtype, TO, {
+        if (!vec) MDMA_FINISH(false, 2);
+        else if (v_dim <= 128) MDMA_FINISH(true, 1);
+        else MDMA_FINISH(true, 2);
+    }));
+#undef MDMA_FINISH
     MDMA_LAUNCH_OK("attention_finish");
     return 0;
 }
