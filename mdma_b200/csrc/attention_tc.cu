@@ -58,6 +58,13 @@ struct AttnTcParams {
 __device__ __forceinline__ float capped_raw(float s, float cap_raw, float cap_rate) {
     return fmaf(-2.0f * cap_raw, __fdividef(1.0f, 1.0f + ptx::ex2_approx(s * cap_rate)), cap_raw);
 }
+// The same where |x| <= kCapSmall, without the special-function unit that the softmax's exponentials keep busy: cap_raw x = s,
+// so the result is s tanh(x) / x with the series 1 - x^2/3 + 2 x^4/15 - 17 x^6/315 + 62 x^8/2835 (the next term is below 1e-8).
+constexpr float kCapSmall = 0.25f;
+__device__ __forceinline__ float capped_raw_small(float s, float x_rate) {
+    const float x = s * x_rate, t = x * x;
+    return s * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 62.0f / 2835.0f, -17.0f / 315.0f), 2.0f / 15.0f), -1.0f / 3.0f), 1.0f);
+}
 
 // shared memory map (bytes), all tiles 1024-aligned:
 //   Q: 2 halves x [128 rows x 128 B]           32 KB
@@ -260,8 +267,18 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             if (i & 1) ptx::mbar_arrive(s_read);              // both blocks of the pair are in registers: S may be overwritten
             const int key0 = block_of(i) * kTcKeys + half * 32;
             if (EXT && p.cap_raw > 0.f) {
+                float a4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                for (int j = 0; j < 32; ++j) sv[j] = capped_raw(sv[j], p.cap_raw, p.cap_rate);
+                for (int j = 0; j < 32; ++j) a4[j & 3] = fmaxf(a4[j & 3], fabsf(sv[j]));
+                const float x_rate = p.cap_rate * 0.34657359027997264f;      // ln(2) / 2
+                // (rows nobody owns may hold anything; a NaN is passed over by fmaxf and masked below either way)
+                if (__all_sync(0xffffffffu, fmaxf(fmaxf(a4[0], a4[1]), fmaxf(a4[2], a4[3])) * x_rate <= kCapSmall)) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) sv[j] = capped_raw_small(sv[j], x_rate);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) sv[j] = capped_raw(sv[j], p.cap_raw, p.cap_rate);
+                }
             }
             if (slope_raw != 0.f) {
 #pragma unroll
