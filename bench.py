@@ -41,6 +41,11 @@ rule, windowed attention whose heads' weights are mixed, retention, dense and
 routed feed-forwards, norms after the sublayers) beside a Tubusun (the other
 model with linear attention and routed experts), a Fizadra (the other one whose
 heads are mixed) and a Llama.
+
+`--compare salipel` does the same for the Salipel architecture (attention within
+chunks, differential attention, a window that keeps the first tokens side by
+side with a matrix memory, dense and routed feed-forwards) beside a Tubusun
+(windowed attention side by side with linear attention) and a Llama.
 """
 from __future__ import annotations
 
